@@ -6,7 +6,7 @@ addresses the same page in every layer of the group, so a request has one block
 table per group, not per layer.  What a page holds may differ between the layers
 of a group (other head counts and sizes): layers with equal entries are stacked in
 one tensor per entry, a *variant* of the group.  Groups with a window give pages back as soon as no later
-query can read them.  Beside the pages, every live request owns one *state
+query can read them (the pages of first tokens that stay visible beside the window are kept).  Beside the pages, every live request owns one *state
 slot*: a row in each fixed-size state tensor that mixers with state declare
 (this architecture's attention declares none; the slot still exists and is
 what ``StepContext.slots`` carries).
@@ -170,7 +170,7 @@ class CacheManager:
     def add_layer(self, layer: int, cache: Optional[PagedCacheSpec], state: Optional[StateSpec],
                   extra: Optional[Dict[str, PagedCacheSpec]] = None) -> None:
         """Declares what one layer keeps.  Layers with equal needs - pages for the same positions, that is the
-        same window and the same positions per entry - share a group (one pool, one block table per request);
+        same window, kept first tokens and positions per entry - share a group (one pool, one block table per request);
         within it, layers whose entries are equal share a variant (one stacked tensor per entry).  ``extra``:
         further paged caches of the layer by name (pooled entries, one per block of positions), each placed in a
         group the same way."""
@@ -184,11 +184,15 @@ class CacheManager:
 
     def _add_paged(self, layer, cache: PagedCacheSpec) -> None:
         for index, group in enumerate(self.groups):
-            if group.spec.window == cache.window and group.spec.stride == cache.stride:
+            if (group.spec.window == cache.window and group.spec.stride == cache.stride
+                    and group.spec.keep_first == cache.keep_first):
                 break
         else:
             window = -1 if cache.window is None else int(cache.window)
-            if cache.stride == 1:
+            if cache.keep_first:
+                index = _rt.check(self._lib.tge_rt_cache_add_group_kept(self._cache, window, int(cache.stride),
+                                                                        int(cache.keep_first)))
+            elif cache.stride == 1:
                 index = _rt.check(self._lib.tge_rt_cache_add_group(self._cache, window))
             else:
                 index = _rt.check(self._lib.tge_rt_cache_add_group_strided(self._cache, window, int(cache.stride)))

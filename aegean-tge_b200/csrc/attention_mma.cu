@@ -15,7 +15,9 @@
 // splits in split order.
 //
 // Masking is by absolute position: key t is visible to the query at position p
-// when t <= p and, with a window w > 0, t > p - w.
+// when t <= p and, with a window w > 0, t > p - w or t < keep_first (the first
+// tokens of a request stay visible beside its window): a block then visits the
+// tiles of the kept tokens and those of the window, and skips what lies between.
 #include <cuda.h>
 
 #include <stdlib.h>
@@ -69,6 +71,9 @@ struct AttnParams {
   int early_tiles;           // decode: key tiles of settled positions asked for before the dependency wait (0: none)
   int heads, kv_heads, group, bq;
   int window, split_tokens, num_splits;
+  int keep_first;            // with a window: the first so many positions stay visible (0: none)
+  const __nv_bfloat16* gate; // null, or [tokens, heads] logits: a head's output is multiplied by their logistic function
+  int gate_stride;
   float scale_log2;
 };
 
@@ -77,6 +82,41 @@ __device__ __forceinline__ uint32_t smem_u32(const void* p) { return (uint32_t)_
 // The bias of `head` for the key `distance` positions back, in base-2 units like a scaled score.
 __device__ __forceinline__ float distance_bias(const AttnParams& p, int head, int distance) {
   return p.dist_bias[(size_t)head * p.dist_span + min(max(distance, 0), p.dist_span - 1)] * LOG2E;
+}
+
+// The keys a block visits, in its run [first, last) of positions (the whole request when the keys are not cut): the tiles
+// of the kept first tokens, then those from the start of the window (of the block's first query) on.
+struct KeyTiles {
+  int lo, hi;                // the window's part: [lo, hi)
+  int keep;                  // positions below this are visible beside it (0: none)
+  int kept_tiles, kept_first, k_first, num_tiles;
+  __device__ __forceinline__ KeyTiles(const AttnParams& p, int pos0, int q_count, int split) {
+    int first = 0, last = 0x7fffffff;
+    if (p.num_splits > 1) {
+      first = split * p.split_tokens;
+      last = first + p.split_tokens;
+    }
+    lo = max(p.window > 0 ? max(pos0 - p.window + 1, 0) : 0, first);
+    hi = min(pos0 + q_count, last);
+    keep = p.window > 0 ? min(p.keep_first, hi) : 0;
+    kept_first = first;
+    kept_tiles = keep > first && lo > first ? (keep - first + BKV - 1) / BKV : 0;
+    k_first = lo / BKV * BKV;
+    if (kept_tiles > 0) k_first = max(k_first, first + kept_tiles * BKV);
+    num_tiles = kept_tiles + (lo < hi && k_first < hi ? (hi - k_first + BKV - 1) / BKV : 0);
+  }
+  __device__ __forceinline__ int start(int tile) const {
+    return tile < kept_tiles ? kept_first + tile * BKV : k_first + (tile - kept_tiles) * BKV;
+  }
+  __device__ __forceinline__ bool visible(int kpos) const { return (kpos >= lo || kpos < keep) && kpos < hi; }
+  // a visible position of a run of keys from k0 on, if it has any
+  __device__ __forceinline__ int probe(int k0) const { return k0 < keep ? k0 : max(k0, lo); }
+};
+
+// What a head's gate multiplies its output by.
+__device__ __forceinline__ float head_gate(const AttnParams& p, int token, int head) {
+  if (p.gate == nullptr) return 1.0f;
+  return 1.0f / (1.0f + __expf(-__bfloat162float(p.gate[(size_t)token * p.gate_stride + head])));
 }
 
 // The denominator `l` (relative to the running maximum `m_log2`, in base-2 units) with the head's sink in it.
@@ -113,10 +153,10 @@ __device__ __forceinline__ uint32_t pack_bf16(float lo, float hi) {
 }
 
 // Copies positions [k0, k0 + BKV) of one kv head into a shared tile; positions
-// outside [lo, hi) are zero-filled so that masked columns never meet NaNs.
+// the block does not see are zero-filled so that masked columns never meet NaNs.
 template <int NWARPS, int WIDTH = HD>
 __device__ __forceinline__ void load_tile(const AttnParams& p, const __nv_bfloat16* pages, const int* table, int kvh,
-                                          __nv_bfloat16* tile, int k0, int lo, int hi, bool& bad_page, int pitch = WIDTH) {
+                                          __nv_bfloat16* tile, int k0, const KeyTiles& keys, bool& bad_page, int pitch = WIDTH) {
   constexpr int CHUNKS = WIDTH / 8;      // 16-byte chunks per row
   for (int c = threadIdx.x; c < BKV * CHUNKS; c += NWARPS * 32) {
     const int j = c / CHUNKS, part = c - j * CHUNKS;
@@ -124,7 +164,7 @@ __device__ __forceinline__ void load_tile(const AttnParams& p, const __nv_bfloat
     const uint32_t dst = smem_u32(tile + j * (WIDTH + 8) + part * 8);
     const void* src = pages;
     int bytes = 0;
-    if (kpos >= lo && kpos < hi) {
+    if (keys.visible(kpos)) {
       const int page_index = kpos >> p.page_shift;
       const int page = page_index < p.max_pages ? table[page_index] : -1;
       if (page >= 0 && page < p.num_pages) {
@@ -174,13 +214,8 @@ __global__ void __launch_bounds__(NWARPS * 32) attention_mma_kernel(const AttnPa
   const int* table = p.block_table + (size_t)seq * p.max_pages;
 
   // key range of the block: union over its rows, cut to this split
-  int lo = p.window > 0 ? max(pos0 - p.window + 1, 0) : 0;
-  int hi = pos0 + q_count;                                 // exclusive
-  if (p.num_splits > 1) {
-    lo = max(lo, split * p.split_tokens);
-    hi = min(hi, (split + 1) * p.split_tokens);
-  }
-  if (lo >= hi) return;
+  const KeyTiles keys(p, pos0, q_count, split);
+  if (keys.num_tiles <= 0) return;
 
   // this thread's two rows
   int row_token[2], row_pos[2], row_head[2];
@@ -215,18 +250,17 @@ __global__ void __launch_bounds__(NWARPS * 32) attention_mma_kernel(const AttnPa
   float m_run[2] = {-INFINITY, -INFINITY}, l_run[2] = {0.0f, 0.0f};
 
   bool bad_page = false;
-  const int k_first = lo / BKV * BKV;
-  const int num_tiles = (hi - k_first + BKV - 1) / BKV;
-  load_tile<NWARPS>(p, p.k_pages, table, kvh, sK, k_first, lo, hi, bad_page);
-  load_tile<NWARPS, DV>(p, p.v_pages, table, kvh, sV, k_first, lo, hi, bad_page, p.v_pitch);
+  const int num_tiles = keys.num_tiles;
+  load_tile<NWARPS>(p, p.k_pages, table, kvh, sK, keys.start(0), keys, bad_page);
+  load_tile<NWARPS, DV>(p, p.v_pages, table, kvh, sV, keys.start(0), keys, bad_page, p.v_pitch);
   cp_async_commit();
 
   for (int it = 0; it < num_tiles; ++it) {
     const int stage = it & 1;
-    const int k0 = k_first + it * BKV;
+    const int k0 = keys.start(it);
     if (it + 1 < num_tiles) {
-      load_tile<NWARPS>(p, p.k_pages, table, kvh, sK + (stage ^ 1) * BKV * ROW_ELEMS, k0 + BKV, lo, hi, bad_page);
-      load_tile<NWARPS, DV>(p, p.v_pages, table, kvh, sV + (stage ^ 1) * BKV * V_ROW_ELEMS, k0 + BKV, lo, hi, bad_page, p.v_pitch);
+      load_tile<NWARPS>(p, p.k_pages, table, kvh, sK + (stage ^ 1) * BKV * ROW_ELEMS, keys.start(it + 1), keys, bad_page);
+      load_tile<NWARPS, DV>(p, p.v_pages, table, kvh, sV + (stage ^ 1) * BKV * V_ROW_ELEMS, keys.start(it + 1), keys, bad_page, p.v_pitch);
       cp_async_commit();
       cp_async_wait<1>();
     } else {
@@ -267,7 +301,7 @@ __global__ void __launch_bounds__(NWARPS * 32) attention_mma_kernel(const AttnPa
 #pragma unroll
         for (int e = 0; e < 2; ++e) {
           const int kpos = k0 + n * 8 + 2 * t4 + e;
-          const bool visible = row_valid[i] && kpos <= row_pos[i] && kpos >= first_key && kpos >= lo && kpos < hi;
+          const bool visible = row_valid[i] && kpos <= row_pos[i] && (kpos >= first_key || kpos < keys.keep) && keys.visible(kpos);
           float s = -INFINITY;
           if (visible) {
             s = s_acc[n][2 * i + e] * p.scale_log2;
@@ -335,7 +369,7 @@ __global__ void __launch_bounds__(NWARPS * 32) attention_mma_kernel(const AttnPa
     if (!row_valid[i]) continue;
     if (p.num_splits == 1) {
       const float l_all = with_sink(p, row_head[i], m_run[i], l_run[i]);
-      const float inv = l_all > 0.0f ? 1.0f / l_all : 0.0f;
+      const float inv = (l_all > 0.0f ? 1.0f / l_all : 0.0f) * head_gate(p, row_token[i], row_head[i]);
       __nv_bfloat16* dst = p.out + (size_t)row_token[i] * p.out_stride + (size_t)row_head[i] * DV;
 #pragma unroll
       for (int d = 0; d < DV / 8; ++d) {
@@ -379,18 +413,14 @@ __global__ void __launch_bounds__(DEC_WARPS * 32) attention_decode_kernel(const 
   const int token = p.q_start[seq];
   const int pos = p.start_pos[seq];
 
-  int lo = p.window > 0 ? max(pos - p.window + 1, 0) : 0;
-  int hi = pos + 1;
-  if (p.num_splits > 1) {
-    lo = max(lo, split * p.split_tokens);
-    hi = min(hi, (split + 1) * p.split_tokens);
-  }
-  if (lo >= hi) return;
+  const KeyTiles keys(p, pos, 1, split);
+  if (keys.num_tiles <= 0) return;
+  const int lo = keys.lo, hi = keys.hi;
 
   // The page ids of this block's key range, fetched once: the copy loops then index shared memory.
   // (The staged row is addressed like the global one, so ids before first_page are never read.)
   int* local_table = reinterpret_cast<int*>(smem_raw + (size_t)DEC_STAGES * STAGE_ELEMS * sizeof(__nv_bfloat16));
-  const int first_page = lo >> p.page_shift, last_page = (hi - 1) >> p.page_shift;
+  const int first_page = keys.probe(keys.start(0)) >> p.page_shift, last_page = (hi - 1) >> p.page_shift;
   for (int i = first_page + tid; i <= last_page; i += DEC_WARPS * 32)
     local_table[i - first_page] = i < p.max_pages ? p.block_table[(size_t)seq * p.max_pages + i] : -1;
   __syncthreads();
@@ -417,13 +447,12 @@ __global__ void __launch_bounds__(DEC_WARPS * 32) attention_decode_kernel(const 
   float m_run[2] = {-INFINITY, -INFINITY}, l_run[2] = {0.0f, 0.0f};
 
   bool bad_page = false;
-  const int k_first = lo / BKV * BKV;
-  const int num_tiles = (hi - k_first + BKV - 1) / BKV;
+  const int num_tiles = keys.num_tiles;
 #pragma unroll
   for (int s = 0; s < DEC_STAGES - 1; ++s) {
     if (s < num_tiles) {
-      load_tile<DEC_WARPS>(p, p.k_pages, table, kvh, stages + s * STAGE_ELEMS, k_first + s * BKV, lo, hi, bad_page);
-      load_tile<DEC_WARPS, DV>(p, p.v_pages, table, kvh, stages + s * STAGE_ELEMS + BKV * ROW_ELEMS, k_first + s * BKV, lo, hi, bad_page, p.v_pitch);
+      load_tile<DEC_WARPS>(p, p.k_pages, table, kvh, stages + s * STAGE_ELEMS, keys.start(s), keys, bad_page);
+      load_tile<DEC_WARPS, DV>(p, p.v_pages, table, kvh, stages + s * STAGE_ELEMS + BKV * ROW_ELEMS, keys.start(s), keys, bad_page, p.v_pitch);
     }
     cp_async_commit();
   }
@@ -434,15 +463,15 @@ __global__ void __launch_bounds__(DEC_WARPS * 32) attention_decode_kernel(const 
       const int next = it + DEC_STAGES - 1;
       if (next < num_tiles) {
         __nv_bfloat16* dst = stages + (next % DEC_STAGES) * STAGE_ELEMS;
-        load_tile<DEC_WARPS>(p, p.k_pages, table, kvh, dst, k_first + next * BKV, lo, hi, bad_page);
-        load_tile<DEC_WARPS, DV>(p, p.v_pages, table, kvh, dst + BKV * ROW_ELEMS, k_first + next * BKV, lo, hi, bad_page, p.v_pitch);
+        load_tile<DEC_WARPS>(p, p.k_pages, table, kvh, dst, keys.start(next), keys, bad_page);
+        load_tile<DEC_WARPS, DV>(p, p.v_pages, table, kvh, dst + BKV * ROW_ELEMS, keys.start(next), keys, bad_page, p.v_pitch);
       }
       cp_async_commit();
     }
     const __nv_bfloat16* tK = stages + (it % DEC_STAGES) * STAGE_ELEMS;
     const __nv_bfloat16* tV = tK + BKV * ROW_ELEMS;
-    const int k0 = k_first + it * BKV + warp * 16;     // this warp's 16 positions
-    if (k0 >= hi || k0 + 16 <= lo) continue;            // nothing visible in this slice (warp-uniform)
+    const int k0 = keys.start(it) + warp * 16;          // this warp's 16 positions
+    if (k0 >= hi || (k0 + 16 <= lo && k0 >= keys.keep)) continue;   // nothing visible in this slice (warp-uniform)
 
     float s_acc[2][4];
 #pragma unroll
@@ -469,7 +498,7 @@ __global__ void __launch_bounds__(DEC_WARPS * 32) attention_decode_kernel(const 
 #pragma unroll
         for (int e = 0; e < 2; ++e) {
           const int kpos = k0 + n * 8 + 2 * t4 + e;
-          const bool visible = row_valid && kpos >= lo && kpos < hi;
+          const bool visible = row_valid && keys.visible(kpos);
           float sv = -INFINITY;
           if (visible) {
             sv = s_acc[n][2 * i + e] * p.scale_log2;
@@ -555,7 +584,8 @@ __global__ void __launch_bounds__(DEC_WARPS * 32) attention_decode_kernel(const 
     const int head = kvh * p.group + r;
     if (p.num_splits == 1) {
       const float l_all = with_sink(p, head, m, l);
-      p.out[(size_t)token * p.out_stride + (size_t)head * DV + d] = __float2bfloat16_rn(l_all > 0.0f ? acc / l_all : 0.0f);
+      p.out[(size_t)token * p.out_stride + (size_t)head * DV + d] =
+          __float2bfloat16_rn((l_all > 0.0f ? acc / l_all : 0.0f) * head_gate(p, token, head));
     } else {
       const size_t slot = ((size_t)split * p.total_tokens + token) * p.heads + head;
       p.partial_o[slot * DV + d] = acc;
@@ -653,18 +683,13 @@ __global__ void __launch_bounds__((4 * GROUPS + 1) * 32) attention_decode_tma_ke
   const int seq = blockIdx.x, kvh = blockIdx.y, split = blockIdx.z;
   const int token = p.q_start[seq];
   const int pos = p.start_pos[seq];
-  int lo = p.window > 0 ? max(pos - p.window + 1, 0) : 0;
-  int hi = pos + 1;
-  if (p.num_splits > 1) {
-    lo = max(lo, split * p.split_tokens);
-    hi = min(hi, (split + 1) * p.split_tokens);
-  }
-  if (lo >= hi) return;
+  const KeyTiles keys(p, pos, 1, split);
+  if (keys.num_tiles <= 0) return;
+  const int lo = keys.lo, hi = keys.hi;
 
-  const int k_first = lo / BKV * BKV;
-  const int num_tiles = (hi - k_first + BKV - 1) / BKV;
-  const int first_page = k_first >> p.page_shift;
-  const int last_page = (k_first + num_tiles * BKV - 1) >> p.page_shift;
+  const int num_tiles = keys.num_tiles;
+  const int first_page = keys.start(0) >> p.page_shift;
+  const int last_page = (keys.start(num_tiles - 1) + BKV - 1) >> p.page_shift;
   for (int i = first_page + tid; i <= last_page; i += THREADS) {
     int page = i < p.max_pages ? p.block_table[(size_t)seq * p.max_pages + i] : -1;
     if (page >= p.num_pages) page = -2;                                // reported below, never fetched
@@ -693,15 +718,16 @@ __global__ void __launch_bounds__((4 * GROUPS + 1) * 32) attention_decode_tma_ke
     const int stage = tile % STAGES;
     const uint32_t k_dst = base + stage * TMA_STAGE_BYTES, v_dst = k_dst + TMA_TILE_BYTES;
     const uint32_t bar = full_bar(stage);
+    const int tile_first = keys.start(tile);
     int boxes = 0;
     for (int j = 0; j < pages_per_tile; ++j) {
-      const int page = local_table[((k_first + tile * BKV) >> p.page_shift) + j - first_page];
-      if (page >= 0 && (k_first + tile * BKV + (j << p.page_shift)) < hi) ++boxes;
+      const int page = local_table[(tile_first >> p.page_shift) + j - first_page];
+      if (page >= 0 && (tile_first + (j << p.page_shift)) < hi) ++boxes;
     }
     mbar_expect_tx(bar, (uint32_t)boxes * 2u * TMA_BLOCKS * (uint32_t)(p.page_size * 128));
     for (int j = 0; j < pages_per_tile; ++j) {
-      const int page = local_table[((k_first + tile * BKV) >> p.page_shift) + j - first_page];
-      if (page < 0 || (k_first + tile * BKV + (j << p.page_shift)) >= hi) continue;
+      const int page = local_table[(tile_first >> p.page_shift) + j - first_page];
+      if (page < 0 || (tile_first + (j << p.page_shift)) >= hi) continue;
       const int row = (page * p.kv_heads + kvh) << p.page_shift;
 #pragma unroll
       for (int b = 0; b < TMA_BLOCKS; ++b) {
@@ -716,9 +742,8 @@ __global__ void __launch_bounds__((4 * GROUPS + 1) * 32) attention_decode_tma_ke
     // block-wide.  A stage is refilled once all computing warps have released it.
     if (elect_one()) {
       // tiles that end before this step's own position hold nothing this step writes
-      const int settled = pos >= k_first ? (pos - k_first) / BKV : 0;
       int tile = 0;
-      for (; tile < num_tiles && tile < p.early_tiles && tile < settled; ++tile) issue(tile);
+      for (; tile < num_tiles && tile < p.early_tiles && keys.start(tile) + BKV <= pos; ++tile) issue(tile);
       pdl_wait();
       for (; tile < num_tiles; ++tile) {
         if (tile >= STAGES)
@@ -752,16 +777,16 @@ __global__ void __launch_bounds__((4 * GROUPS + 1) * 32) attention_decode_tma_ke
   const int group = warp >> 2, w4 = warp & 3;            // this warp's group and its quarter of a tile's keys
   for (int it = group; it < (warp < WARPS ? num_tiles : 0); it += GROUPS) {
     const int stage = it % STAGES;
-    const int k0 = k_first + it * BKV + w4 * 16;
+    const int k0 = keys.start(it) + w4 * 16;
     // every warp sees every copy land, also of tiles it has no visible position in: the parity of a wait
     // only tells phases apart while nobody is a whole phase behind
     mbar_wait_bounded(full_bar(stage), (uint32_t)(it / STAGES) & 1u, p.status);
-    if (k0 >= hi || k0 + 16 <= lo) {
+    if (k0 >= hi || (k0 + 16 <= lo && k0 >= keys.keep)) {
       if (lane == 0) mbar_arrive(empty_bar(stage));
       continue;
     }
     const uint32_t tK = base + stage * TMA_STAGE_BYTES, tV = tK + TMA_TILE_BYTES;
-    if (local_table[(max(k0, lo) >> p.page_shift) - first_page] < 0) bad_page = true;   // a visible position without a page
+    if (local_table[(keys.probe(k0) >> p.page_shift) - first_page] < 0) bad_page = true;   // a visible position without a page
 
     float s_acc[2][4];
 #pragma unroll
@@ -787,7 +812,7 @@ __global__ void __launch_bounds__((4 * GROUPS + 1) * 32) attention_decode_tma_ke
 #pragma unroll
         for (int e = 0; e < 2; ++e) {
           const int kpos = k0 + n * 8 + 2 * t4 + e;
-          const bool visible = row_valid && kpos >= lo && kpos < hi;
+          const bool visible = row_valid && keys.visible(kpos);
           float sv = -INFINITY;
           if (visible) {
             sv = s_acc[n][2 * i + e] * p.scale_log2;
@@ -875,7 +900,8 @@ __global__ void __launch_bounds__((4 * GROUPS + 1) * 32) attention_decode_tma_ke
     const int head = kvh * p.group + r;
     if (p.num_splits == 1) {
       const float l_all = with_sink(p, head, m, l);
-      p.out[(size_t)token * p.out_stride + (size_t)head * HD + d] = __float2bfloat16_rn(l_all > 0.0f ? acc / l_all : 0.0f);
+      p.out[(size_t)token * p.out_stride + (size_t)head * HD + d] =
+          __float2bfloat16_rn((l_all > 0.0f ? acc / l_all : 0.0f) * head_gate(p, token, head));
     } else {
       const size_t slot = ((size_t)split * p.total_tokens + token) * p.heads + head;
       p.partial_o[slot * HD + d] = acc;
@@ -936,18 +962,13 @@ __global__ void __launch_bounds__(PRE_THREADS) attention_prefill_tma_kernel(
   const int q_count = min(p.bq, q_len - q_first);
   const int pos0 = p.start_pos[seq] + q_first;
 
-  int lo = p.window > 0 ? max(pos0 - p.window + 1, 0) : 0;
-  int hi = pos0 + q_count;
-  if (p.num_splits > 1) {
-    lo = max(lo, split * p.split_tokens);
-    hi = min(hi, (split + 1) * p.split_tokens);
-  }
-  if (lo >= hi) return;
+  const KeyTiles keys(p, pos0, q_count, split);
+  if (keys.num_tiles <= 0) return;
+  const int lo = keys.lo, hi = keys.hi;
 
-  const int k_first = lo / BKV * BKV;
-  const int num_tiles = (hi - k_first + BKV - 1) / BKV;
-  const int first_page = k_first >> p.page_shift;
-  const int last_page = (k_first + num_tiles * BKV - 1) >> p.page_shift;
+  const int num_tiles = keys.num_tiles;
+  const int first_page = keys.start(0) >> p.page_shift;
+  const int last_page = (keys.start(num_tiles - 1) + BKV - 1) >> p.page_shift;
   for (int i = first_page + tid; i <= last_page; i += PRE_THREADS) {
     int page = i < p.max_pages ? p.block_table[(size_t)seq * p.max_pages + i] : -1;
     if (page >= p.num_pages) page = -2;
@@ -972,15 +993,16 @@ __global__ void __launch_bounds__(PRE_THREADS) attention_prefill_tma_kernel(
     const int stage = tile % PRE_STAGES;
     const uint32_t k_dst = base + stage * TMA_STAGE_BYTES, v_dst = k_dst + TMA_TILE_BYTES;
     const uint32_t bar = bars + 8 * stage;
+    const int tile_first = keys.start(tile);
     int boxes = 0;
     for (int j = 0; j < pages_per_tile; ++j) {
-      const int page = local_table[((k_first + tile * BKV) >> p.page_shift) + j - first_page];
-      if (page >= 0 && (k_first + tile * BKV + (j << p.page_shift)) < hi) ++boxes;
+      const int page = local_table[(tile_first >> p.page_shift) + j - first_page];
+      if (page >= 0 && (tile_first + (j << p.page_shift)) < hi) ++boxes;
     }
     mbar_expect_tx(bar, (uint32_t)boxes * 2u * TMA_BLOCKS * (uint32_t)(p.page_size * 128));
     for (int j = 0; j < pages_per_tile; ++j) {
-      const int page = local_table[((k_first + tile * BKV) >> p.page_shift) + j - first_page];
-      if (page < 0 || (k_first + tile * BKV + (j << p.page_shift)) >= hi) continue;
+      const int page = local_table[(tile_first >> p.page_shift) + j - first_page];
+      if (page < 0 || (tile_first + (j << p.page_shift)) >= hi) continue;
       const int row = (page * p.kv_heads + kvh) << p.page_shift;
 #pragma unroll
       for (int b = 0; b < TMA_BLOCKS; ++b) {
@@ -1040,15 +1062,15 @@ __global__ void __launch_bounds__(PRE_THREADS) attention_prefill_tma_kernel(
     const int stage = it % PRE_STAGES;
     mbar_wait_bounded(bars + 8 * stage, (uint32_t)(it / PRE_STAGES) & 1u, p.status);
     const uint32_t tK = base + stage * TMA_STAGE_BYTES, tV = tK + TMA_TILE_BYTES;
-    const int k0 = k_first + it * BKV;
+    const int k0 = keys.start(it);
     // nothing in this tile is visible to this warp's rows (before their windows or after their positions):
     // release the stage at once
-    const bool skip = !warp_active || k0 > warp_pos_hi || (p.window > 0 && k0 + BKV <= warp_pos_lo - p.window + 1);
+    const bool skip = !warp_active || k0 > warp_pos_hi || (p.window > 0 && k0 + BKV <= warp_pos_lo - p.window + 1 && k0 >= keys.keep);
     if (skip) {
       if (lane == 0) mbar_arrive(bars + 8 * (PRE_STAGES + stage));
       continue;
     }
-    if (local_table[(max(k0, lo) >> p.page_shift) - first_page] < 0) bad_page = true;
+    if (local_table[(keys.probe(k0) >> p.page_shift) - first_page] < 0) bad_page = true;
 
     float s_acc[BKV / 8][4];
 #pragma unroll
@@ -1068,8 +1090,8 @@ __global__ void __launch_bounds__(PRE_THREADS) attention_prefill_tma_kernel(
       }
     }
     // a tile wholly inside [lo, hi), before every row's position and inside every row's window needs no mask
-    const bool clean = k0 >= lo && k0 + BKV <= hi && k0 + BKV - 1 <= warp_pos_lo &&
-                       (p.window == 0 || k0 >= warp_pos_hi - p.window + 1) && warp_q_hi < q_count &&
+    const bool clean = k0 + BKV <= hi && k0 + BKV - 1 <= warp_pos_lo &&
+                       ((k0 >= lo && (p.window == 0 || k0 >= warp_pos_hi - p.window + 1)) || k0 + BKV <= keys.keep) && warp_q_hi < q_count &&
                        (warp * 16 + 15) / p.group < q_count;
     float corr[2];
 #pragma unroll
@@ -1084,7 +1106,7 @@ __global__ void __launch_bounds__(PRE_THREADS) attention_prefill_tma_kernel(
           if (p.dist_bias != nullptr) sv += distance_bias(p, row_head[i], row_pos[i] - (k0 + n * 8 + 2 * t4 + e));
           if (!clean) {
             const int kpos = k0 + n * 8 + 2 * t4 + e;
-            const bool visible = row_valid[i] && kpos <= row_pos[i] && kpos >= first_key && kpos >= lo && kpos < hi;
+            const bool visible = row_valid[i] && kpos <= row_pos[i] && (kpos >= first_key || kpos < keys.keep) && keys.visible(kpos);
             sv = visible ? sv : -INFINITY;
           }
           s_acc[n][2 * i + e] = sv;
@@ -1148,7 +1170,7 @@ __global__ void __launch_bounds__(PRE_THREADS) attention_prefill_tma_kernel(
     if (!row_valid[i]) continue;
     if (p.num_splits == 1) {
       const float l_all = with_sink(p, row_head[i], m_run[i], l_run[i]);
-      const float inv = l_all > 0.0f ? 1.0f / l_all : 0.0f;
+      const float inv = (l_all > 0.0f ? 1.0f / l_all : 0.0f) * head_gate(p, row_token[i], row_head[i]);
       __nv_bfloat16* dst = p.out + (size_t)row_token[i] * p.out_stride + (size_t)row_head[i] * HD;
 #pragma unroll
       for (int d = 0; d < HD / 8; ++d)
@@ -1216,12 +1238,14 @@ template <int HELD>                                                  // splits w
 __global__ void attention_merge_kernel(const float* __restrict__ partial_o, const float* __restrict__ partial_ml,
                                        const int* __restrict__ positions, __nv_bfloat16* __restrict__ out,
                                        int out_stride, int total_tokens, int heads, int window, int split_tokens,
-                                       int num_splits, int first_token, const float* __restrict__ sink) {
+                                       int num_splits, int first_token, const float* __restrict__ sink, int keep_first,
+                                       const __nv_bfloat16* __restrict__ gate, int gate_stride) {
   pdl_trigger();
   const int t = blockIdx.x + first_token, h = blockIdx.y;
   const int pos = positions[t];                                     // given to the step: not the previous kernel's work
   const float sink_log2 = sink != nullptr ? sink[h] * LOG2E : -INFINITY;   // the sink joins the merged denominator once
   pdl_wait();
+  const float factor = gate != nullptr ? 1.0f / (1.0f + __expf(-__bfloat162float(gate[(size_t)t * gate_stride + h]))) : 1.0f;
   const size_t stride = (size_t)total_tokens * heads;               // slots per split
   const size_t slot0 = (size_t)t * heads + h;
   if (num_splits <= HELD) {
@@ -1242,7 +1266,7 @@ __global__ void attention_merge_kernel(const float* __restrict__ partial_o, cons
       for (int i = 0; i < HELD; ++i) o[i] = i < num_splits ? partial_o[((size_t)i * stride + slot0) * DV + d] : 0.0f;
 #pragma unroll
       for (int i = 0; i < HELD; ++i) {
-        const bool live = i >= s_lo && i <= s_hi;
+        const bool live = i <= s_hi && (i >= s_lo || i * split_tokens < keep_first);
         ml[i] = live ? ml[i] : make_float2(-INFINITY, 0.0f);
         o[i] = live ? o[i] : 0.0f;
       }
@@ -1258,26 +1282,34 @@ __global__ void attention_merge_kernel(const float* __restrict__ partial_o, cons
         acc += scale * o[i];
       }
       if (sink != nullptr) l += exp2f(sink_log2 - m_use);
-      out[(size_t)t * out_stride + (size_t)h * DV + d] = __float2bfloat16_rn(acc * (l > 0.0f ? 1.0f / l : 0.0f));
+      out[(size_t)t * out_stride + (size_t)h * DV + d] = __float2bfloat16_rn(acc * (l > 0.0f ? 1.0f / l : 0.0f) * factor);
     }
     return;
   }
   const int first_key = window > 0 ? max(pos - window + 1, 0) : 0;
   const int s_lo = first_key / split_tokens;
   const int s_hi = min(pos / split_tokens, num_splits - 1);
+  // the runs of the kept first tokens, then those of the window
+  const int kept_runs = min(s_lo, (keep_first + split_tokens - 1) / split_tokens);
+  const int skipped = s_lo - kept_runs;
   float m = -INFINITY;
-  for (int s = s_lo; s <= s_hi; ++s) m = fmaxf(m, partial_ml[((size_t)s * stride + slot0) * 2]);
+  for (int i = 0; i <= s_hi - skipped; ++i) {
+    const int s = i < kept_runs ? i : i + skipped;
+    m = fmaxf(m, partial_ml[((size_t)s * stride + slot0) * 2]);
+  }
   const float m_use = m == -INFINITY ? 0.0f : m;
   float l = 0.0f;
-  for (int s = s_lo; s <= s_hi; ++s) {
+  for (int i = 0; i <= s_hi - skipped; ++i) {
+    const int s = i < kept_runs ? i : i + skipped;
     const size_t slot = (size_t)s * stride + slot0;
     l += exp2f(partial_ml[slot * 2] - m_use) * partial_ml[slot * 2 + 1];
   }
   if (sink != nullptr) l += exp2f(sink_log2 - m_use);
-  const float inv = l > 0.0f ? 1.0f / l : 0.0f;
+  const float inv = (l > 0.0f ? 1.0f / l : 0.0f) * factor;
   for (int d = threadIdx.x; d < DV; d += blockDim.x) {
     float acc = 0.0f;
-    for (int s = s_lo; s <= s_hi; ++s) {
+    for (int i = 0; i <= s_hi - skipped; ++i) {
+      const int s = i < kept_runs ? i : i + skipped;
       const size_t slot = (size_t)s * stride + slot0;
       acc += exp2f(partial_ml[slot * 2] - m_use) * partial_o[slot * DV + d];
     }
@@ -1287,16 +1319,16 @@ __global__ void attention_merge_kernel(const float* __restrict__ partial_o, cons
 
 // Sixteen states in registers serve most steps; a single long request cut into up to 48 splits takes the wider
 // instance, and beyond that the kernel walks the splits in a loop.
-void launch_merge(dim3 grid, cudaStream_t stream, const float* partial_o, const float* partial_ml, const int* positions,
-                  __nv_bfloat16* out, int out_stride, int total_tokens, int heads, int window, int split_tokens,
-                  int num_splits, int first_token, const float* sink) {
+void launch_merge(const AttnParams& p, const int* positions, int first_token, cudaStream_t stream) {
+  const dim3 grid(p.total_tokens - first_token, p.heads);
   const int threads = DV >= 128 ? 128 : (DV >= 64 ? 64 : 32);
-  if (num_splits <= 16)
-    tge_launch(attention_merge_kernel<16>, grid, threads, 0, stream, partial_o, partial_ml, positions, out, out_stride,
-               total_tokens, heads, window, split_tokens, num_splits, first_token, sink);
-  else
-    tge_launch(attention_merge_kernel<48>, grid, threads, 0, stream, partial_o, partial_ml, positions, out, out_stride,
-               total_tokens, heads, window, split_tokens, num_splits, first_token, sink);
+  auto run = [&](auto kernel) {
+    tge_launch(kernel, grid, threads, 0, stream, (const float*)p.partial_o, (const float*)p.partial_ml, positions, p.out, p.out_stride,
+               p.total_tokens, p.heads, p.window, p.split_tokens, p.num_splits, first_token, p.sink, p.keep_first, p.gate,
+               p.gate_stride);
+  };
+  if (p.num_splits <= 16) run(attention_merge_kernel<16>);
+  else run(attention_merge_kernel<48>);
 }
 
 template <int NWARPS>
@@ -1338,7 +1370,7 @@ static int attention_dispatch(const void* q, int q_stride, const void* k_pages, 
                               int tokens, int max_q_len, int max_ctx_len, void* out, int out_stride, int heads,
                               int kv_heads, float scale, int window, int split_tokens, float* scratch, int* status,
                               int first_token, const float* sink, int leave_states, int v_pitch, const float* dist_bias,
-                              int dist_span, cudaStream_t stream) {
+                              int dist_span, int keep_first, const void* gate, int gate_stride, cudaStream_t stream) {
   TGE_REQUIRE(tokens >= 0 && num_seqs >= 0, "attention_mma: negative sizes");
   TGE_REQUIRE(dist_bias == nullptr || (dist_span > 0 && scale != 0.0f), "attention_mma: a bias by distance needs its span");
   TGE_REQUIRE(heads > 0 && kv_heads > 0 && heads % kv_heads == 0,
@@ -1358,6 +1390,11 @@ static int attention_dispatch(const void* q, int q_stride, const void* k_pages, 
   p.out = (__nv_bfloat16*)out; p.status = status; p.sink = sink;
   p.dist_bias = dist_bias; p.dist_span = dist_span; p.bias_to_raw = dist_bias != nullptr ? 1.0f / scale : 0.0f;
   p.leave_states = leave_states;
+  TGE_REQUIRE(keep_first >= 0 && (gate == nullptr || gate_stride >= heads), "attention_mma: %d kept positions, gate rows of %d for %d heads",
+              keep_first, gate_stride, heads);
+  TGE_REQUIRE(!leave_states || (keep_first == 0 && gate == nullptr), "attention_mma: kept first tokens and gates go without pooled blocks");
+  p.keep_first = window > 0 ? keep_first : 0;
+  p.gate = (const __nv_bfloat16*)gate; p.gate_stride = gate_stride;
   if (v_pitch == 0) v_pitch = DV;
   TGE_REQUIRE(v_pitch >= DV && v_pitch % 8 == 0, "attention_mma: a value pitch of %d (values of %d) must be a multiple of 8", v_pitch, DV);
   TGE_REQUIRE(v_pitch == DV || !(TGE_TMA_KERNELS), "attention_mma: values inside the keys' entries are not served at equal sizes");
@@ -1418,8 +1455,7 @@ static int attention_dispatch(const void* q, int q_stride, const void* k_pages, 
     int rc = tge_check_launch("attention_decode_tma");
     if (rc != 0) return rc;
     if (num_splits > 1 && !p.leave_states) {
-      dim3 mgrid(tokens - first_token, heads);
-      launch_merge(mgrid, stream, p.partial_o, p.partial_ml, positions, p.out, out_stride, tokens, heads, window, p.split_tokens, num_splits, first_token, p.sink);
+      launch_merge(p, positions, first_token, stream);
       return tge_launched("attention_merge", 2);
     }
     return 1;
@@ -1445,8 +1481,7 @@ static int attention_dispatch(const void* q, int q_stride, const void* k_pages, 
     int rc = tge_check_launch("attention_decode");
     if (rc != 0) return rc;
     if (num_splits > 1 && !p.leave_states) {
-      dim3 mgrid(tokens - first_token, heads);
-      launch_merge(mgrid, stream, p.partial_o, p.partial_ml, positions, p.out, out_stride, tokens, heads, window, p.split_tokens, num_splits, first_token, p.sink);
+      launch_merge(p, positions, first_token, stream);
       return tge_launched("attention_merge", 2);
     }
     return 1;
@@ -1481,8 +1516,7 @@ static int attention_dispatch(const void* q, int q_stride, const void* k_pages, 
         int rc2 = tge_check_launch("attention_prefill_tc2");
         if (rc2 != 0) return rc2;
         if (num_splits > 1 && !p.leave_states) {
-          dim3 mgrid(tokens - first_token, heads);
-          launch_merge(mgrid, stream, p.partial_o, p.partial_ml, positions, p.out, out_stride, tokens, heads, window, p.split_tokens, num_splits, first_token, p.sink);
+          launch_merge(p, positions, first_token, stream);
           return tge_launched("attention_merge", 2);
         }
         return 1;
@@ -1503,8 +1537,7 @@ static int attention_dispatch(const void* q, int q_stride, const void* k_pages, 
       int rc = tge_check_launch("attention_prefill_tc");
       if (rc != 0) return rc;
       if (num_splits > 1 && !p.leave_states) {
-        dim3 mgrid(tokens - first_token, heads);
-        launch_merge(mgrid, stream, p.partial_o, p.partial_ml, positions, p.out, out_stride, tokens, heads, window, p.split_tokens, num_splits, first_token, p.sink);
+        launch_merge(p, positions, first_token, stream);
         return tge_launched("attention_merge", 2);
       }
       return 1;
@@ -1526,8 +1559,7 @@ static int attention_dispatch(const void* q, int q_stride, const void* k_pages, 
       int rc = tge_check_launch("attention_prefill_tma");
       if (rc != 0) return rc;
       if (num_splits > 1 && !p.leave_states) {
-        dim3 mgrid(tokens - first_token, heads);
-        launch_merge(mgrid, stream, p.partial_o, p.partial_ml, positions, p.out, out_stride, tokens, heads, window, p.split_tokens, num_splits, first_token, p.sink);
+        launch_merge(p, positions, first_token, stream);
         return tge_launched("attention_merge", 2);
       }
       return 1;
@@ -1546,8 +1578,7 @@ static int attention_dispatch(const void* q, int q_stride, const void* k_pages, 
   else rc = launch<4>(p, tiles, stream);
   if (rc != 0) return rc;
   if (num_splits > 1 && !p.leave_states) {
-    dim3 grid(tokens - first_token, heads);
-    launch_merge(grid, stream, p.partial_o, p.partial_ml, positions, p.out, out_stride, tokens, heads, window, p.split_tokens, num_splits, first_token, p.sink);
+    launch_merge(p, positions, first_token, stream);
     return tge_launched("attention_merge", 2);
   }
   return 1;
@@ -1563,13 +1594,17 @@ static int attention_dispatch(const void* q, int q_stride, const void* k_pages, 
 // route beyond rounding.
 // `dist_bias` (float32 [heads, dist_span], or null): a learned bias by distance, added unscaled to the scaled score of the
 // key n positions back, entry min(n, dist_span - 1) of the head's row; every kernel adds it where it scales its scores.
+// `keep_first` (with a window): the first so many positions stay visible beside the window.  `gate` (bfloat16 [tokens,
+// gate_stride], or null): logits of one gate per token and head; whoever writes a head's output multiplies it by their
+// logistic function.
 TGE_API int tge_attention_mma(const void* q, int q_stride, const void* k_pages, const void* v_pages,
                               const int* block_table, int max_pages, int num_pages, int page_size,
                               const int* q_start, const int* start_pos, const int* positions, int num_seqs,
                               int tokens, int max_q_len, int max_ctx_len, void* out, int out_stride, int heads,
                               int kv_heads, float scale, int window, int split_tokens, float* scratch, int* status,
                               int decode_prefix, int prefix_split_tokens, const float* sink, int leave_states,
-                              int v_pitch, const float* dist_bias, int dist_span, cudaStream_t stream) {
+                              int v_pitch, const float* dist_bias, int dist_span, int keep_first, const void* gate,
+                              int gate_stride, cudaStream_t stream) {
   TGE_REQUIRE(decode_prefix >= 0 && decode_prefix <= num_seqs, "attention_mma: %d leading single tokens of %d sequences",
               decode_prefix, num_seqs);
   TGE_REQUIRE(prefix_split_tokens >= 0 && prefix_split_tokens % BKV == 0,
@@ -1577,16 +1612,16 @@ TGE_API int tge_attention_mma(const void* q, int q_stride, const void* k_pages, 
   if (decode_prefix == 0 || max_q_len <= 1 || decode_prefix == num_seqs || kv_heads <= 0 || heads / kv_heads > 16)
     return attention_dispatch(q, q_stride, k_pages, v_pages, block_table, max_pages, num_pages, page_size, q_start, start_pos,
                               positions, num_seqs, tokens, max_q_len, max_ctx_len, out, out_stride, heads, kv_heads, scale,
-                              window, split_tokens, scratch, status, 0, sink, leave_states, v_pitch, dist_bias, dist_span, stream);
+                              window, split_tokens, scratch, status, 0, sink, leave_states, v_pitch, dist_bias, dist_span, keep_first, gate, gate_stride, stream);
   const int first = attention_dispatch(q, q_stride, k_pages, v_pages, block_table, max_pages, num_pages, page_size, q_start,
                                        start_pos, positions, decode_prefix, decode_prefix, 1, max_ctx_len, out, out_stride,
                                        heads, kv_heads, scale, window, prefix_split_tokens, scratch, status, 0, sink, leave_states, v_pitch, dist_bias,
-                                       dist_span, stream);
+                                       dist_span, keep_first, gate, gate_stride, stream);
   if (first < 0) return first;
   const int rest = attention_dispatch(q, q_stride, k_pages, v_pages, block_table + (size_t)decode_prefix * max_pages, max_pages,
                                       num_pages, page_size, q_start + decode_prefix, start_pos + decode_prefix, positions,
                                       num_seqs - decode_prefix, tokens, max_q_len, max_ctx_len, out, out_stride, heads,
                                       kv_heads, scale, window, split_tokens, scratch, status, decode_prefix, sink, leave_states, v_pitch, dist_bias,
-                                      dist_span, stream);
+                                      dist_span, keep_first, gate, gate_stride, stream);
   return rest < 0 ? rest : first + rest;
 }

@@ -16,7 +16,9 @@
 // block of `pool` positions that lies wholly before its window (block b if b*pool + pool - 1 <= p - window); they
 // are read from pages of their own, entry b where position b would be, and visited before the tokens.
 // `dist_bias` [heads, span] (float32): a learned bias added to the scaled score of the key at distance n, entry
-// min(n, span - 1) of the head's row.
+// min(n, span - 1) of the head's row.  With a window and `keep_first` > 0 the first so many positions stay visible
+// beside the window.  `gate` [tokens, heads] (the run's format): logits of one gate per head; the output is multiplied by
+// their logistic function.
 #include "common.cuh"
 
 namespace {
@@ -30,7 +32,8 @@ __global__ void __launch_bounds__(128) attention_simt_kernel(
     const int* __restrict__ positions, const int* __restrict__ seq_of_token, T* __restrict__ out, int out_stride,
     int heads, int kv_heads, int head_dim, int value_dim, int v_pitch, const float* __restrict__ sink, float scale, int window,
     int pool, const T* __restrict__ kp_pages, const T* __restrict__ vp_pages, const int* __restrict__ pool_table,
-    int pool_max_pages, int pool_num_pages, const float* __restrict__ dist_bias, int dist_span, int* status) {
+    int pool_max_pages, int pool_num_pages, const float* __restrict__ dist_bias, int dist_span, int keep_first,
+    const T* __restrict__ gate, int gate_stride, int* status) {
   const int t = blockIdx.x;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int h = blockIdx.y * 4 + warp;
@@ -85,7 +88,14 @@ __global__ void __launch_bounds__(128) attention_simt_kernel(
       m = m_new;
     }
   }
-  for (int page_index = first / page_size; page_index * page_size <= pos; ++page_index) {
+  // the pages of the kept first tokens, then those of the window (a page that holds keys of both is walked once)
+  const int kept = min(keep_first, first);
+  const int kept_pages = (kept + page_size - 1) / page_size;
+  for (int page_index = kept > 0 ? 0 : first / page_size; page_index * page_size <= pos; ++page_index) {
+    if (page_index == kept_pages && kept > 0) {
+      page_index = max(page_index, first / page_size);
+      if (page_index * page_size > pos) break;
+    }
     const int page = page_index < max_pages ? table[page_index] : -1;
     if (page < 0 || page >= num_pages) {
       if (lane == 0) atomicOr(status, TGE_STATUS_BAD_PAGE);
@@ -95,7 +105,12 @@ __global__ void __launch_bounds__(128) attention_simt_kernel(
     const size_t vbase = ((size_t)page * kv_heads + kvh) * page_size * v_pitch;   // v_pitch: numbers between two values' starts
     const int lo = max(first - page_index * page_size, 0);
     const int hi = min(pos - page_index * page_size, page_size - 1);
-    for (int slot = lo; slot <= hi; ++slot) {
+    const int kept_here = kept - page_index * page_size;             // slots below this are kept first tokens
+    for (int slot = kept_here > 0 ? 0 : lo; slot <= hi; ++slot) {
+      if (slot < lo && slot >= kept_here) {
+        slot = lo;
+        if (slot > hi) break;
+      }
       const T* krow = k_pages + base + (size_t)slot * head_dim;
       const T* vrow = v_pages + vbase + (size_t)slot * v_pitch;
       float dot = 0.0f;
@@ -128,7 +143,8 @@ __global__ void __launch_bounds__(128) attention_simt_kernel(
 #pragma unroll
     for (int i = 0; i < MAX_PER_LANE; ++i) acc[i] *= corr;
   }
-  const float inv = l > 0.0f ? 1.0f / l : 0.0f;
+  float inv = l > 0.0f ? 1.0f / l : 0.0f;
+  if (gate != nullptr) inv *= 1.0f / (1.0f + expf(-to_float<T>(gate[(size_t)t * gate_stride + h])));
   T* orow = out + (size_t)t * out_stride + (size_t)h * value_dim;
 #pragma unroll
   for (int i = 0; i < MAX_PER_LANE; ++i) {
@@ -232,7 +248,8 @@ TGE_API int tge_attention_simt(const void* q, int q_stride, const void* k_pages,
                                int heads, int kv_heads, int head_dim, int value_dim, const float* sink, float scale,
                                int window, int is_bf16, int pool, const void* kp_pages, const void* vp_pages,
                                const int* pool_table, int pool_max_pages, int pool_num_pages, int v_pitch,
-                               const float* dist_bias, int dist_span, int* status, cudaStream_t stream) {
+                               const float* dist_bias, int dist_span, int keep_first, const void* gate, int gate_stride,
+                               int* status, cudaStream_t stream) {
   // v_pitch: numbers between the starts of two positions' values in `v_pages` (0: value_dim, values packed).  A cache
   // whose values are the leading part of its keys passes the keys' pages twice and the keys' size here.
   if (v_pitch == 0) v_pitch = value_dim;
@@ -245,7 +262,10 @@ TGE_API int tge_attention_simt(const void* q, int q_stride, const void* k_pages,
   TGE_REQUIRE(value_dim > 0 && value_dim <= 32 * MAX_PER_LANE, "attention: value_dim %d outside (0, %d]", value_dim,
               32 * MAX_PER_LANE);
   TGE_REQUIRE(page_size > 0 && max_pages > 0 && num_pages > 0, "attention: bad page geometry");
-  TGE_REQUIRE(window >= 0, "attention: negative window");
+  TGE_REQUIRE(window >= 0 && keep_first >= 0, "attention: a window of %d with %d kept positions", window, keep_first);
+  TGE_REQUIRE(pool == 0 || keep_first == 0, "attention: kept first tokens go without pooled blocks");
+  TGE_REQUIRE(gate == nullptr || gate_stride >= heads, "attention: gate rows of %d for %d heads", gate_stride, heads);
+  if (window == 0) keep_first = 0;
   TGE_REQUIRE(dist_bias == nullptr || dist_span > 0, "attention: a bias by distance needs its span");
   TGE_REQUIRE(pool >= 0 && (pool == 0 || (window > 0 && kp_pages != nullptr && vp_pages != nullptr && pool_table != nullptr &&
                                           pool_max_pages > 0 && pool_num_pages > 0)),
@@ -257,13 +277,13 @@ TGE_API int tge_attention_simt(const void* q, int q_stride, const void* k_pages,
         (const __nv_bfloat16*)q, q_stride, (const __nv_bfloat16*)k_pages, (const __nv_bfloat16*)v_pages, block_table,
         max_pages, num_pages, page_size, positions, seq_of_token, (__nv_bfloat16*)out, out_stride, heads, kv_heads,
         head_dim, value_dim, v_pitch, sink, scale, window, pool, (const __nv_bfloat16*)kp_pages, (const __nv_bfloat16*)vp_pages,
-        pool_table, pool_max_pages, pool_num_pages, dist_bias, dist_span, status);
+        pool_table, pool_max_pages, pool_num_pages, dist_bias, dist_span, keep_first, (const __nv_bfloat16*)gate, gate_stride, status);
   else
     attention_simt_kernel<float><<<grid, 128, 0, stream>>>(
         (const float*)q, q_stride, (const float*)k_pages, (const float*)v_pages, block_table, max_pages, num_pages,
         page_size, positions, seq_of_token, (float*)out, out_stride, heads, kv_heads, head_dim, value_dim, v_pitch, sink, scale,
         window, pool, (const float*)kp_pages, (const float*)vp_pages, pool_table, pool_max_pages, pool_num_pages, dist_bias,
-        dist_span, status);
+        dist_span, keep_first, (const float*)gate, gate_stride, status);
   return tge_launched("attention_simt", 1);
 }
 

@@ -88,18 +88,13 @@ __global__ void __launch_bounds__(THREADS, 1) attention_prefill_tc2_kernel(
   const int q_len = p.q_start[seq + 1] - q_begin;
   const int q_total = min(QTILES * p.bq, q_len - q_first);          // queries of both tiles together
   const int pos0 = p.start_pos[seq] + q_first;
-  int lo = p.window > 0 ? max(pos0 - p.window + 1, 0) : 0;
-  int hi = pos0 + q_total;
-  if (p.num_splits > 1) {
-    lo = max(lo, split * p.split_tokens);
-    hi = min(hi, (split + 1) * p.split_tokens);
-  }
-  if (lo >= hi) return;
+  const KeyTiles keys(p, pos0, q_total, split);
+  if (keys.num_tiles <= 0) return;
+  const int lo = keys.lo, hi = keys.hi;
 
-  const int k_first = lo / BKV * BKV;
-  const int num_tiles = (hi - k_first + BKV - 1) / BKV;
-  const int first_page = k_first >> p.page_shift;
-  const int last_page = (k_first + num_tiles * BKV - 1) >> p.page_shift;
+  const int num_tiles = keys.num_tiles;
+  const int first_page = keys.start(0) >> p.page_shift;
+  const int last_page = (keys.start(num_tiles - 1) + BKV - 1) >> p.page_shift;
   for (int i = first_page + tid; i <= last_page; i += THREADS) {
     int page = i < p.max_pages ? p.block_table[(size_t)seq * p.max_pages + i] : -1;
     if (page >= p.num_pages) page = -2;
@@ -169,7 +164,7 @@ __global__ void __launch_bounds__(THREADS, 1) attention_prefill_tc2_kernel(
       const int stage = tile % STAGES;
       if (tile >= STAGES) mbar_wait_bounded(empty_bar + 8 * stage, (uint32_t)(tile / STAGES - 1) & 1u, p.status);
       const uint32_t k_dst = stages + stage * TMA_STAGE_BYTES, v_dst = k_dst + TMA_TILE_BYTES;
-      const int tile_first = k_first + tile * BKV;
+      const int tile_first = keys.start(tile);
       int wanted = 0;
       for (int j = lane; j < pages_per_tile; j += 32) {
         const int page = local_table[(tile_first >> p.page_shift) + j - first_page];
@@ -252,10 +247,10 @@ __global__ void __launch_bounds__(THREADS, 1) attention_prefill_tc2_kernel(
     const float step_raw = tc::RESCALE_STEP / p.scale_log2;
     bool bad_page = false;
     for (int it = 0; it < num_tiles; ++it) {
-      const int k0 = k_first + it * BKV;
+      const int k0 = keys.start(it);
       mbar_wait_bounded(my_s_bar + 8 * (it & 1), (uint32_t)(it >> 1) & 1u, p.status);
       fence_after();
-      if (local_table[(max(k0, lo) >> p.page_shift) - first_page] < 0) bad_page = true;
+      if (local_table[(keys.probe(k0) >> p.page_shift) - first_page] < 0) bad_page = true;
       uint32_t s_bits[BKV];
       const uint32_t s_now = s_tmem(qt, it & 1);
       load32(s_now + lane_base, s_bits);
@@ -281,7 +276,7 @@ __global__ void __launch_bounds__(THREADS, 1) attention_prefill_tc2_kernel(
       }
       // a tile that every row of the warp sees whole needs no mask
       // (rows beyond the tile's queries hold zeros and are never stored: they need none either)
-      const bool whole = !row_valid || (k0 + BKV - 1 <= row_pos && k0 >= first_key && k0 >= lo && k0 + BKV <= hi);
+      const bool whole = !row_valid || (k0 + BKV - 1 <= row_pos && ((k0 >= first_key && k0 >= lo) || k0 + BKV <= keys.keep) && k0 + BKV <= hi);
       float mx = -INFINITY;
       if (__all_sync(0xffffffffu, whole)) {
 #pragma unroll
@@ -290,7 +285,7 @@ __global__ void __launch_bounds__(THREADS, 1) attention_prefill_tc2_kernel(
 #pragma unroll
         for (int j = 0; j < BKV; ++j) {
           const int kpos = k0 + j;
-          const bool visible = row_valid && kpos <= row_pos && kpos >= first_key && kpos >= lo && kpos < hi;
+          const bool visible = row_valid && kpos <= row_pos && (kpos >= first_key || kpos < keys.keep) && keys.visible(kpos);
           const float sv = visible ? __uint_as_float(s_bits[j]) : -INFINITY;
           s_bits[j] = __float_as_uint(sv);
           mx = fmaxf(mx, sv);
@@ -351,7 +346,7 @@ __global__ void __launch_bounds__(THREADS, 1) attention_prefill_tc2_kernel(
     fence_after();
     // the running maximum is kept in the scores' own units here; the sink joins in scaled base-2 units
     const float l_all = p.num_splits == 1 ? with_sink(p, row_head, m_run == -INFINITY ? -INFINITY : m_run * p.scale_log2, l_run) : l_run;
-    const float inv = (p.num_splits == 1) ? (l_all > 0.0f ? 1.0f / l_all : 0.0f) : 1.0f;
+    const float inv = (p.num_splits == 1) ? (l_all > 0.0f ? 1.0f / l_all : 0.0f) * head_gate(p, row_token, row_head) : 1.0f;
     const size_t slot = ((size_t)split * p.total_tokens + row_token) * p.heads + row_head;
 #pragma unroll
     for (int c = 0; c < HD / 32; ++c) {

@@ -611,7 +611,68 @@ __global__ void __launch_bounds__(QKN_THREADS) qk_norm_kv_store_vec_kernel(
   }
 }
 
-// qkv: [tokens, >= heads*head_dim + kv_heads*(head_dim + value_dim)] rows of [q | k | v], row stride in elements.
+// The same for the norm over each head: `lanes` lanes (a power of two, one per 16 bytes of a head) share a head, which
+// stays in registers between its sum of squares and its scaling.
+__global__ void __launch_bounds__(QKN_THREADS) qk_head_norm_kv_store_vec_kernel(
+    __nv_bfloat16* __restrict__ qkv, int row_stride, const float* __restrict__ q_weight, const float* __restrict__ k_weight,
+    float eps, const int* __restrict__ positions, const int* __restrict__ seq_of_token, const int* __restrict__ block_table,
+    int max_pages, __nv_bfloat16* __restrict__ k_pages, __nv_bfloat16* __restrict__ v_pages, int num_pages, int page_size,
+    int heads, int kv_heads, int head_dim, int value_dim, int store_kv, int lanes, int* status) {
+  pdl_trigger();
+  const int t = blockIdx.x;
+  const int pos = positions[t];
+  bool store = store_kv != 0;
+  size_t k_base = 0, v_base = 0;
+  if (store) {
+    const int page_index = pos / page_size;
+    const int page = (pos >= 0 && page_index < max_pages) ? block_table[(size_t)seq_of_token[t] * max_pages + page_index] : -1;
+    if (page < 0 || page >= num_pages) {
+      if (threadIdx.x == 0) atomicOr(status, TGE_STATUS_BAD_PAGE);
+      store = false;
+    } else {
+      k_base = ((size_t)page * kv_heads * page_size + (pos % page_size)) * head_dim;
+      v_base = ((size_t)page * kv_heads * page_size + (pos % page_size)) * value_dim;
+    }
+  }
+  pdl_wait();
+  uint4* row = reinterpret_cast<uint4*>(qkv + (size_t)t * row_stride);
+  const int per_head = head_dim / 8, total = heads + kv_heads;
+  const int mine = threadIdx.x & (lanes - 1), groups = QKN_THREADS / lanes;
+  for (int base = 0; base < total; base += groups) {
+    const int unit = base + (int)threadIdx.x / lanes;
+    const bool valid = unit < total && mine < per_head;
+    const uint4 raw = valid ? row[unit * per_head + mine] : make_uint4(0u, 0u, 0u, 0u);
+    float f[8];
+    unpack8(raw, f);
+    float sum = 0.0f;
+#pragma unroll
+    for (int e = 0; e < 8; ++e) sum = fmaf(f[e], f[e], sum);
+    for (int step = lanes >> 1; step > 0; step >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, step);
+    if (!valid) continue;                                  // the shuffles above were the last ones of this round
+    const bool is_q = unit < heads;
+    const float* weight = is_q ? q_weight : k_weight;
+    uint4 done = raw;
+    if (weight != nullptr) {
+      const float factor = 1.0f / sqrtf(sum / (float)head_dim + eps);
+      const float4 w0 = *reinterpret_cast<const float4*>(weight + mine * 8), w1 = *reinterpret_cast<const float4*>(weight + mine * 8 + 4);
+      f[0] *= factor * w0.x; f[1] *= factor * w0.y; f[2] *= factor * w0.z; f[3] *= factor * w0.w;
+      f[4] *= factor * w1.x; f[5] *= factor * w1.y; f[6] *= factor * w1.z; f[7] *= factor * w1.w;
+      done = pack8(f);
+      row[unit * per_head + mine] = done;
+    }
+    if (!is_q && store)
+      *reinterpret_cast<uint4*>(k_pages + k_base + (size_t)(unit - heads) * page_size * head_dim + mine * 8) = done;
+  }
+  if (!store) return;
+  const uint4* v_row = row + total * per_head;
+  for (int u = threadIdx.x; u < kv_heads * value_dim / 8; u += QKN_THREADS) {
+    const int h = u * 8 / value_dim, d = u * 8 - h * value_dim;
+    *reinterpret_cast<uint4*>(v_pages + v_base + (size_t)h * page_size * value_dim + d) = v_row[u];
+  }
+}
+
+// qkv: [tokens, >= heads*head_dim + kv_heads*(head_dim + value_dim)] rows of [q | k | v], row stride in elements; no kv
+// heads: rows of q alone (a layer that reads another layer's cache), nothing is stored.
 // q_weight / k_weight: float32, heads*head_dim and kv_heads*head_dim long (or head_dim each with per_head), or null.
 // v_other: null, or the other layer's values [tokens, kv_heads*value_dim] with its row stride; blend: device float.
 TGE_API int tge_qk_norm_kv_store(void* qkv, int is_bf16, int row_stride, const float* q_weight, const float* k_weight,
@@ -620,7 +681,8 @@ TGE_API int tge_qk_norm_kv_store(void* qkv, int is_bf16, int row_stride, const f
                                  void* k_pages, void* v_pages, int num_pages, int page_size, int tokens, int heads,
                                  int kv_heads, int head_dim, int value_dim, int store_kv, int* status,
                                  cudaStream_t stream) {
-  TGE_REQUIRE(tokens >= 0 && heads > 0 && kv_heads > 0 && head_dim > 0 && value_dim > 0, "qk_norm_kv_store: bad sizes");
+  TGE_REQUIRE(tokens >= 0 && heads > 0 && kv_heads >= 0 && head_dim > 0 && value_dim > 0, "qk_norm_kv_store: bad sizes");
+  TGE_REQUIRE(kv_heads > 0 || !store_kv, "qk_norm_kv_store: without kv heads there is nothing to store");
   TGE_REQUIRE(row_stride >= heads * head_dim + kv_heads * (head_dim + value_dim), "qk_norm_kv_store: rows of %d elements "
               "do not hold q, k and v", row_stride);
   TGE_REQUIRE(eps > 0.0f || (q_weight == nullptr && k_weight == nullptr), "qk_norm_kv_store: eps must be positive");
@@ -645,6 +707,15 @@ TGE_API int tge_qk_norm_kv_store(void* qkv, int is_bf16, int row_stride, const f
     else if (per_thread <= 8) launch(qk_norm_kv_store_vec_kernel<8>);
     else launch(qk_norm_kv_store_vec_kernel<QKN_UNITS>);
     return tge_launched("qk_norm_kv_store_vec", 1);
+  }
+  if (is_bf16 && per_head && v_other == nullptr && aligned16 && head_dim % 8 == 0 && head_dim <= 256 && value_dim % 8 == 0 &&
+      row_stride % 8 == 0) {
+    int lanes = 1;
+    while (lanes * 8 < head_dim) lanes *= 2;
+    tge_launch(qk_head_norm_kv_store_vec_kernel, tokens, QKN_THREADS, 0, stream, (__nv_bfloat16*)qkv, row_stride, q_weight,
+               k_weight, eps, positions, seq_of_token, block_table, max_pages, (__nv_bfloat16*)k_pages, (__nv_bfloat16*)v_pages,
+               num_pages, page_size, heads, kv_heads, head_dim, value_dim, store_kv, lanes, status);
+    return tge_launched("qk_head_norm_kv_store_vec", 1);
   }
   if (is_bf16)
     tge_launch(qk_norm_kv_store_kernel<__nv_bfloat16>, tokens, 256, 0, stream, (__nv_bfloat16*)qkv, row_stride, q_weight,

@@ -1,7 +1,8 @@
 // Kernels of a routed feed-forward (a mixture of small experts) and of activations that stand alone.
 //
-//  * router_topk      - from float32 router logits: softmax over all outputs, the choice by score + correction inside
-//                       the best groups of neighbouring outputs, the chosen outputs' plain scores over their sum.
+//  * router_topk      - from float32 router logits: softmax over all outputs or each output's logistic function, the
+//                       choice by score + correction inside the best groups of neighbouring outputs, the chosen
+//                       outputs' plain scores, over their sum or as they are.
 //  * activation       - relu(z)^2, or the two-parameter form z > 0: softplus(p) z^2 + z/2, else
 //                       (1/2 + softplus(q)) (exp(z) - 1 - z) + z/2, in place on rows of the run dtype.
 //  * expert_up / expert_down_add - few tokens (a decode step): every (token, chosen expert) pair reads its expert's
@@ -13,6 +14,9 @@
 //  * expert_sort / expert_gather / expert_combine_add - many tokens: the pairs are grouped by expert so that each
 //                       expert's rows form one block of a buffer, which ordinary products then multiply; the last
 //                       kernel adds the weighted rows back into the stream, again in the order of the choice.
+//
+// An expert is relu(up h)^2 or a clamped gated one, min(g, L) sigmoid(alpha min(g, L)) (clamp(u, -L, L) + offset) with
+// the gate and up rows interleaved in its first matrix; a choice's weight multiplies the expert's output or its input.
 //
 // The router, the weights, every accumulation and the sum into the stream are float32.
 #include <limits.h>
@@ -43,7 +47,8 @@ __device__ __forceinline__ void warp_argmax(const float* values, int n, int lane
 // kept flags).
 __global__ void __launch_bounds__(128) router_topk_kernel(const float* __restrict__ logits, long long ld,
                                                           const float* __restrict__ correction, int tokens, int outputs,
-                                                          int top, int group_count, int group_keep, int* __restrict__ ids,
+                                                          int top, int group_count, int group_keep, int logistic,
+                                                          int over_sum, int* __restrict__ ids,
                                                           float* __restrict__ weights) {
   extern __shared__ float router_smem[];
   pdl_trigger();
@@ -56,21 +61,30 @@ __global__ void __launch_bounds__(128) router_topk_kernel(const float* __restric
   float* group_best = choice + outputs;
   float* kept = group_best + outputs;
   const float* z = logits + (size_t)t * ld;
-  float m = -INFINITY;
-  for (int i = lane; i < outputs; i += 32) m = fmaxf(m, z[i]);
-  m = warp_max(m);
-  float sum = 0.0f;
-  for (int i = lane; i < outputs; i += 32) {
-    const float e = expf(z[i] - m);
-    score[i] = e;
-    sum += e;
-  }
-  sum = warp_sum(sum);
-  const float inv = 1.0f / sum;
-  for (int i = lane; i < outputs; i += 32) {
-    const float s = score[i] * inv;
-    score[i] = s;
-    choice[i] = s + (correction != nullptr ? correction[i] : 0.0f);
+  if (logistic) {
+    for (int i = lane; i < outputs; i += 32) {
+      const float s = 1.0f / (1.0f + expf(-z[i]));
+      score[i] = s;
+      // the logits order like the scores and do not saturate
+      choice[i] = correction != nullptr ? s + correction[i] : z[i];
+    }
+  } else {
+    float m = -INFINITY;
+    for (int i = lane; i < outputs; i += 32) m = fmaxf(m, z[i]);
+    m = warp_max(m);
+    float sum = 0.0f;
+    for (int i = lane; i < outputs; i += 32) {
+      const float e = expf(z[i] - m);
+      score[i] = e;
+      sum += e;
+    }
+    sum = warp_sum(sum);
+    const float inv = 1.0f / sum;
+    for (int i = lane; i < outputs; i += 32) {
+      const float s = score[i] * inv;
+      score[i] = s;
+      choice[i] = s + (correction != nullptr ? correction[i] : 0.0f);
+    }
   }
   __syncwarp();
   if (group_count > 1 && group_keep < group_count) {
@@ -106,7 +120,7 @@ __global__ void __launch_bounds__(128) router_topk_kernel(const float* __restric
     chosen_sum += score[where];
     __syncwarp();
   }
-  chosen_sum += 1e-20f;
+  chosen_sum = over_sum ? chosen_sum + 1e-20f : 1.0f;
   if (lane == 0)
     for (int n = 0; n < top; ++n) weights[(size_t)t * top + n] = score[ids[(size_t)t * top + n]] / chosen_sum;
 }
@@ -203,11 +217,25 @@ __device__ __forceinline__ float warp_dot<__nv_bfloat16>(const __nv_bfloat16* __
   return warp_sum(acc);
 }
 
-// inner[pair, j] = relu(w_up[expert][j, :] . h[token, :])^2 for the pairs whose choice is an expert.
+// What an expert applies between its matrices: relu(z)^2, or the clamped gate on interleaved (g, u).
+struct ExpertAct {
+  int gated;
+  float limit, alpha, offset;
+};
+
+__device__ __forceinline__ float clamped_gate(const ExpertAct& act, float g, float u) {
+  g = fminf(g, act.limit);
+  u = fminf(fmaxf(u, -act.limit), act.limit);
+  return g / (1.0f + expf(-act.alpha * g)) * (u + act.offset);
+}
+
+// inner[pair, j] = relu(z_j)^2 or the gate on (z_2j, z_2j+1), z = w_up[expert] h[token] (times the pair's weight, if the
+// weight is the input's), for the pairs whose choice is an expert.
 template <typename T>
 __global__ void __launch_bounds__(256) expert_up_kernel(const T* __restrict__ h, long long ld_h, const T* __restrict__ w_up,
-                                                        const int* __restrict__ ids, T* __restrict__ inner, int top,
-                                                        int experts, int width, int ff) {
+                                                        const int* __restrict__ ids, const float* __restrict__ in_weights,
+                                                        T* __restrict__ inner, int top, int experts, int width, int ff,
+                                                        ExpertAct act) {
   pdl_trigger();
   pdl_wait();
   const int pair = blockIdx.x;
@@ -215,18 +243,25 @@ __global__ void __launch_bounds__(256) expert_up_kernel(const T* __restrict__ h,
   if (expert < 0 || expert >= experts) return;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const T* row = h + (size_t)(pair / top) * ld_h;
-  const T* w = w_up + (size_t)expert * ff * width;
+  const float scale = in_weights != nullptr ? in_weights[pair] : 1.0f;
+  const T* w = w_up + (size_t)expert * (act.gated ? 2 : 1) * ff * width;
   for (int j = blockIdx.y * 8 + warp; j < ff; j += gridDim.y * 8) {
+    if (act.gated) {
+      const float g = warp_dot<T>(row, w + (size_t)2 * j * width, width, lane) * scale;
+      const float u = warp_dot<T>(row, w + ((size_t)2 * j + 1) * width, width, lane) * scale;
+      if (lane == 0) inner[(size_t)pair * ff + j] = from_float<T>(clamped_gate(act, g, u));
+      continue;
+    }
     const float dot = warp_dot<T>(row, w + (size_t)j * width, width, lane);
     if (lane == 0) {
-      const float p = fmaxf(dot, 0.0f);
+      const float p = fmaxf(dot * scale, 0.0f);
       inner[(size_t)pair * ff + j] = from_float<T>(p * p);
     }
   }
 }
 
 // x[token, n] += sum over the token's choices, in their order, of weight * (w_down[expert][n, :] . inner[pair, :]), or
-// weight * h[token, n] for an identity expert.
+// weight * h[token, n] for an identity expert; null weights count as one.
 template <typename T>
 __global__ void __launch_bounds__(256) expert_down_add_kernel(const T* __restrict__ inner, const T* __restrict__ w_down,
                                                               const T* __restrict__ h, long long ld_h,
@@ -242,7 +277,7 @@ __global__ void __launch_bounds__(256) expert_down_add_kernel(const T* __restric
     for (int k = 0; k < top; ++k) {
       const int pair = t * top + k;
       const int expert = ids[pair];
-      const float weight = weights[pair];
+      const float weight = weights != nullptr ? weights[pair] : 1.0f;
       if (expert >= 0 && expert < experts)
         acc = fmaf(weight, warp_dot<T>(inner + (size_t)pair * ff, w_down + (size_t)expert * down_expert + (size_t)n * down_row, ff, lane), acc);
       else
@@ -286,14 +321,33 @@ __global__ void __launch_bounds__(1024) expert_sort_kernel(const int* __restrict
 
 template <typename T>
 __global__ void __launch_bounds__(256) expert_gather_kernel(const T* __restrict__ h, long long ld_h, const int* __restrict__ place,
-                                                            T* __restrict__ grouped, int top, int width) {
+                                                            const float* __restrict__ in_weights, T* __restrict__ grouped,
+                                                            int top, int width) {
   pdl_trigger();
   pdl_wait();
   const int pair = blockIdx.x;
   const int row = place[pair];
   if (row < 0) return;
   const T* src = h + (size_t)(pair / top) * ld_h;
-  for (int i = threadIdx.x; i < width; i += blockDim.x) grouped[(size_t)row * width + i] = src[i];
+  T* dst = grouped + (size_t)row * width;
+  const float scale = in_weights != nullptr ? in_weights[pair] : 1.0f;
+  if (sizeof(T) == 2 && width % 8 == 0 && ld_h % 8 == 0 && ((uintptr_t)h & 15) == 0 && ((uintptr_t)grouped & 15) == 0) {
+    for (int i = threadIdx.x; i < width / 8; i += blockDim.x) {
+      uint4 raw = reinterpret_cast<const uint4*>(src)[i];
+      if (in_weights != nullptr) {
+        __nv_bfloat162* two = reinterpret_cast<__nv_bfloat162*>(&raw);
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          const float2 f = __bfloat1622float2(two[e]);
+          two[e] = __floats2bfloat162_rn(f.x * scale, f.y * scale);
+        }
+      }
+      reinterpret_cast<uint4*>(dst)[i] = raw;
+    }
+    return;
+  }
+  for (int i = threadIdx.x; i < width; i += blockDim.x)
+    dst[i] = in_weights != nullptr ? from_float<T>(to_float<T>(src[i]) * scale) : src[i];
 }
 
 template <typename T>
@@ -309,7 +363,7 @@ __global__ void __launch_bounds__(256) expert_combine_add_kernel(const float* __
       const int pair = t * top + k;
       const int row = place[pair];
       const float v = row >= 0 ? outputs[(size_t)row * width + n] : to_float<T>(h[(size_t)t * ld_h + n]);
-      acc = fmaf(weights[pair], v, acc);
+      acc = fmaf(weights != nullptr ? weights[pair] : 1.0f, v, acc);
     }
     x[(size_t)t * width + n] += acc;
   }
@@ -353,11 +407,53 @@ __global__ void __launch_bounds__(256) expert_dense_weigh_kernel(T* __restrict__
   }
 }
 
+// The dense path of gated experts: z [tokens, experts * 2 ff] (interleaved gate and up of every expert) -> out [tokens,
+// experts * ff], a chosen expert's activated values and zeros elsewhere.  `weigh_input`: the weight multiplies (g, u), else
+// the activated value.
+template <typename T>
+__global__ void __launch_bounds__(256) expert_dense_gate_kernel(const T* __restrict__ z, const int* __restrict__ ids,
+                                                                const float* __restrict__ weights, T* __restrict__ out, int top,
+                                                                int experts, int ff, int weigh_input, ExpertAct act) {
+  pdl_trigger();
+  pdl_wait();
+  const int t = blockIdx.x, e = blockIdx.y;
+  float w = 0.0f;
+  bool chosen = false;
+  for (int k = 0; k < top; ++k)
+    if (ids[t * top + k] == e) { w = weights[t * top + k]; chosen = true; }
+  const T* src = z + ((size_t)t * experts + e) * 2 * ff;
+  T* dst = out + ((size_t)t * experts + e) * ff;
+  const float in = weigh_input ? w : 1.0f, after = weigh_input ? 1.0f : w;
+  if (sizeof(T) == 2 && ff % 4 == 0) {
+    // four values at a time: 16 bytes in, 8 bytes out (the buffers are the wrapper's own, so aligned)
+    for (int j = threadIdx.x; j < ff / 4; j += blockDim.x) {
+      uint2 packed = make_uint2(0u, 0u);
+      if (chosen) {
+        const uint4 raw = reinterpret_cast<const uint4*>(src)[j];
+        const __nv_bfloat162* two = reinterpret_cast<const __nv_bfloat162*>(&raw);
+        float y[4];
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+          const float2 gu = __bfloat1622float2(two[i]);
+          y[i] = after * clamped_gate(act, gu.x * in, gu.y * in);
+        }
+        *reinterpret_cast<__nv_bfloat162*>(&packed.x) = __floats2bfloat162_rn(y[0], y[1]);
+        *reinterpret_cast<__nv_bfloat162*>(&packed.y) = __floats2bfloat162_rn(y[2], y[3]);
+      }
+      reinterpret_cast<uint2*>(dst)[j] = packed;
+    }
+    return;
+  }
+  for (int j = threadIdx.x; j < ff; j += blockDim.x)
+    dst[j] = from_float<T>(chosen ? after * clamped_gate(act, to_float<T>(src[2 * j]) * in, to_float<T>(src[2 * j + 1]) * in) : 0.0f);
+}
+
 }  // namespace
 
 // logits float32 [tokens, ld]; correction float32 [outputs] or null; ids int32 [tokens, top]; weights float32 [tokens, top].
 TGE_API int tge_router_topk(const float* logits, long long ld, const float* correction, int tokens, int outputs, int top,
-                            int group_count, int group_keep, int* ids, float* weights, cudaStream_t stream) {
+                            int group_count, int group_keep, int logistic, int over_sum, int* ids, float* weights,
+                            cudaStream_t stream) {
   TGE_REQUIRE(tokens >= 0 && outputs > 0 && outputs <= 1024, "router_topk: 1 to 1024 outputs, not %d", outputs);
   TGE_REQUIRE(top > 0 && top <= outputs, "router_topk: %d choices of %d outputs", top, outputs);
   TGE_REQUIRE(group_count > 0 && outputs % group_count == 0 && group_keep > 0 && group_keep <= group_count,
@@ -373,7 +469,7 @@ TGE_API int tge_router_topk(const float* logits, long long ld, const float* corr
     }
   }
   tge_launch(router_topk_kernel, dim3((tokens + 3) / 4), dim3(128), smem, stream, logits, ld, correction, tokens, outputs, top,
-             group_count, group_keep, ids, weights);
+             group_count, group_keep, logistic, over_sum, ids, weights);
   return tge_launched("router_topk", 1);
 }
 
@@ -399,23 +495,29 @@ TGE_API int tge_activation(void* rows, long long ld, int count, int width, int k
 
 // The direct path.  h: run dtype [tokens, >= width] with row stride ld_h; w_up [experts, ff, width]; row n of expert
 // e's down matrix (ff numbers) starts at w_down + e * down_expert + n * down_row; inner: run dtype scratch
-// [tokens * top, ff]; x: the float32 stream [tokens, width].
+// [tokens * top, ff]; x: the float32 stream [tokens, width].  With `gated` w_up is [experts, 2 ff, width], gate and up rows
+// interleaved.
 TGE_API int tge_experts_direct(const void* h, long long ld_h, const void* w_up, const void* w_down, long long down_expert,
                                long long down_row, const int* ids, const float* weights, void* inner, float* x, int tokens,
-                               int top, int experts, int width, int ff, int is_bf16, cudaStream_t stream) {
+                               int top, int experts, int width, int ff, int weigh_input, int gated, float limit,
+                               float alpha, float offset, int is_bf16, cudaStream_t stream) {
   TGE_REQUIRE(tokens >= 0 && top > 0 && experts >= 0 && width > 0 && ff > 0, "experts: bad shape");
+  TGE_REQUIRE(!gated || limit > 0.0f, "experts: the gate's limit must be positive");
   if (tokens == 0) return 0;
+  const ExpertAct act{gated, limit, alpha, offset};
+  const float* in_weights = weigh_input ? weights : nullptr;
+  if (weigh_input) weights = nullptr;
   const int up_y = (ff + 7) / 8 < 64 ? (ff + 7) / 8 : 64;
   const int down_y = (width + 7) / 8 < 64 ? (width + 7) / 8 : 64;
   if (is_bf16) {
     tge_launch(expert_up_kernel<__nv_bfloat16>, dim3(tokens * top, up_y), dim3(256), 0, stream, (const __nv_bfloat16*)h, ld_h,
-               (const __nv_bfloat16*)w_up, ids, (__nv_bfloat16*)inner, top, experts, width, ff);
+               (const __nv_bfloat16*)w_up, ids, in_weights, (__nv_bfloat16*)inner, top, experts, width, ff, act);
     tge_launch(expert_down_add_kernel<__nv_bfloat16>, dim3(tokens, down_y), dim3(256), 0, stream, (const __nv_bfloat16*)inner,
                (const __nv_bfloat16*)w_down, (const __nv_bfloat16*)h, ld_h, ids, weights, x, top, experts, width, ff, down_expert,
                down_row);
   } else {
     tge_launch(expert_up_kernel<float>, dim3(tokens * top, up_y), dim3(256), 0, stream, (const float*)h, ld_h,
-               (const float*)w_up, ids, (float*)inner, top, experts, width, ff);
+               (const float*)w_up, ids, in_weights, (float*)inner, top, experts, width, ff, act);
     tge_launch(expert_down_add_kernel<float>, dim3(tokens, down_y), dim3(256), 0, stream, (const float*)inner,
                (const float*)w_down, (const float*)h, ld_h, ids, weights, x, top, experts, width, ff, down_expert, down_row);
   }
@@ -423,19 +525,19 @@ TGE_API int tge_experts_direct(const void* h, long long ld_h, const void* w_up, 
 }
 
 // The grouped path, first half: place int32 [tokens * top], offsets int32 [experts + 1], grouped run dtype
-// [tokens * top, width] (the rows of expert e at offsets[e] .. offsets[e + 1]).
-TGE_API int tge_experts_group(const void* h, long long ld_h, const int* ids, int* place, int* offsets, void* grouped,
-                              int tokens, int top, int experts, int width, int is_bf16, cudaStream_t stream) {
+// [tokens * top, width] (the rows of expert e at offsets[e] .. offsets[e + 1]), times the pairs' weights if given.
+TGE_API int tge_experts_group(const void* h, long long ld_h, const int* ids, const float* in_weights, int* place, int* offsets,
+                              void* grouped, int tokens, int top, int experts, int width, int is_bf16, cudaStream_t stream) {
   TGE_REQUIRE(tokens >= 0 && top > 0 && experts > 0 && experts <= 4096 && width > 0, "experts: bad shape");
   if (tokens == 0) return 0;
   tge_launch(expert_sort_kernel, dim3(1), dim3(1024), (size_t)2 * experts * sizeof(int), stream, ids, tokens * top, experts,
              place, offsets);
   if (is_bf16)
     tge_launch(expert_gather_kernel<__nv_bfloat16>, dim3(tokens * top), dim3(256), 0, stream, (const __nv_bfloat16*)h, ld_h,
-               (const int*)place, (__nv_bfloat16*)grouped, top, width);
+               (const int*)place, in_weights, (__nv_bfloat16*)grouped, top, width);
   else
     tge_launch(expert_gather_kernel<float>, dim3(tokens * top), dim3(256), 0, stream, (const float*)h, ld_h, (const int*)place,
-               (float*)grouped, top, width);
+               in_weights, (float*)grouped, top, width);
   return tge_launched("experts_group", 2);
 }
 
@@ -466,4 +568,21 @@ TGE_API int tge_experts_dense_weigh(void* z, const int* ids, const float* weight
     tge_launch(expert_dense_weigh_kernel<float>, dim3(tokens, experts + 1), dim3(256), 0, stream, (float*)z, ids, weights,
                (const float*)h, ld_h, x, top, experts, width, ff);
   return tge_launched("experts_dense_weigh", 1);
+}
+
+// The dense path of gated experts: z run dtype [tokens, experts * 2 ff] -> out [tokens, experts * ff] (see the kernel).
+TGE_API int tge_experts_dense_gate(const void* z, const int* ids, const float* weights, void* out, int tokens, int top,
+                                   int experts, int ff, int weigh_input, float limit, float alpha, float offset, int is_bf16,
+                                   cudaStream_t stream) {
+  TGE_REQUIRE(tokens >= 0 && top > 0 && experts > 0 && experts < 65535 && ff > 0 && limit > 0.0f, "experts: bad shape");
+  TGE_REQUIRE(((uintptr_t)z & 15) == 0 && ((uintptr_t)out & 15) == 0, "experts: rows must start on 16 bytes");
+  if (tokens == 0) return 0;
+  const ExpertAct act{1, limit, alpha, offset};
+  if (is_bf16)
+    tge_launch(expert_dense_gate_kernel<__nv_bfloat16>, dim3(tokens, experts), dim3(256), 0, stream, (const __nv_bfloat16*)z, ids,
+               weights, (__nv_bfloat16*)out, top, experts, ff, weigh_input, act);
+  else
+    tge_launch(expert_dense_gate_kernel<float>, dim3(tokens, experts), dim3(256), 0, stream, (const float*)z, ids, weights,
+               (float*)out, top, experts, ff, weigh_input, act);
+  return tge_launched("experts_dense_gate", 1);
 }

@@ -97,6 +97,7 @@ struct TgeRtCache {
   struct Group {
     int window;                                              // < 0: none
     int stride = 1;                                          // positions per entry: a group of pooled entries keeps one per block
+    int keep_first = 0;                                      // with a window: the first positions that stay readable beside it
     std::unique_ptr<TgeRtPool> pool;
     std::unordered_map<int64_t, std::vector<int>> tables;    // request -> logical page -> physical id
   };
@@ -172,7 +173,9 @@ struct TgeRtCache {
       if (it == group.tables.end()) continue;
       std::vector<int>& table = it->second;
       const int end = std::min(first_needed_page(group, computed_tokens), (int)table.size());
-      for (int index = 0; index < end; ++index) {
+      // a page that holds any of the kept first positions stays
+      const int kept = (group.keep_first / group.stride + page_size - 1) / page_size;
+      for (int index = kept; index < end; ++index) {
         if (table[index] != NO_PAGE) {
           group.pool->release(table[index]);
           table[index] = NO_PAGE;
@@ -554,10 +557,15 @@ TgeRtCache* tge_rt_cache_create(int page_size, int max_requests) {
 void tge_rt_cache_destroy(TgeRtCache* cache) { delete cache; }
 int tge_rt_cache_add_group(TgeRtCache* cache, int window) { return tge_rt_cache_add_group_strided(cache, window, 1); }
 int tge_rt_cache_add_group_strided(TgeRtCache* cache, int window, int stride) {
+  return tge_rt_cache_add_group_kept(cache, window, stride, 0);
+}
+int tge_rt_cache_add_group_kept(TgeRtCache* cache, int window, int stride, int keep_first) {
   if (cache->groups.size() >= TGE_RT_MAX_GROUPS) return fail(TGE_RT_VALUE_ERROR, "cache manager: at most %d groups", TGE_RT_MAX_GROUPS);
   TgeRtCache::Group group;
   if (stride <= 0) return fail(TGE_RT_VALUE_ERROR, "cache manager: a group keeps one entry per %d positions", stride);
+  if (keep_first < 0) return fail(TGE_RT_VALUE_ERROR, "cache manager: %d kept positions", keep_first);
   group.window = window;
+  group.keep_first = keep_first;
   group.stride = stride;
   group.pool.reset(new TgeRtPool(1));
   cache->groups.push_back(std::move(group));

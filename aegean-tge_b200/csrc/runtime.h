@@ -42,6 +42,8 @@ void tge_rt_cache_destroy(TgeRtCache* cache);
 int tge_rt_cache_add_group(TgeRtCache* cache, int window);            // window < 0: every key is kept; returns the group's index
 // A group that keeps one entry per `stride` positions (the whole blocks among a request's tokens): pooled keys and values.
 int tge_rt_cache_add_group_strided(TgeRtCache* cache, int window, int stride);
+// With a window: the pages of the first `keep_first` positions are never given back while the request lives.
+int tge_rt_cache_add_group_kept(TgeRtCache* cache, int window, int stride, int keep_first);
 int tge_rt_cache_set_pool_size(TgeRtCache* cache, int group, int num_pages);
 TgeRtPool* tge_rt_cache_pool(TgeRtCache* cache, int group);          // owned by the cache
 int tge_rt_cache_groups(const TgeRtCache* cache);

@@ -114,8 +114,12 @@ class DecoderModel:
     def declare_cache(self, manager: CacheManager) -> None:
         for index, (block, layer) in enumerate(zip(self.blocks, self.spec.layers)):
             if layer.cache_from is None:
-                manager.add_layer(index, block.mixer.cache_spec(), block.mixer.state_spec(),
-                                  block.mixer.extra_cache_specs())
+                spec = block.mixer.cache_spec()
+                for reader, other in zip(self.blocks, self.spec.layers):
+                    # a layer that reads this one's entries may look further back than this one does
+                    if other.cache_from == index and spec is not None and reader.mixer.cache_spec() is not None:
+                        spec = spec.covering(reader.mixer.cache_spec())
+                manager.add_layer(index, spec, block.mixer.state_spec(), block.mixer.extra_cache_specs())
             else:
                 manager.add_layer(index, None, block.mixer.state_spec())
 

@@ -93,7 +93,7 @@ def core() -> ctypes.CDLL:
         _declare(lib, "tge_attention_simt", [_c_ptr, _c_int, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_int, _c_int, _c_ptr,
                                              _c_ptr, _c_ptr, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_ptr,
                                              _c_float, _c_int, _c_int, _c_int, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_int,
-                                             _c_int, _c_ptr, _c_int, _c_ptr, _c_ptr])
+                                             _c_int, _c_ptr, _c_int, _c_int, _c_ptr, _c_int, _c_ptr, _c_ptr])
         _declare(lib, "tge_attention_pooled_merge", [_c_ptr, _c_int, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_int, _c_int, _c_ptr,
                                                      _c_ptr, _c_ptr, _c_ptr, _c_int, _c_int, _c_ptr, _c_int, _c_int, _c_int,
                                                      _c_int, _c_int, _c_int, _c_float, _c_int, _c_int, _c_ptr, _c_int, _c_ptr,
@@ -114,14 +114,20 @@ def core() -> ctypes.CDLL:
         _declare(lib, "tge_latent_scatter", [_c_ptr, _c_ll, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_ptr, _c_ptr,
                                              _c_int, _c_ptr])
         _declare(lib, "tge_gate_rows", [_c_ptr, _c_ll, _c_ptr, _c_ll, _c_int, _c_int, _c_int, _c_int, _c_int, _c_ptr])
-        _declare(lib, "tge_router_topk", [_c_ptr, _c_ll, _c_ptr, _c_int, _c_int, _c_int, _c_int, _c_int, _c_ptr, _c_ptr,
-                                          _c_ptr])
+        _declare(lib, "tge_router_topk", [_c_ptr, _c_ll, _c_ptr, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int,
+                                          _c_ptr, _c_ptr, _c_ptr])
         _declare(lib, "tge_activation", [_c_ptr, _c_ll, _c_int, _c_int, _c_int, _c_ptr, _c_int, _c_ptr])
         _declare(lib, "tge_experts_direct", [_c_ptr, _c_ll, _c_ptr, _c_ptr, _c_ll, _c_ll, _c_ptr, _c_ptr, _c_ptr, _c_ptr,
-                                             _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_ptr])
+                                             _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_float, _c_float,
+                                             _c_float, _c_int, _c_ptr])
         _declare(lib, "tge_experts_dense_weigh", [_c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_ll, _c_ptr, _c_int, _c_int, _c_int,
                                                   _c_int, _c_int, _c_int, _c_ptr])
-        _declare(lib, "tge_experts_group", [_c_ptr, _c_ll, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_int, _c_int, _c_int,
+        _declare(lib, "tge_experts_dense_gate", [_c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_int, _c_int, _c_int, _c_int,
+                                                 _c_float, _c_float, _c_float, _c_int, _c_ptr])
+        _declare(lib, "tge_mlstm_step", [_c_ptr, _c_int, _c_ll, _c_ptr, _c_ll, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_ptr,
+                                         _c_ptr, _c_ll, _c_int, _c_int, _c_int, _c_int, _c_int, _c_float, _c_float, _c_float,
+                                         _c_ptr])
+        _declare(lib, "tge_experts_group", [_c_ptr, _c_ll, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_int, _c_int, _c_int,
                                             _c_int, _c_ptr])
         _declare(lib, "tge_experts_combine_add", [_c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_ll, _c_ptr, _c_int, _c_int, _c_int,
                                                   _c_int, _c_ptr])
@@ -180,7 +186,7 @@ def attention_lib(head_dim: int, value_dim: int = 0) -> ctypes.CDLL:
         _declare(lib, "tge_attention_mma", [_c_ptr, _c_int, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_int, _c_int, _c_ptr,
                                             _c_ptr, _c_ptr, _c_int, _c_int, _c_int, _c_int, _c_ptr, _c_int, _c_int,
                                             _c_int, _c_float, _c_int, _c_int, _c_ptr, _c_ptr, _c_int, _c_int, _c_ptr,
-                                            _c_int, _c_int, _c_ptr, _c_int, _c_ptr])
+                                            _c_int, _c_int, _c_ptr, _c_int, _c_int, _c_ptr, _c_int, _c_ptr])
         lib.tge_attention_mma_scratch_floats.argtypes = [_c_int, _c_int, _c_int]
         lib.tge_attention_mma_scratch_floats.restype = _c_ll
         if lib.tge_attention_mma_head_dim() != head_dim or lib.tge_attention_mma_value_dim() != value_dim:
@@ -752,7 +758,8 @@ def attention(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tensor, blo
               force_simt: bool = False, typical_ctx_len: int = 0, decode_prefix: int = 0,
               sink: Optional[torch.Tensor] = None, pool: int = 0, pooled_k: Optional[torch.Tensor] = None,
               pooled_v: Optional[torch.Tensor] = None, pool_table: Optional[torch.Tensor] = None,
-              values_in_keys: int = 0, dist_bias: Optional[torch.Tensor] = None) -> torch.Tensor:
+              values_in_keys: int = 0, dist_bias: Optional[torch.Tensor] = None, keep_first: int = 0,
+              gate: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Paged causal attention of a flat batch of portions.
 
     q: [T, >= heads*head_dim] (dense rows, any row stride) holding rotated queries;
@@ -773,6 +780,9 @@ def attention(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tensor, blo
     ``dist_bias`` (float32 [heads, span]): a learned bias by distance, added unscaled to the scaled score of the key
     that lies n positions back, entry min(n, span - 1) of the head's row; every attention kernel adds it where it
     scales its scores.
+    ``keep_first`` (with a window): the first so many positions of a request stay visible beside the window.
+    ``gate`` (run dtype [T, heads], dense rows, any row stride): logits of one gate per head; whoever writes a head's
+    output multiplies it by their logistic function.
     """
     v_pitch = 0
     if values_in_keys:
@@ -824,6 +834,19 @@ def attention(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tensor, blo
             raise KernelError(f"attention: a bias by distance is [heads, span] (and goes without pooled blocks), got "
                               f"{tuple(dist_bias.shape)}")
         dist_span = dist_bias.shape[1]
+    keep_first = int(keep_first) if window > 0 else 0
+    if pool and (keep_first or gate is not None):
+        raise KernelError("attention: kept first tokens and gates go without pooled blocks")
+    gate_stride = 0
+    if gate is not None:
+        _want(gate, "head gates", q.dtype, contiguous=False)
+        gate_stride = _rows_2d(gate, "head gates")
+        if tuple(gate.shape) != (tokens, heads):
+            raise KernelError(f"attention: gates must be [{tokens}, {heads}], got {tuple(gate.shape)}")
+    # what a query's keys span, for the choice of runs: with a window, the window's tiles and the kept tokens'
+    span = max_ctx_len
+    if window > 0 and not pool:
+        span = min(max_ctx_len, (-(-window // 64) + 1 + -(-keep_first // 64)) * 64)
     use_mma = (q.dtype == torch.bfloat16 and USE_MMA_ATTENTION and not force_simt and pairs_ok
                and mma_attention_supports(head_dim, heads, kv_heads, page_size, value_dim)
                and not (v_pitch and value_dim == head_dim))
@@ -844,12 +867,11 @@ def attention(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tensor, blo
                 max_ctx_len = max(max_ctx_len, 128)
                 split_tokens = 64 * -(-max_ctx_len // 128)
         if split_tokens == 0:
-            split_tokens = choose_attention_split(tokens, num_seqs, max_q_len, typical_ctx_len or max_ctx_len,
-                                                  heads, kv_heads, bound=max_ctx_len)
+            split_tokens = choose_attention_split(tokens, num_seqs, max_q_len, min(typical_ctx_len or max_ctx_len, span),
+                                                  heads, kv_heads, bound=span)
             # the single tokens at the head of a mixed step are a decode batch of their own: a few of them deep in
             # long contexts want their keys cut although the portions beside them do not
-            prefix_split = choose_attention_split(prefix, prefix, 1, max_ctx_len, heads, kv_heads,
-                                                  bound=max_ctx_len) if prefix else 0
+            prefix_split = choose_attention_split(prefix, prefix, 1, span, heads, kv_heads, bound=span) if prefix else 0
         count = lambda split: 1 if split == 0 or max_ctx_len <= split else -(-max_ctx_len // split)
         splits = max(count(split_tokens), count(prefix_split) if prefix else 1)
         need = lib.tge_attention_mma_scratch_floats(tokens, heads, splits)
@@ -859,7 +881,8 @@ def attention(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tensor, blo
                                      start_pos.data_ptr(), positions.data_ptr(), num_seqs, tokens, max_q_len,
                                      max_ctx_len, out.data_ptr(), out_stride, heads, kv_heads, float(scale), window,
                                      split_tokens, _ptr(scratch), status_word().data_ptr(), prefix, prefix_split,
-                                     _ptr(sink), int(bool(pool)), v_pitch, _ptr(dist_bias), dist_span, _stream()), lib)
+                                     _ptr(sink), int(bool(pool)), v_pitch, _ptr(dist_bias), dist_span,
+                                     keep_first, _ptr(gate), gate_stride, _stream()), lib)
         if pool:
             core_lib = core()
             states = scratch.data_ptr()
@@ -877,7 +900,8 @@ def attention(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tensor, blo
                                   seq_of_token.data_ptr(), out.data_ptr(), out_stride, tokens, heads, kv_heads,
                                   head_dim, value_dim, _ptr(sink), float(scale), window, int(q.dtype == torch.bfloat16),
                                   int(pool), _ptr(pooled_k), _ptr(pooled_v), _ptr(pool_table), pool_width, pool_pages,
-                                  v_pitch, _ptr(dist_bias), dist_span, status_word().data_ptr(), _stream()), lib)
+                                  v_pitch, _ptr(dist_bias), dist_span, keep_first, _ptr(gate), gate_stride,
+                                  status_word().data_ptr(), _stream()), lib)
     return out
 
 
@@ -1419,11 +1443,12 @@ ACT_RELU_SQUARED, ACT_XIELU = 0, 1
 
 
 def router_topk(logits: torch.Tensor, correction: Optional[torch.Tensor], top: int, group_count: int = 1,
-                group_keep: int = 1):
+                group_keep: int = 1, logistic: bool = False, over_sum: bool = True):
     """(ids int32 [T, top], weights float32 [T, top]) from float32 router logits [T, outputs]: scores = softmax over
     all outputs; the ``top`` outputs with the largest score + correction are chosen (the lowest index among equals),
     only inside the ``group_keep`` of ``group_count`` groups of neighbouring outputs whose best such value is largest;
-    weights = the chosen outputs' scores over their sum (+ 1e-20)."""
+    weights = the chosen outputs' scores over their sum (+ 1e-20), or as they are without ``over_sum``.  ``logistic``: an
+    output's score is the logistic function of its own logit."""
     _want(logits, "router logits", torch.float32, contiguous=False)
     ld = _rows_2d(logits, "router logits")
     tokens, outputs = logits.shape
@@ -1435,7 +1460,7 @@ def router_topk(logits: torch.Tensor, correction: Optional[torch.Tensor], top: i
     weights = torch.empty((tokens, top), dtype=torch.float32, device=logits.device)
     lib = core()
     _check(lib.tge_router_topk(logits.data_ptr(), ld, _ptr(correction), tokens, outputs, int(top), int(group_count),
-                               int(group_keep), ids.data_ptr(), weights.data_ptr(), _stream()), lib)
+                               int(group_keep), int(logistic), int(over_sum), ids.data_ptr(), weights.data_ptr(), _stream()), lib)
     return ids, weights
 
 
@@ -1455,10 +1480,12 @@ def activation(rows: torch.Tensor, kind: int, params: Optional[torch.Tensor] = N
 
 
 def experts_direct(h: torch.Tensor, w_up: torch.Tensor, w_down: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor,
-                   x: torch.Tensor) -> None:
+                   x: torch.Tensor, gate=None, weigh_input: bool = False) -> None:
     """x[t] += sum_k weights[t, k] * (w_down[e] relu(w_up[e] h[t])^2 with e = ids[t, k], or h[t] itself when e is
     beyond the experts), every pair reading its expert's rows directly: for steps of few tokens.  w_up [experts, ff,
-    width], w_down [width, experts, ff] (the experts' down matrices side by side), x float32 [T, width]."""
+    width], w_down [width, experts, ff] (the experts' down matrices side by side), x float32 [T, width].
+    ``gate`` (limit, alpha, offset): clamped gated experts instead, w_up [experts, 2 ff, width] with gate and up rows
+    interleaved.  ``weigh_input``: the weight multiplies the expert's input, not its output."""
     _want(h, "expert input", _FLOAT, contiguous=False)
     _want(w_up, "expert up weights", h.dtype)
     _want(w_down, "expert down weights", h.dtype)
@@ -1466,7 +1493,7 @@ def experts_direct(h: torch.Tensor, w_up: torch.Tensor, w_down: torch.Tensor, id
     _want(weights, "expert weights", torch.float32)
     _want(x, "stream", torch.float32)
     tokens, width = x.shape
-    experts, ff = w_up.shape[0], w_up.shape[1]
+    experts, ff = w_up.shape[0], w_up.shape[1] // (1 if gate is None else 2)
     top = ids.shape[1]
     if w_up.shape[2] != width or tuple(w_down.shape) != (width, experts, ff) or h.shape[0] != tokens or h.shape[1] != width:
         raise KernelError("experts: shapes do not agree")
@@ -1474,7 +1501,27 @@ def experts_direct(h: torch.Tensor, w_up: torch.Tensor, w_down: torch.Tensor, id
     lib = core()
     _check(lib.tge_experts_direct(h.data_ptr(), _rows_2d(h, "expert input"), w_up.data_ptr(), w_down.data_ptr(), ff,
                                   experts * ff, ids.data_ptr(), weights.data_ptr(), inner.data_ptr(), x.data_ptr(), tokens, top,
-                                  experts, width, ff, int(h.dtype == torch.bfloat16), _stream()), lib)
+                                  experts, width, ff, int(weigh_input), int(gate is not None),
+                                  *(float(v) for v in (gate or (1.0, 1.0, 1.0))), int(h.dtype == torch.bfloat16), _stream()), lib)
+
+
+def experts_dense_gate(z: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor, experts: int, gate,
+                       weigh_input: bool) -> torch.Tensor:
+    """z [T, experts * 2 ff] (gate and up of every expert for every token, interleaved) -> [T, experts * ff]: for a token's
+    chosen experts min(g, L) sigmoid(alpha min(g, L)) (clamp(u, -L, L) + offset) with ``gate`` = (L, alpha, offset), the
+    weight multiplying (g, u) with ``weigh_input`` and the value without; zeros for the other experts."""
+    _want(z, "expert rows", _FLOAT)
+    _want(ids, "expert ids", torch.int32)
+    _want(weights, "expert weights", torch.float32)
+    tokens, columns = z.shape
+    if columns % (2 * experts) or ids.shape[0] != tokens or weights.shape != ids.shape:
+        raise KernelError("experts: shapes do not agree")
+    out = torch.empty((tokens, columns // 2), dtype=z.dtype, device=z.device)
+    lib = core()
+    _check(lib.tge_experts_dense_gate(z.data_ptr(), ids.data_ptr(), weights.data_ptr(), out.data_ptr(), tokens, ids.shape[1],
+                                      int(experts), columns // (2 * experts), int(weigh_input), *(float(v) for v in gate),
+                                      int(z.dtype == torch.bfloat16), _stream()), lib)
+    return out
 
 
 def experts_dense_weigh(z: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor, h: torch.Tensor, x: torch.Tensor,
@@ -1497,10 +1544,14 @@ def experts_dense_weigh(z: torch.Tensor, ids: torch.Tensor, weights: torch.Tenso
     return z
 
 
-def experts_group(h: torch.Tensor, ids: torch.Tensor, experts: int):
+def experts_group(h: torch.Tensor, ids: torch.Tensor, experts: int, in_weights: Optional[torch.Tensor] = None):
     """Groups the (token, choice) pairs by expert: (place int32 [T * top]: a pair's row among the grouped rows, -1 for
     choices beyond the experts; offsets int32 [experts + 1]; grouped [T * top, width]: copies of the pairs' input rows,
-    expert e's at offsets[e] .. offsets[e + 1])."""
+    expert e's at offsets[e] .. offsets[e + 1]), times ``in_weights`` [T, top] if given."""
+    if in_weights is not None:
+        _want(in_weights, "expert weights", torch.float32)
+        if in_weights.shape != ids.shape:
+            raise KernelError("experts: one weight per choice")
     _want(h, "expert input", _FLOAT, contiguous=False)
     _want(ids, "expert ids", torch.int32)
     tokens, width = h.shape
@@ -1509,23 +1560,26 @@ def experts_group(h: torch.Tensor, ids: torch.Tensor, experts: int):
     offsets = torch.empty(experts + 1, dtype=torch.int32, device=h.device)
     grouped = torch.empty((tokens * top, width), dtype=h.dtype, device=h.device)
     lib = core()
-    _check(lib.tge_experts_group(h.data_ptr(), _rows_2d(h, "expert input"), ids.data_ptr(), place.data_ptr(), offsets.data_ptr(),
+    _check(lib.tge_experts_group(h.data_ptr(), _rows_2d(h, "expert input"), ids.data_ptr(), _ptr(in_weights), place.data_ptr(),
+                                 offsets.data_ptr(),
                                  grouped.data_ptr(), tokens, top, int(experts), width, int(h.dtype == torch.bfloat16), _stream()), lib)
     return place, offsets, grouped
 
 
-def experts_combine_add(outputs: torch.Tensor, place: torch.Tensor, weights: torch.Tensor, h: torch.Tensor,
+def experts_combine_add(outputs: torch.Tensor, place: torch.Tensor, weights: Optional[torch.Tensor], h: torch.Tensor,
                         x: torch.Tensor) -> None:
-    """x[t] += sum_k weights[t, k] * (outputs[place[t, k]] or, where place is -1, h[t]); outputs float32 grouped rows."""
+    """x[t] += sum_k weights[t, k] * (outputs[place[t, k]] or, where place is -1, h[t]); outputs float32 grouped rows;
+    ``weights`` None: all one."""
     _want(outputs, "expert outputs", torch.float32)
     _want(place, "expert places", torch.int32)
-    _want(weights, "expert weights", torch.float32)
+    if weights is not None:
+        _want(weights, "expert weights", torch.float32)
     _want(h, "expert input", _FLOAT, contiguous=False)
     _want(x, "stream", torch.float32)
     tokens, width = x.shape
-    top = weights.shape[1]
+    top = place.numel() // max(tokens, 1)
     lib = core()
-    _check(lib.tge_experts_combine_add(outputs.data_ptr(), place.data_ptr(), weights.data_ptr(), h.data_ptr(),
+    _check(lib.tge_experts_combine_add(outputs.data_ptr(), place.data_ptr(), _ptr(weights), h.data_ptr(),
                                        _rows_2d(h, "expert input"), x.data_ptr(), tokens, top, width,
                                        int(h.dtype == torch.bfloat16), _stream()), lib)
 
@@ -1610,6 +1664,41 @@ def gated_rule_scan(qk: torch.Tensor, v: torch.Tensor, gates: torch.Tensor, stat
     _check(lib.tge_gated_rule_scan(qk.data_ptr(), v.data_ptr(), gates.data_ptr(), _ptr(skip), int(delta), heads, groups, dim,
                                    vdim, state.data_ptr(), slots.data_ptr(), q_start.data_ptr(), out.data_ptr(), num_seqs,
                                    tokens, _stream()), lib)
+    return out
+
+
+def mlstm_step(rows: torch.Tensor, gates: torch.Tensor, heads: int, dim: int, vdim: int, norm_weight: torch.Tensor,
+               state: torch.Tensor, normaliser: torch.Tensor, maximum: torch.Tensor, slots: torch.Tensor, q_start: torch.Tensor,
+               num_seqs: int, cap: float, q_scale: float, eps: float, longest: int = 2 ** 31 - 1,
+               out: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """The matrix memory of an mLSTM, token by token, with the readout's norm and gate.
+
+    ``rows`` [T, q | k | v | g] (run dtype, dense rows), ``gates`` float32 [T, zi | zf] (their biases in them); per head
+    i = cap tanh(zi / cap), f = logsigmoid(cap tanh(zf / cap)), m' = max(f + m, i), S <- exp(f + m - m') S + exp(i - m') k v^T,
+    n likewise with k alone, o = S^T (q_scale q) / (max(|n . q_scale q|, exp(-m')) + 1e-6); out = o over its root mean square
+    per head, times ``norm_weight``, times sigmoid(g).  ``state`` float32 [slots, heads, dim, vdim], ``normaliser``
+    [slots, heads, dim] and ``maximum`` [slots, heads] are read and written in rows ``slots``.  Portions of more than
+    ``longest`` tokens are left alone, their output rows too."""
+    _want(rows, "projections", _FLOAT, contiguous=False)
+    _want(gates, "gate logits", torch.float32, contiguous=False)
+    for name, t in (("norm weight", norm_weight), ("state", state), ("normaliser", normaliser), ("maximum", maximum)):
+        _want(t, name, torch.float32)
+    _want(slots, "slots", torch.int32)
+    _want(q_start, "q_start", torch.int32)
+    tokens = rows.shape[0]
+    if (rows.shape[1] < 2 * heads * (dim + vdim) or gates.shape[0] != tokens or gates.shape[1] < 2 * heads
+            or tuple(state.shape[1:]) != (heads, dim, vdim) or tuple(normaliser.shape[1:]) != (heads, dim)
+            or tuple(maximum.shape[1:]) != (heads,) or norm_weight.numel() != heads * vdim):
+        raise KernelError(f"mlstm_step: rows {tuple(rows.shape)}, gates {tuple(gates.shape)}, state {tuple(state.shape)}, "
+                          f"normaliser {tuple(normaliser.shape)}, maximum {tuple(maximum.shape)}")
+    if out is None:
+        out = torch.empty((tokens, heads * vdim), dtype=rows.dtype, device=rows.device)
+    _want(out, "readout", rows.dtype, contiguous=False)
+    lib = core()
+    _check(lib.tge_mlstm_step(rows.data_ptr(), int(rows.dtype == torch.bfloat16), _rows_2d(rows, "projections"), gates.data_ptr(),
+                              _rows_2d(gates, "gate logits"), norm_weight.data_ptr(), state.data_ptr(), normaliser.data_ptr(),
+                              maximum.data_ptr(), slots.data_ptr(), q_start.data_ptr(), out.data_ptr(), _rows_2d(out, "readout"),
+                              num_seqs, heads, dim, vdim, int(longest), float(cap), float(q_scale), float(eps), _stream()), lib)
     return out
 
 

@@ -41,6 +41,13 @@ to ``far``, where the last row is reached and kept.  Product of q and k with
 the biases, one kernel that stores the values, normalises, applies the
 temperature and stores the keys, then the attention with the bias expanded
 to one entry per distance.
+
+And five that go with values of their own and no rotation (the *separate* path): the bias by distance; an RMS norm of q
+and k per head without a weight (``qk_norm`` with ``"weight": False``); a window beside which the first ``keep_first``
+tokens of the request stay visible; one gate per head (``head_gate``), the logistic function of a projection of the same
+input, that multiplies the head's output where the attention writes it; and a layer that has no keys and values of its own
+(``own_kv: False``) because it reads an earlier layer's cache.  The gate's rows lie below q, k and v in the one input
+product; one kernel normalises and stores, and the attention adds the bias and applies the gate.
 """
 from __future__ import annotations
 
@@ -69,6 +76,9 @@ class GQAttention(Mixer):
     The keyed path: ``values`` (``"own"``, the default, or ``"keys"``: no ``v.weight`` / ``v.bias``), ``q_temp`` (None
     or ``{"coef": c, "every": n}``), ``distance_bias`` (None or ``{"far": D}``; weight ``rel`` float32 [rows, heads], the
     rows taken from the tensor).
+    The separate path: ``distance_bias`` with values of their own, ``qk_norm`` ``{"scope": "head", "eps": e, "weight": False}``
+    (no ``q_norm.weight`` / ``k_norm.weight``), ``keep_first`` (0, or with a window how many first tokens stay visible),
+    ``head_gate`` (bool; ``gate.weight`` [heads, hidden]), ``own_kv`` (default True; False: no ``k.weight`` / ``v.weight``).
     """
     graph_safe = True
     can_defer_norm = True
@@ -109,8 +119,14 @@ class GQAttention(Mixer):
         self.dist_far = None if dist is None else float(dist["far"])
         if self.q_temp is not None and self.q_temp[1] <= 0:
             raise ValueError("attention: q_temp.every must be positive")
-        if (self.q_temp is not None or self.dist_far is not None) and not self.values_are_keys:
-            raise ValueError("attention: a query temperature and a bias by distance are built for values that are the keys")
+        if self.q_temp is not None and not self.values_are_keys:
+            raise ValueError("attention: a query temperature is built for values that are the keys")
+        self.norm_weights = norm is None or bool(norm.get("weight", True))
+        self.keep_first = int(p.get("keep_first") or 0)
+        self.head_gate = bool(p.get("head_gate", False))
+        self.own_kv = bool(p.get("own_kv", True))
+        if self.keep_first < 0 or (self.keep_first and self.window is None):
+            raise ValueError("attention: kept first tokens go with a window")
         self.dist_table: Optional[torch.Tensor] = None
         self.taps = int(p.get("short_conv") or 0)
         self.pool = int(p.get("pool") or 0)
@@ -145,6 +161,22 @@ class GQAttention(Mixer):
                                  "size go with a per-head q/k norm or none, without biases on q, k, v or value mixing")
             if tables is None:
                 raise ValueError("attention: the general path rotates by tables, or not at all")
+        # the separate path: one kernel normalises and stores behind the product, the attention does the rest
+        self.separate = not self.values_are_keys and (self.dist_far is not None or not self.norm_weights or self.keep_first > 0
+                                                      or self.head_gate or not self.own_kv)
+        if self.separate:
+            if (self.general or self.rotates or self.value_mix is not None or self.qkv_bias
+                    or (self.qk_norm is not None and self.qk_norm[0] != "head")):
+                raise ValueError("attention: a bias by distance, kept first tokens, a gate per head or borrowed keys and values go "
+                                 "with no rotation, a per-head q/k norm or none, and neither convolution, pooled blocks, biases on "
+                                 "q, k, v nor value mixing")
+        elif self.keep_first or self.head_gate or not self.own_kv or not self.norm_weights:
+            raise ValueError("attention: values that are the keys go without kept first tokens, gates or borrowed keys")
+        # rows of the gate inside the input product, padded with zero rows so that a product's row stays a multiple of 16 bytes
+        self.gate_rows = 0
+        if self.head_gate:
+            kv = self.kv_dim + self.v_dim if self.own_kv else 0
+            self.gate_rows = self.heads + -(self.q_dim + kv + self.heads) % 16
         self.conv_w: Optional[torch.Tensor] = None
         self.q_norm_w: Optional[torch.Tensor] = None
         self.k_norm_w: Optional[torch.Tensor] = None
@@ -166,9 +198,13 @@ class GQAttention(Mixer):
         }
         if self.values_are_keys:
             del specs["v.weight"]
+        if not self.own_kv:
+            del specs["k.weight"], specs["v.weight"]
+        if self.head_gate:
+            specs["gate.weight"] = ParamSpec((self.heads, self.hidden))
         if self.dist_far is not None:
             specs["rel"] = ParamSpec((-1, self.heads), role="vector")
-        if self.qk_norm is not None:
+        if self.qk_norm is not None and self.norm_weights:
             per_head = self.qk_norm[0] == "head"
             specs["q_norm.weight"] = ParamSpec((self.head_dim if per_head else self.q_dim,), role="vector")
             specs["k_norm.weight"] = ParamSpec((self.head_dim if per_head else self.kv_dim,), role="vector")
@@ -193,15 +229,21 @@ class GQAttention(Mixer):
 
     def load(self, tensors: Dict[str, torch.Tensor]) -> None:
         # rows of q, then k, then v: one product serves all three
-        rows = ("q", "k") if self.values_are_keys else ("q", "k", "v")
-        self.w_qkv = torch.cat([tensors[f"{t}.weight"] for t in rows], dim=0).contiguous()
+        rows = ("q", "k") if self.values_are_keys else ("q", "k", "v") if self.own_kv else ("q",)
+        blocks = [tensors[f"{t}.weight"] for t in rows]
+        if self.head_gate:
+            gate = tensors["gate.weight"]
+            blocks += [gate, gate.new_zeros((self.gate_rows - self.heads, self.hidden))]
+        self.w_qkv = torch.cat(blocks, dim=0).contiguous()
         if self.qkv_bias:
             self.b_qkv = torch.cat([tensors[f"{t}.bias"] for t in rows]).contiguous()
         if self.dist_far is not None:
             self.dist_table = self.expand_distance_bias(tensors["rel"], self.dist_far)
         self.w_o = tensors["o.weight"].contiguous()
         self.b_o = tensors["o.bias"].contiguous() if self.o_bias else None
-        if self.qk_norm is not None:
+        if self.qk_norm is not None and not self.norm_weights:
+            self.q_norm_w = self.k_norm_w = torch.ones(self.head_dim, dtype=torch.float32, device=self.w_o.device)
+        elif self.qk_norm is not None:
             self.q_norm_w = tensors["q_norm.weight"].contiguous()
             self.k_norm_w = tensors["k_norm.weight"].contiguous()
         if self.sinks:
@@ -239,7 +281,14 @@ class GQAttention(Mixer):
         return rel.float()[index].t().contiguous()
 
     def flops(self, tokens: int, pairs: float) -> float:
-        products = 2.0 * tokens * (self.q_dim + self.kv_dim + self.v_dim + self.o_dim) * self.hidden
+        kv = self.kv_dim + self.v_dim if self.own_kv else 0
+        products = 2.0 * tokens * (self.q_dim + kv + self.o_dim + (self.heads if self.head_gate else 0)) * self.hidden
+        if self.separate and self.window is not None:
+            # a query meets at most the window's keys and the kept ones
+            limit = int(self.window) + self.keep_first
+            if 2.0 * pairs == tokens * (tokens + 1.0):                    # a whole prompt
+                pairs -= max(tokens - limit, 0) * (tokens - limit + 1.0) / 2.0
+            pairs = min(pairs, float(tokens * limit))
         return products + 2.0 * self.heads * (self.head_dim + self.value_dim) * pairs     # scores and weighted values
 
     def attend_keyed(self, h, ctx: StepContext, cache: LayerCache, out: Optional[torch.Tensor] = None) -> torch.Tensor:
@@ -261,12 +310,38 @@ class GQAttention(Mixer):
                              typical_ctx_len=ctx.typical_ctx_len, decode_prefix=ctx.decode_prefix, sink=self.sink, out=out,
                              dist_bias=self.dist_table)
 
+    def attend_separate(self, h, ctx: StepContext, cache: LayerCache, out: Optional[torch.Tensor] = None) -> torch.Tensor:
+        """Product of q, k, v and the gates; q and k normalised, k and v stored; attention with bias, kept tokens and gates."""
+        ops = self.ops
+        complete = getattr(h, "complete", None)
+        if complete is not None:
+            h = complete()
+        k_pages, v_pages = cache.paged["k"], cache.paged["v"]
+        table = ctx.block_tables[cache.group]
+        rows = ops.linear(h, self.w_qkv, None, ops.GEMM_STORE)
+        if self.own_kv and not cache.owner:
+            raise RuntimeError("attention: a layer with keys of its own was given another layer's cache")
+        if self.own_kv or self.qk_norm is not None:
+            ops.qk_norm_kv_store(rows, self.q_norm_w, self.k_norm_w if self.own_kv else None, self.qk_norm[1] if self.qk_norm else 1.0,
+                                 True, ctx.positions, ctx.seq_of_token, table if self.own_kv else None,
+                                 k_pages if self.own_kv else None, v_pages if self.own_kv else None, self.heads,
+                                 self.kv_heads if self.own_kv else 0, self.head_dim, self.value_dim)
+        gate = None
+        if self.head_gate:
+            first = self.q_dim + (self.kv_dim + self.v_dim if self.own_kv else 0)
+            gate = rows[:, first:first + self.heads]
+        return ops.attention(rows[:, :self.q_dim], k_pages, v_pages, table, ctx.q_start, ctx.start_pos, ctx.positions,
+                             ctx.seq_of_token, ctx.num_seqs, ctx.max_q_len, ctx.max_ctx_len, self.heads, self.kv_heads,
+                             self.head_dim, self.scale, window=int(self.window or 0), split_tokens=ctx.attn_split_tokens,
+                             typical_ctx_len=ctx.typical_ctx_len, decode_prefix=ctx.decode_prefix, sink=self.sink, out=out,
+                             dist_bias=self.dist_table, keep_first=self.keep_first, gate=gate)
+
     def cache_spec(self) -> Optional[PagedCacheSpec]:
         # with pooled blocks a token is also read when its block is averaged, which is when the block's last token
         # arrives: the pages keep whichever reaches further back, the window or a block
         window = None if self.window is None else max(int(self.window), self.pool)
         return PagedCacheSpec(entries=(("k", (self.kv_heads, self.head_dim)), ("v", (self.kv_heads, self.value_dim))),
-                              window=window)
+                              window=window, keep_first=self.keep_first)
 
     def extra_cache_specs(self) -> Dict[str, PagedCacheSpec]:
         if not self.pool:
@@ -310,7 +385,7 @@ class GQAttention(Mixer):
         multiplied together with q, k and v.  A mixer whose small-batch kernel can carry them (whole-projection
         q/k norm, no rotation, no biases) puts them below its own rows in one tensor and returns the view that now
         holds them (the caller uses it in place of its copy); None: it cannot."""
-        if (self.plain or self.general or self.values_are_keys or self.rotates or self.qkv_bias
+        if (self.plain or self.general or self.values_are_keys or self.separate or self.rotates or self.qkv_bias
                 or (self.qk_norm is not None and self.qk_norm[0] != "projection")):
             return None
         if self.w_qkv is None or rows.dtype != self.w_qkv.dtype or rows.shape[1] != self.hidden:
@@ -326,8 +401,9 @@ class GQAttention(Mixer):
 
         ``beside``: (output view, epilogue) for the rows that :meth:`share_input_projection` took in; the result is
         then a pair (rows, whether the shared rows were multiplied and activated here)."""
-        if self.general or self.values_are_keys:
-            a = (self.attend_keyed if self.values_are_keys else self.attend_general)(h, ctx, cache, out=out)
+        if self.general or self.values_are_keys or self.separate:
+            attend = self.attend_keyed if self.values_are_keys else self.attend_separate if self.separate else self.attend_general
+            a = attend(h, ctx, cache, out=out)
             return a if beside is None else (a, False)
         ops = self.ops
         k_pages, v_pages = cache.paged["k"], cache.paged["v"]

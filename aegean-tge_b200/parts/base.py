@@ -62,14 +62,25 @@ class PagedCacheSpec:
     pages wholly behind the window are given back.  ``stride`` > 1: one entry per
     block of that many positions (pooled keys and values), kept once the block
     is whole; entry b of a request then sits where position b would.
+    ``keep_first``: with a window, the first so many tokens of a request stay readable beside it, and their pages
+    are kept.
     """
 
     entries: Tuple[Tuple[str, Tuple[int, ...]], ...]
     window: Optional[int] = None
     stride: int = 1
+    keep_first: int = 0
 
     def group_key(self) -> Tuple:
-        return (self.entries, self.window, self.stride)
+        return (self.entries, self.window, self.stride, self.keep_first)
+
+    def covering(self, other: "PagedCacheSpec") -> "PagedCacheSpec":
+        """This spec, keeping also whatever ``other`` may read of the same entries (another layer's mixer over them)."""
+        if other.entries != self.entries or other.stride != self.stride:
+            raise ValueError(f"a mixer reads entries {other.entries} of a cache that keeps {self.entries}")
+        if self.window is None or other.window is None:
+            return PagedCacheSpec(self.entries, None, self.stride)
+        return PagedCacheSpec(self.entries, max(self.window, other.window), self.stride, max(self.keep_first, other.keep_first))
 
 
 @dataclass(frozen=True)
@@ -239,7 +250,7 @@ class Mixer(Part):
         total = 0
         spec = self.cache_spec()
         if spec is not None:
-            seen = context if spec.window is None else min(context, int(spec.window))
+            seen = context if spec.window is None else min(context, int(spec.window) + int(spec.keep_first))
             total += seen * per_entry(spec) * self.env.dtype.itemsize
         for extra in self.extra_cache_specs().values():
             total += (context // extra.stride) * per_entry(extra) * self.env.dtype.itemsize

@@ -18,7 +18,16 @@ one dt per head); x, B and C pass the convolution (with a bias) and SiLU; dt <- 
 
 y times silu(z), normalised in ``norm_groups`` equal parts (the gate comes before the norm), times a weight; then Wo.
 
-Both keep, per request, the state S in float32 and the convolution's last taps-1 inputs.  They share their kernels:
+``matrix_lstm``: q = Wq h, k = Wk h (``heads`` heads of ``head_dim``), v = Wv h; per head a log input gate i = cap tanh((Wi h +
+bi) / cap) and a log forget gate f = logsigmoid(cap tanh((Wf h + bf) / cap)), a running maximum m that starts at 0, and
+
+    m' = max(f + m, i);  S <- exp(f + m - m') S + exp(i - m') k v^T;  n <- likewise with k alone
+    o = S^T q' / (max(|n . q'|, exp(-m')) + 1e-6),   q' = q head_dim^-1/2
+
+each head's o over its root mean square, times a weight of all heads' size, times sigmoid(Wg h); then Wo.  It has kernels of
+its own (``ops.mlstm_step``) and keeps S, n and m per request.
+
+The first two keep, per request, the state S in float32 and the convolution's last taps-1 inputs.  They share their kernels:
 ``ops.gated_prepare`` readies what the recurrence takes, ``ops.gated_rule_scan`` walks the tokens (the state-space
 recurrence is the delta rule without its correction, with k = B, q = C, b = dt), ``ops.gated_norm`` normalises and gates.
 """
@@ -29,6 +38,8 @@ from typing import Dict, Optional
 import torch
 
 from .base import MIXERS, LayerCache, Mixer, ParamSpec, StateSpec, StepContext
+
+MLSTM_MAX_KEYS, MLSTM_MAX_VALUES = 1024, 1024      # what a block's shared memory holds of one head's vectors
 
 
 class _MatrixStateMixer(Mixer):
@@ -194,3 +205,85 @@ class StateSpace(_MatrixStateMixer):
                                 skip=self.skip)
         return ops.gated_norm(y, raw[:, :self.o_dim], self.norm_w, self.norm_groups, self.eps, sigmoid=False, out=out,
                               gate_first=True, out_dtype=self.env.dtype)
+
+
+@MIXERS.register("matrix_lstm")
+class MatrixLSTM(Mixer):
+    """params: ``hidden_size``, ``heads``, ``head_dim``, ``value_dim``, ``gate_cap``, ``eps`` (of the readout's norm).
+    weights: ``q|k|v|g|o.weight``, ``i|f.weight`` [heads, hidden], ``i|f.bias`` (float32 [heads]), ``norm.weight`` (float32
+    [heads value_dim]).  q, k, v and g come from one product in the run's format; the two gates' logits from a product of
+    their own that is stored in float32, their biases in its epilogue."""
+    graph_safe = True
+
+    def __init__(self, spec, env):
+        super().__init__(spec, env)
+        p = spec.params
+        self.hidden = int(p["hidden_size"])
+        self.heads = int(p["heads"])
+        self.key_dim = int(p["head_dim"])
+        self.value_dim = int(p["value_dim"])
+        self.cap = float(p["gate_cap"])
+        self.eps = float(p["eps"])
+        if min(self.hidden, self.heads, self.key_dim, self.value_dim) <= 0 or not self.cap > 0.0 or not self.eps > 0.0:
+            raise ValueError("matrix_lstm: sizes, the gates' cap and eps must be positive")
+        if self.value_dim > MLSTM_MAX_VALUES or self.key_dim > MLSTM_MAX_KEYS:
+            raise ValueError(f"matrix_lstm: heads of {self.key_dim} x {self.value_dim} (up to {MLSTM_MAX_KEYS} x {MLSTM_MAX_VALUES})")
+        self.qk_dim = self.heads * self.key_dim
+        self.o_dim = self.heads * self.value_dim
+        self.w_in: Optional[torch.Tensor] = None
+        self.w_gates: Optional[torch.Tensor] = None
+        self.b_gates: Optional[torch.Tensor] = None
+        self.w_o: Optional[torch.Tensor] = None
+        self.norm_w: Optional[torch.Tensor] = None
+
+    def param_specs(self) -> Dict[str, ParamSpec]:
+        return {"q.weight": ParamSpec((self.qk_dim, self.hidden)), "k.weight": ParamSpec((self.qk_dim, self.hidden)),
+                "v.weight": ParamSpec((self.o_dim, self.hidden)), "g.weight": ParamSpec((self.o_dim, self.hidden)),
+                "i.weight": ParamSpec((self.heads, self.hidden)), "f.weight": ParamSpec((self.heads, self.hidden)),
+                "i.bias": ParamSpec((self.heads,), role="vector"), "f.bias": ParamSpec((self.heads,), role="vector"),
+                "norm.weight": ParamSpec((self.o_dim,), role="vector"), "o.weight": ParamSpec((self.hidden, self.o_dim))}
+
+    def load(self, tensors: Dict[str, torch.Tensor]) -> None:
+        self.w_in = torch.cat([tensors[f"{t}.weight"] for t in ("q", "k", "v", "g")], dim=0).contiguous()
+        self.w_gates = torch.cat([tensors["i.weight"], tensors["f.weight"]], dim=0).contiguous()
+        self.b_gates = torch.cat([tensors["i.bias"], tensors["f.bias"]]).contiguous()
+        self.norm_w = tensors["norm.weight"].contiguous()
+        self.w_o = tensors["o.weight"].contiguous()
+
+    def state_spec(self) -> Optional[StateSpec]:
+        return StateSpec(entries=(("state", (self.heads, self.key_dim, self.value_dim)), ("normaliser", (self.heads, self.key_dim)),
+                                  ("maximum", (self.heads,))))
+
+    def flops(self, tokens: int, pairs: float) -> float:
+        products = 2.0 * tokens * (2 * self.qk_dim + 3 * self.o_dim + 2 * self.heads) * self.hidden
+        return products + 4.0 * tokens * self.heads * self.key_dim * (self.value_dim + 1)      # write and readout
+
+    def inner(self, h: torch.Tensor, ctx: StepContext, cache: LayerCache, out: Optional[torch.Tensor] = None):
+        ops = self.ops
+        complete = getattr(h, "complete", None)
+        if complete is not None:
+            h = complete()
+        rows = ops.linear(h, self.w_in, None, ops.GEMM_STORE)
+        gates = ops.linear(h, self.w_gates, self.b_gates, ops.GEMM_STORE_F32)
+        state = cache.state
+        return ops.mlstm_step(rows, gates, self.heads, self.key_dim, self.value_dim, self.norm_w, state["state"],
+                              state["normaliser"], state["maximum"], ctx.slots, ctx.q_start, ctx.num_seqs, self.cap,
+                              self.key_dim ** -0.5, self.eps, out=out)
+
+    def output_projection(self):
+        return self.w_o, None
+
+    def forward(self, h: torch.Tensor, ctx: StepContext, cache: LayerCache) -> torch.Tensor:
+        return self.ops.linear(self.inner(h, ctx, cache), self.w_o, None, self.ops.GEMM_STORE)
+
+    def forward_f32(self, h, ctx: StepContext, cache: LayerCache, out=None, alpha: float = 1.0, accumulate: bool = False):
+        epilogue = self.ops.GEMM_ADD_F32 if accumulate else self.ops.GEMM_STORE_F32
+        return self.ops.linear(self.inner(h, ctx, cache), self.w_o, None, epilogue, out=out, alpha=alpha)
+
+    def forward_add(self, h: torch.Tensor, x: torch.Tensor, ctx: StepContext, cache: LayerCache, next_norm=None):
+        a = self.inner(h, ctx, cache)
+        fused = next_norm.fusable() if next_norm is not None else None
+        if fused is not None:
+            return self.ops.linear_add_norm(a, self.w_o, None, x, fused[0], fused[1], self.env.dtype)
+        self.ops.linear(a, self.w_o, None, self.ops.GEMM_ADD_F32, out=x)
+        return None

@@ -8,6 +8,11 @@ With h the input, R = experts + identity router outputs:
     w_k = s_k / (sum of the chosen s + 1e-20)
     out = sum_k w_k E_k(h)      E_e(h) = Wdown_e relu(Wup_e h)^2 for an expert, h itself for an identity output
 
+Parameters change four things: the scores may be each output's own logistic function instead of the softmax; the weights
+the chosen scores as they are instead of over their sum; a weight may multiply its expert's INPUT, E(w h), instead of the
+output; and an expert may be a clamped gated feed-forward, Wdown (g sigmoid(alpha g) (u + offset)) with g = min(Wgate h, L)
+and u = clamp(Wup h, -L, L), its gate and up rows interleaved in one matrix.
+
 The correction steers the choice only; the weights use the plain scores.  Identity outputs are the last ``identity``
 router outputs and have no tensors.  The sum over a token's choices is formed in float32 in the order of the choice
 and added into the float32 stream.
@@ -41,14 +46,17 @@ DENSE_MAX_TOKENS = 256      # beyond this many tokens the wasted products of the
 class RoutedExperts(FeedForward):
     """params: ``hidden_size``, ``intermediate_size`` (an expert's inner width), ``experts``, ``top``, optional
     ``identity`` (default 0), ``group_count`` / ``group_keep`` (default 1 / 1: no groups), ``correction`` (bool,
-    default True: the checkpoint holds a correction of the choice), ``activation`` (``"relu_squared"``, the only one
-    the expert kernels apply so far), ``router_bias`` (bool, default False: a bias added to the router's logits, so it
+    default True: the checkpoint holds a correction of the choice), ``activation`` (``"relu_squared"`` or
+    ``"clamped_glu"``, the latter with ``limit`` and optionally ``alpha``, default 1.702, and ``up_offset``, default 1),
+    ``score`` (``"softmax"`` or ``"logistic"``), ``weights_over_sum`` (bool, default True), ``weigh`` (``"output"`` or
+    ``"input"``; the latter without identity experts), ``router_bias`` (bool, default False: a bias added to the router's logits, so it
     steers the choice and the weights alike), ``shared`` (None, or the PartSpec of a feed-forward that every token
     uses and whose output is added; its parameters are this part's under ``shared.<local name>``).
     With no correction and no groups the weights are the softmax over the chosen logits alone: a chosen output's share
     of the softmax over all, divided by the chosen ones' sum, is the same number.
     weights: ``router.weight`` [experts + identity, hidden], ``router.bias`` and ``correction`` (float32 [experts +
-    identity]), ``experts.<e>.up.weight`` [inner, hidden], ``experts.<e>.down.weight`` [hidden, inner]."""
+    identity]), ``experts.<e>.up.weight`` [inner, hidden] (and ``experts.<e>.gate.weight`` of gated ones),
+    ``experts.<e>.down.weight`` [hidden, inner]."""
     graph_safe = True
 
     def __init__(self, spec, env):
@@ -69,8 +77,22 @@ class RoutedExperts(FeedForward):
             self.graph_safe = bool(self.shared.graph_safe)
         self.router_bias: Optional[torch.Tensor] = None
         self.outputs = self.experts + self.identity
-        if str(p.get("activation", "relu_squared")) != "relu_squared":
+        activation = str(p.get("activation", "relu_squared"))
+        self.gate = None                       # (limit, alpha, offset) of clamped gated experts
+        if activation == "clamped_glu":
+            self.gate = (float(p["limit"]), float(p.get("alpha", 1.702)), float(p.get("up_offset", 1.0)))
+            if not self.gate[0] > 0.0:
+                raise ValueError("routed_experts: the limit must be positive")
+        elif activation != "relu_squared":
             raise ValueError(f"routed_experts: unknown activation '{p.get('activation')}'")
+        self.matrices = 2 if self.gate is None else 3
+        self.logistic = str(p.get("score", "softmax")) == "logistic"
+        self.over_sum = bool(p.get("weights_over_sum", True))
+        self.weigh_input = str(p.get("weigh", "output")) == "input"
+        if str(p.get("score", "softmax")) not in ("softmax", "logistic") or str(p.get("weigh", "output")) not in ("output", "input"):
+            raise ValueError(f"routed_experts: score {p.get('score')!r} or weigh {p.get('weigh')!r} is not known")
+        if self.weigh_input and (self.identity or self.gate is None):
+            raise ValueError("routed_experts: weights on the input go with gated experts and without identity experts")
         if min(self.hidden, self.inner_size, self.top, self.group_count, self.group_keep) <= 0 or self.experts < 0 \
                 or self.identity < 0 or self.outputs <= 0:
             raise ValueError("routed_experts: sizes must be positive")
@@ -82,7 +104,7 @@ class RoutedExperts(FeedForward):
             raise ValueError("routed_experts: the router kernel takes up to 1024 outputs")
         self.w_router: Optional[torch.Tensor] = None
         self.correction: Optional[torch.Tensor] = None
-        self.w_up: Optional[torch.Tensor] = None         # [experts, inner, hidden]
+        self.w_up: Optional[torch.Tensor] = None         # [experts, inner, hidden]; gated: [experts, 2 inner, hidden]
         self.w_down: Optional[torch.Tensor] = None       # [hidden, experts, inner]
 
     def param_specs(self) -> Dict[str, ParamSpec]:
@@ -94,6 +116,8 @@ class RoutedExperts(FeedForward):
         if self.shared is not None:
             specs.update({f"shared.{local}": param for local, param in self.shared.param_specs().items()})
         for e in range(self.experts):
+            if self.gate is not None:
+                specs[f"experts.{e}.gate.weight"] = ParamSpec((self.inner_size, self.hidden))
             specs[f"experts.{e}.up.weight"] = ParamSpec((self.inner_size, self.hidden))
             specs[f"experts.{e}.down.weight"] = ParamSpec((self.hidden, self.inner_size))
         return specs
@@ -105,7 +129,11 @@ class RoutedExperts(FeedForward):
         if self.shared is not None:
             self.shared.load({name[len("shared."):]: t for name, t in tensors.items() if name.startswith("shared.")})
         if self.experts:
-            self.w_up = torch.stack([tensors[f"experts.{e}.up.weight"] for e in range(self.experts)]).contiguous()
+            if self.gate is None:
+                self.w_up = torch.stack([tensors[f"experts.{e}.up.weight"] for e in range(self.experts)]).contiguous()
+            else:
+                self.w_up = torch.stack([torch.stack([tensors[f"experts.{e}.gate.weight"], tensors[f"experts.{e}.up.weight"]], dim=1)
+                                         .reshape(2 * self.inner_size, self.hidden) for e in range(self.experts)]).contiguous()
             self.w_down = torch.stack([tensors[f"experts.{e}.down.weight"] for e in range(self.experts)], dim=1).contiguous()
         else:
             self.w_up = torch.empty((0, self.inner_size, self.hidden), dtype=self.w_router.dtype, device=self.w_router.device)
@@ -115,7 +143,7 @@ class RoutedExperts(FeedForward):
         """What one token's step reads: the router and the chosen experts (a large batch touches more of them)."""
         item = self.env.dtype.itemsize
         extra = self.shared.param_bytes() if self.shared is not None else 0
-        return (self.outputs * self.hidden + min(self.top, self.experts) * 2 * self.inner_size * self.hidden) * item + 4 * self.outputs + extra
+        return (self.outputs * self.hidden + min(self.top, self.experts) * self.matrices * self.inner_size * self.hidden) * item + 4 * self.outputs + extra
 
     def dense(self, tokens: int) -> bool:
         """Whether a step of this many tokens runs all experts (its choices reach most of them anyway)."""
@@ -127,11 +155,11 @@ class RoutedExperts(FeedForward):
         item = self.env.dtype.itemsize
         reached = self.experts if self.dense(tokens) else self.experts * (1.0 - (1.0 - min(self.top / self.outputs, 1.0)) ** tokens)
         extra = self.shared.param_bytes() if self.shared is not None else 0
-        return int((self.outputs * self.hidden + reached * 2 * self.inner_size * self.hidden) * item) + 4 * self.outputs + extra
+        return int((self.outputs * self.hidden + reached * self.matrices * self.inner_size * self.hidden) * item) + 4 * self.outputs + extra
 
     def flops(self, tokens: int, pairs: float) -> float:
         extra = self.shared.flops(tokens, pairs) if self.shared is not None else 0.0
-        return 2.0 * tokens * (self.outputs * self.hidden + self.top * 2 * self.inner_size * self.hidden) + extra
+        return 2.0 * tokens * (self.outputs * self.hidden + self.top * self.matrices * self.inner_size * self.hidden) + extra
 
     def route(self, h: torch.Tensor):
         """(ids int32 [T, top], weights float32 [T, top]); the logits are a float32 product of the rows as given."""
@@ -139,7 +167,8 @@ class RoutedExperts(FeedForward):
         if complete is not None:
             h = complete()
         logits = self.ops.linear(h, self.w_router, self.router_bias, self.ops.GEMM_STORE_F32)
-        ids, weights = self.ops.router_topk(logits, self.correction, self.top, self.group_count, self.group_keep)
+        ids, weights = self.ops.router_topk(logits, self.correction, self.top, self.group_count, self.group_keep,
+                                            logistic=self.logistic, over_sum=self.over_sum)
         return h, ids, weights
 
     def forward_add(self, h: torch.Tensor, x: torch.Tensor, ctx: StepContext, next_norm=None):
@@ -155,30 +184,42 @@ class RoutedExperts(FeedForward):
         h, ids, weights = self.route(h)
         tokens = h.shape[0]
         few = ctx.max_q_len <= 1 or tokens <= DIRECT_MAX_TOKENS
+        if self.dense(tokens) and self.gate is not None:
+            z = ops.linear(h, self.w_up.view(self.experts * 2 * self.inner_size, self.hidden), None, ops.GEMM_STORE)
+            a = ops.experts_dense_gate(z, ids, weights, self.experts, self.gate, self.weigh_input)
+            ops.linear(a, self.w_down.view(self.hidden, self.experts * self.inner_size), None, ops.GEMM_ADD_F32, out=x)
+            return h
         if self.dense(tokens):
             z = ops.linear(h, self.w_up.view(self.experts * self.inner_size, self.hidden), None, ops.GEMM_STORE)
             ops.experts_dense_weigh(z, ids, weights, h, x, self.experts)
             ops.linear(z, self.w_down.view(self.hidden, self.experts * self.inner_size), None, ops.GEMM_ADD_F32, out=x)
             return h
         if few or self.experts == 0:
-            ops.experts_direct(h, self.w_up, self.w_down, ids, weights, x)
+            ops.experts_direct(h, self.w_up, self.w_down, ids, weights, x, gate=self.gate, weigh_input=self.weigh_input)
             return h
-        place, offsets, grouped = ops.experts_group(h, ids, self.experts)
+        place, offsets, grouped = ops.experts_group(h, ids, self.experts, in_weights=weights if self.weigh_input else None)
         bounds: List[int] = offsets.tolist()             # the host learns the group sizes: not a captured step
         rows = bounds[-1]
         inner = torch.empty((max(rows, 1), self.inner_size), dtype=h.dtype, device=h.device)
         outputs = torch.empty((max(rows, 1), self.hidden), dtype=torch.float32, device=h.device)
+        fused = self.gate is not None and self.gate[1:] == (1.702, 1.0)      # the gate is the product's own epilogue
         for e in range(self.experts):
             lo, hi = bounds[e], bounds[e + 1]
             if hi > lo:
-                ops.linear(grouped[lo:hi], self.w_up[e], None, ops.GEMM_STORE, out=inner[lo:hi])
-        if rows:
+                if fused:
+                    ops.linear(grouped[lo:hi], self.w_up[e], None, ops.GEMM_GLU_CLAMPED, out=inner[lo:hi], alpha=self.gate[0])
+                elif self.gate is not None:
+                    both = ops.linear(grouped[lo:hi], self.w_up[e], None, ops.GEMM_STORE_F32)
+                    ops.gated_clamp_act(both, *self.gate, self.env.dtype, out=inner[lo:hi])
+                else:
+                    ops.linear(grouped[lo:hi], self.w_up[e], None, ops.GEMM_STORE, out=inner[lo:hi])
+        if rows and self.gate is None:
             ops.activation(inner[:rows], ops.ACT_RELU_SQUARED)
         for e in range(self.experts):
             lo, hi = bounds[e], bounds[e + 1]
             if hi > lo:
                 ops.linear(inner[lo:hi], self.w_down[:, e, :], None, ops.GEMM_STORE_F32, out=outputs[lo:hi])
-        ops.experts_combine_add(outputs, place, weights, h, x)
+        ops.experts_combine_add(outputs, place, None if self.weigh_input else weights, h, x)
         return h
 
     def forward_f32(self, h: torch.Tensor, ctx: StepContext) -> torch.Tensor:
