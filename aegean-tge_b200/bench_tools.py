@@ -224,7 +224,31 @@ def paired_configs(width: int, heads: int, kv_heads: int, head_dim: int, gated_i
                "logit_scale": 1.0, "logit_softcap": 50.0, "layers": [layer] * layers}
     return {"qwen2": qwen2, "lepizen": lepizen, "mozepel": mozepel_config(width, heads, kv_heads, head_dim, gated_inner, layers, vocab),
             "puputar": puputar_config(width, heads, head_dim, gated_inner, layers, vocab),
-            "kokolorn": kokolorn_config(width, heads, kv_heads, head_dim, gated_inner, layers, vocab)}
+            "kokolorn": kokolorn_config(width, heads, kv_heads, head_dim, gated_inner, layers, vocab),
+            "fesorax": fesorax_config(width, heads, kv_heads, head_dim, gated_inner, layers, vocab)}
+
+
+def fesorax_config(width: int, heads: int, kv_heads: int, head_dim: int, gated_inner: int, layers: int, vocab: int,
+                   experts: int = 16, top: int = 4, window: int = 1024, keep_first: int = 16) -> dict:
+    """A Fesorax config.json with the width, heads, kv heads, head size and layer count of a Qwen2 shape, its layers by turns
+    mlstm (as many heads, keys and values of ``head_dim``), attention (the shape's GQA over a window with ``keep_first`` kept
+    tokens and a bias by distance up to 2,048), mlstm again and an attention that reads the keys and values of the one
+    before; every layer with ``experts`` gated experts of three sixteenths of the gated inner width, of which ``top`` are
+    used, and a shared one of a quarter of it: as many multiplications per token as the dense feed-forward."""
+    unit = max(gated_inner // 16 // 64 * 64, 64)
+    moe = {"kind": "moe", "expert": {"ff": 3 * unit, "limit": 7.0}, "router": {"experts": experts, "top": top},
+           "shared": {"ff": 4 * unit, "limit": 7.0}}
+    memory = {"type": "mlstm", "mixer": {"heads": heads, "dim": head_dim, "vdim": head_dim, "gate_cap": 15.0}, "mlp": moe}
+    attention = {"heads": heads, "kv_heads": kv_heads, "dim": head_dim, "vdim": head_dim, "scale": head_dim ** -0.5, "bias_max": 2048,
+                 "mask": {"size": window, "keep_first": keep_first}}
+    out = []
+    for n in range(layers):
+        if n % 2 == 0:
+            out.append(memory)
+        else:
+            out.append({"type": "attention", "mixer": dict(attention, **({"kv_from": n - 2} if n % 4 == 3 else {})), "mlp": moe})
+    return {"architecture": "Fesorax", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "embedding": {"scale": 1.0},
+            "postln_alpha": 2.0, "layers": out}
 
 
 def kokolorn_config(width: int, heads: int, kv_heads: int, head_dim: int, gated_inner: int, layers: int, vocab: int,

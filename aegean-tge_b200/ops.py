@@ -127,6 +127,11 @@ def core() -> ctypes.CDLL:
         _declare(lib, "tge_mlstm_step", [_c_ptr, _c_int, _c_ll, _c_ptr, _c_ll, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_ptr,
                                          _c_ptr, _c_ll, _c_int, _c_int, _c_int, _c_int, _c_int, _c_float, _c_float, _c_float,
                                          _c_ptr])
+        lib.tge_mlstm_chunks_supported.argtypes = [_c_int, _c_int]
+        lib.tge_mlstm_chunks_supported.restype = _c_int
+        _declare(lib, "tge_mlstm_chunks", [_c_ptr, _c_ll, _c_ptr, _c_ll, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_ptr,
+                                           _c_ll, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_float, _c_float, _c_float,
+                                           _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_int, _c_ptr])
         _declare(lib, "tge_experts_group", [_c_ptr, _c_ll, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_int, _c_int, _c_int,
                                             _c_int, _c_ptr])
         _declare(lib, "tge_experts_combine_add", [_c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_ll, _c_ptr, _c_int, _c_int, _c_int,
@@ -1665,6 +1670,68 @@ def gated_rule_scan(qk: torch.Tensor, v: torch.Tensor, gates: torch.Tensor, stat
                                    vdim, state.data_ptr(), slots.data_ptr(), q_start.data_ptr(), out.data_ptr(), num_seqs,
                                    tokens, _stream()), lib)
     return out
+
+
+MLSTM_CHUNK = 64            # tokens the chunk kernels take at a time
+MLSTM_SHORT = 16            # portions of up to this many tokens are walked token by token
+MLSTM_WAVE = 64             # chunks whose states lie in scratch memory at a time
+
+
+def mlstm(rows: torch.Tensor, gates: torch.Tensor, heads: int, dim: int, vdim: int, norm_weight: torch.Tensor,
+          state: torch.Tensor, normaliser: torch.Tensor, maximum: torch.Tensor, slots: torch.Tensor, q_start: torch.Tensor,
+          lengths, cap: float, q_scale: float, eps: float, out: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """The matrix memory of an mLSTM over a step of portions (see :func:`mlstm_step`).  ``lengths``: the portions' lengths,
+    known to the host.  In bfloat16, portions of more than ``MLSTM_SHORT`` tokens go through the chunk kernels where the
+    sizes allow it, everything else token by token; the two agree to rounding."""
+    lib = core()
+    fits = (rows.dtype == torch.bfloat16 and bool(lib.tge_mlstm_chunks_supported(dim, vdim)) and rows.stride(0) % 8 == 0
+            and rows.data_ptr() % 16 == 0)
+    if out is None:
+        out = torch.empty((rows.shape[0], heads * vdim), dtype=rows.dtype, device=rows.device)
+    fits = fits and out.stride(0) % 2 == 0 and out.data_ptr() % 4 == 0
+    long = [n for n in lengths if n > MLSTM_SHORT] if fits else []
+    if long:
+        mlstm_chunks(rows, gates, heads, dim, vdim, norm_weight, state, normaliser, maximum, slots, q_start, lengths, cap, q_scale,
+                     eps, out)
+    if len(long) < len(lengths):
+        mlstm_step(rows, gates, heads, dim, vdim, norm_weight, state, normaliser, maximum, slots, q_start, len(lengths), cap,
+                   q_scale, eps, longest=MLSTM_SHORT if long else 2 ** 31 - 1, out=out)
+    return out
+
+
+def mlstm_chunks(rows: torch.Tensor, gates: torch.Tensor, heads: int, dim: int, vdim: int, norm_weight: torch.Tensor,
+                 state: torch.Tensor, normaliser: torch.Tensor, maximum: torch.Tensor, slots: torch.Tensor,
+                 q_start: torch.Tensor, lengths, cap: float, q_scale: float, eps: float, out: torch.Tensor) -> None:
+    """The portions of more than ``MLSTM_SHORT`` tokens, in chunks on the tensor cores (bfloat16); see :func:`mlstm`."""
+    _want(rows, "projections", torch.bfloat16, contiguous=False)
+    _want(out, "readout", torch.bfloat16, contiguous=False)
+    _want(gates, "gate logits", torch.float32, contiguous=False)
+    for name, t in (("norm weight", norm_weight), ("state", state), ("normaliser", normaliser), ("maximum", maximum)):
+        _want(t, name, torch.float32)
+    _want(slots, "slots", torch.int32)
+    _want(q_start, "q_start", torch.int32)
+    tokens, device = rows.shape[0], rows.device
+    if (rows.shape[1] < 2 * heads * (dim + vdim) or gates.shape[0] != tokens or gates.shape[1] < 2 * heads
+            or tuple(state.shape[1:]) != (heads, dim, vdim) or tuple(normaliser.shape[1:]) != (heads, dim)
+            or tuple(maximum.shape[1:]) != (heads,) or norm_weight.numel() != heads * vdim or sum(lengths) != tokens
+            or tuple(out.shape) != (tokens, heads * vdim)):
+        raise KernelError(f"mlstm_chunks: rows {tuple(rows.shape)}, gates {tuple(gates.shape)}, state {tuple(state.shape)}, "
+                          f"normaliser {tuple(normaliser.shape)}, maximum {tuple(maximum.shape)}, portions {list(lengths)}")
+    chunks = sum(-(-n // MLSTM_CHUNK) for n in lengths if n > MLSTM_SHORT)
+    wave = min(chunks, MLSTM_WAVE)
+    g, top = torch.empty((2, heads, tokens), dtype=torch.float64, device=device)
+    floor = torch.empty((heads, tokens), dtype=torch.float32, device=device)
+    start = torch.empty((len(lengths), heads), dtype=torch.float64, device=device)
+    own = torch.empty((wave, heads, dim, vdim), dtype=torch.float32, device=device)
+    before = torch.empty((3, wave, heads, dim, vdim), dtype=torch.bfloat16, device=device)
+    norm_own = torch.empty((wave, heads, dim), dtype=torch.float32, device=device)
+    lib = core()
+    _check(lib.tge_mlstm_chunks(rows.data_ptr(), _rows_2d(rows, "projections"), gates.data_ptr(), _rows_2d(gates, "gate logits"),
+                                norm_weight.data_ptr(), state.data_ptr(), normaliser.data_ptr(), maximum.data_ptr(),
+                                slots.data_ptr(), q_start.data_ptr(), out.data_ptr(), _rows_2d(out, "readout"), len(lengths), tokens,
+                                heads, dim, vdim, MLSTM_SHORT, float(cap), float(q_scale), float(eps), g.data_ptr(), top.data_ptr(),
+                                floor.data_ptr(), start.data_ptr(), own.data_ptr(), before.data_ptr(), norm_own.data_ptr(), chunks,
+                                wave, _stream()), lib)
 
 
 def mlstm_step(rows: torch.Tensor, gates: torch.Tensor, heads: int, dim: int, vdim: int, norm_weight: torch.Tensor,

@@ -25,7 +25,8 @@ bi) / cap) and a log forget gate f = logsigmoid(cap tanh((Wf h + bf) / cap)), a 
     o = S^T q' / (max(|n . q'|, exp(-m')) + 1e-6),   q' = q head_dim^-1/2
 
 each head's o over its root mean square, times a weight of all heads' size, times sigmoid(Wg h); then Wo.  It has kernels of
-its own (``ops.mlstm_step``) and keeps S, n and m per request.
+its own (``ops.mlstm``: single tokens and short portions token by token, longer ones in chunks on the tensor cores) and
+keeps S, n and m per request.
 
 The first two keep, per request, the state S in float32 and the convolution's last taps-1 inputs.  They share their kernels:
 ``ops.gated_prepare`` readies what the recurrence takes, ``ops.gated_rule_scan`` walks the tokens (the state-space
@@ -266,9 +267,9 @@ class MatrixLSTM(Mixer):
         rows = ops.linear(h, self.w_in, None, ops.GEMM_STORE)
         gates = ops.linear(h, self.w_gates, self.b_gates, ops.GEMM_STORE_F32)
         state = cache.state
-        return ops.mlstm_step(rows, gates, self.heads, self.key_dim, self.value_dim, self.norm_w, state["state"],
-                              state["normaliser"], state["maximum"], ctx.slots, ctx.q_start, ctx.num_seqs, self.cap,
-                              self.key_dim ** -0.5, self.eps, out=out)
+        return ops.mlstm(rows, gates, self.heads, self.key_dim, self.value_dim, self.norm_w, state["state"],
+                         state["normaliser"], state["maximum"], ctx.slots, ctx.q_start, ctx.host_q_lens, self.cap,
+                         self.key_dim ** -0.5, self.eps, out=out)
 
     def output_projection(self):
         return self.w_o, None

@@ -130,20 +130,25 @@ def expert(h: np.ndarray, W: Dict[str, np.ndarray], p: str, limit: float) -> np.
     return (g * sigmoid(1.702 * g) * (u + 1.0)) @ W[p + "down"].astype(F).T
 
 
-def route(h: np.ndarray, W: Dict[str, np.ndarray], p: str, top: int, margins: Optional[list] = None):
+def route(h: np.ndarray, W: Dict[str, np.ndarray], p: str, top: int, margins: Optional[list] = None,
+          choice: Optional[np.ndarray] = None):
     """(chosen experts [T, top], their logistic scores [T, top]).  ``margins`` collects, per token, how far the last
-    chosen logit lies above the first one left out."""
+    chosen logit lies above the first one left out.  ``choice`` [T, top]: take these experts instead (another program's
+    choice, whose rounding may have turned a close call); ``margins`` then collects how far its worst expert lies below
+    the best one it left out, as a negative number, or the distance as above where it took the largest."""
     z = h @ W[p + "router"].astype(F).T
-    ids = np.argsort(-z, axis=-1, kind="stable")[:, :top]
+    ids = np.argsort(-z, axis=-1, kind="stable")[:, :top] if choice is None else np.asarray(choice)
     if margins is not None:
-        ordered = -np.sort(-z, axis=-1)
-        margins.append(ordered[:, top - 1] - ordered[:, top] if z.shape[1] > top else np.full(z.shape[0], np.inf))
+        left_out = z.copy()
+        np.put_along_axis(left_out, ids, -np.inf, axis=-1)
+        margins.append(np.take_along_axis(z, ids, axis=-1).min(axis=-1) - left_out.max(axis=-1))
     return ids, sigmoid(np.take_along_axis(z, ids, axis=-1))
 
 
-def moe_ff(h: np.ndarray, W: Dict[str, np.ndarray], p: str, mlp: dict, margins: Optional[list] = None) -> np.ndarray:
+def moe_ff(h: np.ndarray, W: Dict[str, np.ndarray], p: str, mlp: dict, margins: Optional[list] = None,
+           choice: Optional[np.ndarray] = None) -> np.ndarray:
     """The weight multiplies the expert's input."""
-    ids, w = route(h, W, p, mlp["router"]["top"], margins)
+    ids, w = route(h, W, p, mlp["router"]["top"], margins, choice)
     out = np.zeros(h.shape, dtype=F)
     for e in range(mlp["router"]["experts"]):
         for j in range(ids.shape[1]):
@@ -156,9 +161,10 @@ def moe_ff(h: np.ndarray, W: Dict[str, np.ndarray], p: str, mlp: dict, margins: 
 
 
 def forward(config: dict, W: Dict[str, np.ndarray], tokens, streams: Optional[list] = None,
-            margins: Optional[list] = None) -> np.ndarray:
-    """Logits [T, vocab] of one sequence; ``streams`` collects the stream after every layer, ``margins`` every layer's
-    distances from another choice of experts."""
+            margins: Optional[list] = None, choices: Optional[list] = None) -> np.ndarray:
+    """Logits [T, vocab] of one sequence; ``streams`` collects the stream after every layer, ``margins`` every routed layer's
+    distances from another choice of experts; ``choices``: per routed layer, the experts to take (see ``route``)."""
+    choices = iter(choices) if choices is not None else None
     eps, alpha = config["norm"]["eps"], config["postln_alpha"]
     x = W["embed"].astype(F)[np.asarray(tokens)] * (config.get("embedding") or {}).get("scale", 1.0)
     kept: Dict[int, tuple] = {}
@@ -172,7 +178,7 @@ def forward(config: dict, W: Dict[str, np.ndarray], tokens, streams: Optional[li
             raise ValueError(layer["type"])
         x = rms_norm(alpha * x + y, W[p + "norm1"], eps)
         if layer.get("mlp") is not None:
-            x = rms_norm(alpha * x + moe_ff(x, W, p + "mlp.", layer["mlp"], margins), W[p + "norm2"], eps)
+            x = rms_norm(alpha * x + moe_ff(x, W, p + "mlp.", layer["mlp"], margins, next(choices) if choices is not None else None), W[p + "norm2"], eps)
         if streams is not None:
             streams.append(x.copy())
     return rms_norm(x, W["final.norm"], eps) @ W["head"].astype(F).T
