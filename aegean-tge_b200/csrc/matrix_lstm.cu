@@ -29,6 +29,8 @@ namespace {
 constexpr float DENOMINATOR_FLOOR = 1e-6f;
 
 __device__ __forceinline__ float sigmoid_m(float z) { return 1.0f / (1.0f + expf(-z)); }
+// for an output gate whose product is rounded to bfloat16
+__device__ __forceinline__ float sigmoid_fast(float z) { return __fdividef(1.0f, 1.0f + __expf(-z)); }
 __device__ __forceinline__ float log_sigmoid_m(float z) { return fminf(z, 0.0f) - log1pf(expf(-fabsf(z))); }
 __device__ __forceinline__ float soft_cap_m(float z, float cap) { return cap * tanhf(z / cap); }
 
@@ -270,11 +272,11 @@ __device__ __forceinline__ void copies_landed() { asm volatile("cp.async.wait_gr
 __device__ __forceinline__ void copy_rows(__nv_bfloat16* dst, int pitch, const __nv_bfloat16* src, long long ld, int count, int width,
                                           int padded) {
   const int units = padded / 8;
-  for (int e = threadIdx.x; e < CHUNK * units; e += CHUNK_THREADS) {
-    const int r = e / units, u = e - r * units;
-    const bool real = r < count && u * 8 < width;
-    copy16(dst + r * pitch + u * 8, real ? src + (size_t)r * ld + u * 8 : src, real);
-  }
+  for (int r = threadIdx.x >> 4; r < CHUNK; r += CHUNK_THREADS / 16)          // sixteen lanes to a row
+    for (int u = threadIdx.x & 15; u < units; u += 16) {
+      const bool real = r < count && u * 8 < width;
+      copy16(dst + r * pitch + u * 8, real ? src + (size_t)r * ld + u * 8 : src, real);
+    }
 }
 
 constexpr int SCAN_THREADS = 256;
@@ -500,6 +502,10 @@ __global__ void __launch_bounds__(256) mlstm_chunk_carry_kernel(const ChunkParam
 }
 
 constexpr int STATE_ROWS = 32;          // rows of the state before a chunk that lie in shared memory at a time (three parts)
+// The ring of state rows, and after it in the same place the chunk's keys and values.
+__host__ __device__ constexpr int read_ring_elements(int k_pitch, int v_pitch) {
+  return 6 * STATE_ROWS * v_pitch > CHUNK * (k_pitch + v_pitch) ? 6 * STATE_ROWS * v_pitch : CHUNK * (k_pitch + v_pitch);
+}
 
 // The readout of a chunk: what its own earlier tokens and the state before it give, over the denominator, normalised per
 // head, weighted and gated.  Four warps, 16 tokens each.
@@ -512,10 +518,10 @@ __global__ void __launch_bounds__(CHUNK_THREADS) mlstm_chunk_read_kernel(const C
   const int kd = (dim + 15) / 16 * 16, k_pitch = kd + 8;
   constexpr int V_PITCH = VD + 8;
   __nv_bfloat16* qs = reinterpret_cast<__nv_bfloat16*>(chunk_smem);     // [64][k_pitch]
-  __nv_bfloat16* ks = qs + CHUNK * k_pitch;                             // [64][k_pitch]
+  __nv_bfloat16* ss = qs + CHUNK * k_pitch;                             // [2][3][STATE_ROWS][V_PITCH]; once the state is read:
+  __nv_bfloat16* ks = ss;                                               // [64][k_pitch]
   __nv_bfloat16* vs = ks + CHUNK * k_pitch;                             // [64][V_PITCH]
-  __nv_bfloat16* ss = vs + CHUNK * V_PITCH;                             // [2][3][STATE_ROWS][V_PITCH]
-  double* g_s = reinterpret_cast<double*>(ss + 2 * 3 * STATE_ROWS * V_PITCH);    // [64]
+  double* g_s = reinterpret_cast<double*>(ss + read_ring_elements(k_pitch, V_PITCH));    // [64]
   float* n_s = reinterpret_cast<float*>(g_s + CHUNK);                   // [kd]
   float* den_s = n_s + kd;                                              // [64]
   const ChunkPlace at = place_of(p, p.first_chunk + blockIdx.x);
@@ -527,23 +533,23 @@ __global__ void __launch_bounds__(CHUNK_THREADS) mlstm_chunk_read_kernel(const C
   if (at.seq < 0) return;
   const __nv_bfloat16* rows = reinterpret_cast<const __nv_bfloat16*>(p.m.rows) + (size_t)at.first * p.m.ld;
   copy_rows(qs, k_pitch, rows + (size_t)head * dim, p.m.ld, at.count, dim, kd);
-  copy_rows(ks, k_pitch, rows + (size_t)(p.m.heads + head) * dim, p.m.ld, at.count, dim, kd);
-  copy_rows(vs, V_PITCH, rows + (size_t)2 * p.m.heads * dim + (size_t)head * vdim, p.m.ld, at.count, vdim, VD);
   auto fetch_state = [&](int slice) {
     constexpr int UNITS = VD / 8;
     __nv_bfloat16* dst = ss + (slice & 1) * 3 * STATE_ROWS * V_PITCH;
-    for (int e = tid; e < 3 * STATE_ROWS * UNITS; e += CHUNK_THREADS) {
-      const int part = e / (STATE_ROWS * UNITS), rest = e - part * STATE_ROWS * UNITS;
-      const int r = rest / UNITS, u = rest - r * UNITS;
-      const int row = slice * STATE_ROWS + r;
-      const bool real = row < dim && u * 8 < vdim;
-      const __nv_bfloat16* src = p.before + part * plane + unit * entries;
-      copy16(dst + (part * STATE_ROWS + r) * V_PITCH + u * 8, real ? src + (size_t)row * vdim + u * 8 : src, real);
-    }
+    const __nv_bfloat16* src = p.before + unit * entries;
+#pragma unroll
+    for (int part = 0; part < 3; ++part, src += plane)
+#pragma unroll
+      for (int r = tid >> 4; r < STATE_ROWS; r += CHUNK_THREADS / 16) {
+        const int row = slice * STATE_ROWS + r, u = tid & 15;
+        if (u >= UNITS) continue;
+        const bool real = row < dim && u * 8 < vdim;
+        copy16(dst + (part * STATE_ROWS + r) * V_PITCH + u * 8, real ? src + (size_t)row * vdim + u * 8 : src, real);
+      }
     copies_sent();
   };
   const int slices = (kd + STATE_ROWS - 1) / STATE_ROWS;
-  fetch_state(0);                                          // one group with q, k and v
+  fetch_state(0);                                          // one group with q
   if (tid < CHUNK) g_s[tid] = tid < at.count ? p.g[line + tid] : 0.0;
   for (int d = tid; d < kd; d += CHUNK_THREADS) n_s[d] = d < dim ? p.norm_own[unit * dim + d] : 0.0f;
   const double before = top_before(p, at.seq, head, at.first, at.index);
@@ -601,6 +607,10 @@ __global__ void __launch_bounds__(CHUNK_THREADS) mlstm_chunk_read_kernel(const C
     }
     __syncthreads();                                       // the buffer is copied into again two slices on
   }
+  copy_rows(ks, k_pitch, rows + (size_t)(p.m.heads + head) * dim, p.m.ld, at.count, dim, kd);
+  copies_sent();
+  copy_rows(vs, V_PITCH, rows + (size_t)2 * p.m.heads * dim + (size_t)head * vdim, p.m.ld, at.count, vdim, VD);
+  copies_sent();
 #pragma unroll
   for (int n = 0; n < VD / 8; ++n) {
     acc[n][0] *= inter[0]; acc[n][1] *= inter[0];
@@ -612,6 +622,8 @@ __global__ void __launch_bounds__(CHUNK_THREADS) mlstm_chunk_read_kernel(const C
   for (int n = 0; n < CHUNK / 8; ++n)
 #pragma unroll
     for (int e = 0; e < 4; ++e) sc[n][e] = 0.0f;
+  copies_landed<1>();
+  __syncthreads();
   for (int d0 = 0; d0 < kd; d0 += 16) {
     uint32_t a[4];
     ldm4(shared_address(qs + (warp * 16 + (mi & 1) * 8 + (lane & 7)) * k_pitch + d0 + (mi >> 1) * 8), a[0], a[1], a[2], a[3]);
@@ -639,6 +651,8 @@ __global__ void __launch_bounds__(CHUNK_THREADS) mlstm_chunk_read_kernel(const C
         den[i] += w;
       }
   }
+  copies_landed<0>();
+  __syncthreads();
 #pragma unroll
   for (int ksub = 0; ksub < CHUNK / 16; ++ksub) {
     if (ksub > warp) continue;
@@ -692,7 +706,7 @@ __global__ void __launch_bounds__(CHUNK_THREADS) mlstm_chunk_read_kernel(const C
       const float2 gate = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(gate_rows + (size_t)row[i] * p.m.ld + c));
       const float2 w = *reinterpret_cast<const float2*>(p.m.norm_w + (size_t)head * vdim + c);
       *reinterpret_cast<uint32_t*>(out + (size_t)row[i] * p.m.ldo + c) =
-          pack2(acc[n][2 * i] * factor * w.x * sigmoid_m(gate.x), acc[n][2 * i + 1] * factor * w.y * sigmoid_m(gate.y));
+          pack2(acc[n][2 * i] * factor * w.x * sigmoid_fast(gate.x), acc[n][2 * i + 1] * factor * w.y * sigmoid_fast(gate.y));
     }
   }
 }
@@ -705,7 +719,7 @@ template <int VD>
 int launch_chunks(ChunkParams p, int chunks, cudaStream_t stream) {
   const int kd = (p.m.dim + 15) / 16 * 16;
   const size_t write_smem = ((size_t)CHUNK * (VD + 8) + (size_t)3 * CHUNK * (kd + 8)) * 2 + CHUNK * sizeof(float);
-  const size_t read_smem = ((size_t)2 * CHUNK * (kd + 8) + (size_t)CHUNK * (VD + 8) + (size_t)6 * STATE_ROWS * (VD + 8)) * 2 +
+  const size_t read_smem = ((size_t)CHUNK * (kd + 8) + (size_t)read_ring_elements(kd + 8, VD + 8)) * 2 +
                            CHUNK * sizeof(double) + (size_t)(kd + CHUNK) * sizeof(float);
   static size_t configured = 0;
   if (write_smem > configured || read_smem > configured) {

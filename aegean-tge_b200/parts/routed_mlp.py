@@ -223,6 +223,13 @@ class RoutedExperts(FeedForward):
         return h
 
     def forward_f32(self, h: torch.Tensor, ctx: StepContext) -> torch.Tensor:
+        if self.shared is not None:
+            # the feed-forward every token uses writes the rows, the chosen experts add to them
+            complete = getattr(h, "complete", None)
+            h = h if complete is None else complete()
+            out = self.shared.forward_f32(h, ctx)
+            self.add_routed(h, out, ctx)
+            return out
         out = torch.zeros((h.shape[0], self.hidden), dtype=torch.float32, device=h.device)
         self.forward_add(h, out, ctx)
         return out
