@@ -182,13 +182,19 @@ def step_timeline(engine, batch: int, prompt_len: int, prefill: bool, portion: i
     for _ in range(4):
         run()
     torch.cuda.synchronize()
-    with profile(activities=[ProfilerActivity.CUDA]) as prof:
-        run()
-        torch.cuda.synchronize()
+    ops = engine.model.env.ops
+    for _ in range(4):
+        launched = ops.launches
+        with profile(activities=[ProfilerActivity.CUDA]) as prof:
+            run()
+            torch.cuda.synchronize()
+        launched = ops.launches - launched
+        events = [(e.time_range.start, e.time_range.start + e.device_time_total, e.name) for e in prof.events()
+                  if e.device_time_total > 0]
+        if len(events) >= launched:          # the profiler now and then hands over a part of the records only: once more
+            break
     for n in names:
         engine.runner.finish(n)
-    events = [(e.time_range.start, e.time_range.start + e.device_time_total, e.name) for e in prof.events()
-              if e.device_time_total > 0]
     events.sort(key=lambda e: e[1])
     first = min(e[0] for e in events)
     by_name: Dict[str, List[float]] = {}
