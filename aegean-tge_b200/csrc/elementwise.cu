@@ -648,7 +648,7 @@ __global__ void __launch_bounds__(QKN_THREADS) qk_head_norm_kv_store_vec_kernel(
 #pragma unroll
     for (int e = 0; e < 8; ++e) sum = fmaf(f[e], f[e], sum);
     for (int step = lanes >> 1; step > 0; step >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, step);
-    if (!valid) continue;                                  // the shuffles above were the last ones of this round
+    if (!valid) continue;                                  // the shuffles above were the last ones of this pass
     const bool is_q = unit < heads;
     const float* weight = is_q ? q_weight : k_weight;
     uint4 done = raw;
