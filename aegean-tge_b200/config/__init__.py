@@ -13,7 +13,9 @@ from .fesorax import ARCHITECTURE as FESORAX_ARCHITECTURE
 from .fesorax import FesoraxConfig
 from .kokolorn import ARCHITECTURE as KOKOLORN_ARCHITECTURE
 from .kokolorn import KokolornConfig
+from .tazizen import ARCHITECTURE as TAZIZEN_ARCHITECTURE
+from .tazizen import TazizenConfig
 
-__all__ = ["FesoraxConfig", "FESORAX_ARCHITECTURE", "KokolornConfig", "KOKOLORN_ARCHITECTURE", "PuputarConfig", "PUPUTAR_ARCHITECTURE", "LayerSpec", "ModelSpec", "PartSpec", "expected_tensors", "ConfigError",
+__all__ = ["TazizenConfig", "TAZIZEN_ARCHITECTURE", "FesoraxConfig", "FESORAX_ARCHITECTURE", "KokolornConfig", "KOKOLORN_ARCHITECTURE", "PuputarConfig", "PUPUTAR_ARCHITECTURE", "LayerSpec", "ModelSpec", "PartSpec", "expected_tensors", "ConfigError",
            "Qwen2Config", "QWEN2_ARCHITECTURE", "LepizenConfig", "LEPIZEN_ARCHITECTURE", "MozepelConfig", "MOZEPEL_ARCHITECTURE",
            "read_config_json"]

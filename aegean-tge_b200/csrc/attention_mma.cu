@@ -74,6 +74,7 @@ struct AttnParams {
   int keep_first;            // with a window: the first so many positions stay visible (0: none)
   const __nv_bfloat16* gate; // null, or [tokens, heads] logits: a head's output is multiplied by their logistic function
   int gate_stride;
+  int gate_elements;         // the logits are [tokens, heads * DV] instead: one gate per number of a head's output
   float scale_log2;
 };
 
@@ -115,8 +116,30 @@ struct KeyTiles {
 
 // What a head's gate multiplies its output by.
 __device__ __forceinline__ float head_gate(const AttnParams& p, int token, int head) {
-  if (p.gate == nullptr) return 1.0f;
+  if (p.gate == nullptr || p.gate_elements) return 1.0f;
   return 1.0f / (1.0f + __expf(-__bfloat162float(p.gate[(size_t)token * p.gate_stride + head])));
+}
+
+__device__ __forceinline__ float gate_of(float z) { return 1.0f / (1.0f + __expf(-z)); }
+
+// The gates of number `d` of a head's output, of `d` and the one behind it, and of eight from `d` on (gates per element).
+__device__ __forceinline__ float element_gate(const AttnParams& p, int token, int head, int d) {
+  if (!p.gate_elements) return 1.0f;
+  return gate_of(__bfloat162float(p.gate[(size_t)token * p.gate_stride + (size_t)head * DV + d]));
+}
+__device__ __forceinline__ float2 element_gates2(const AttnParams& p, int token, int head, int d) {
+  const float2 z = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(p.gate + (size_t)token * p.gate_stride + (size_t)head * DV + d));
+  return make_float2(gate_of(z.x), gate_of(z.y));
+}
+[[maybe_unused]] __device__ __forceinline__ void element_gates8(const AttnParams& p, int token, int head, int d, float (&g)[8]) {
+  const uint4 raw = *reinterpret_cast<const uint4*>(p.gate + (size_t)token * p.gate_stride + (size_t)head * DV + d);
+  const __nv_bfloat162* two = reinterpret_cast<const __nv_bfloat162*>(&raw);
+#pragma unroll
+  for (int i = 0; i < 4; ++i) {
+    const float2 z = __bfloat1622float2(two[i]);
+    g[2 * i] = gate_of(z.x);
+    g[2 * i + 1] = gate_of(z.y);
+  }
 }
 
 // The denominator `l` (relative to the running maximum `m_log2`, in base-2 units) with the head's sink in it.
@@ -373,8 +396,13 @@ __global__ void __launch_bounds__(NWARPS * 32) attention_mma_kernel(const AttnPa
       __nv_bfloat16* dst = p.out + (size_t)row_token[i] * p.out_stride + (size_t)row_head[i] * DV;
 #pragma unroll
       for (int d = 0; d < DV / 8; ++d) {
+        float2 f = make_float2(inv, inv);
+        if (p.gate_elements) {
+          const float2 g = element_gates2(p, row_token[i], row_head[i], d * 8 + 2 * t4);
+          f = make_float2(inv * g.x, inv * g.y);
+        }
         *reinterpret_cast<uint32_t*>(dst + d * 8 + 2 * t4) =
-            pack_bf16(o_acc[d][2 * i] * inv, o_acc[d][2 * i + 1] * inv);
+            pack_bf16(o_acc[d][2 * i] * f.x, o_acc[d][2 * i + 1] * f.y);
       }
     } else {
       const size_t slot = ((size_t)split * p.total_tokens + row_token[i]) * p.heads + row_head[i];
@@ -585,7 +613,7 @@ __global__ void __launch_bounds__(DEC_WARPS * 32) attention_decode_kernel(const 
     if (p.num_splits == 1) {
       const float l_all = with_sink(p, head, m, l);
       p.out[(size_t)token * p.out_stride + (size_t)head * DV + d] =
-          __float2bfloat16_rn((l_all > 0.0f ? acc / l_all : 0.0f) * head_gate(p, token, head));
+          __float2bfloat16_rn((l_all > 0.0f ? acc / l_all : 0.0f) * head_gate(p, token, head) * element_gate(p, token, head, d));
     } else {
       const size_t slot = ((size_t)split * p.total_tokens + token) * p.heads + head;
       p.partial_o[slot * DV + d] = acc;
@@ -901,7 +929,7 @@ __global__ void __launch_bounds__((4 * GROUPS + 1) * 32) attention_decode_tma_ke
     if (p.num_splits == 1) {
       const float l_all = with_sink(p, head, m, l);
       p.out[(size_t)token * p.out_stride + (size_t)head * HD + d] =
-          __float2bfloat16_rn((l_all > 0.0f ? acc / l_all : 0.0f) * head_gate(p, token, head));
+          __float2bfloat16_rn((l_all > 0.0f ? acc / l_all : 0.0f) * head_gate(p, token, head) * element_gate(p, token, head, d));
     } else {
       const size_t slot = ((size_t)split * p.total_tokens + token) * p.heads + head;
       p.partial_o[slot * HD + d] = acc;
@@ -1173,8 +1201,14 @@ __global__ void __launch_bounds__(PRE_THREADS) attention_prefill_tma_kernel(
       const float inv = (l_all > 0.0f ? 1.0f / l_all : 0.0f) * head_gate(p, row_token[i], row_head[i]);
       __nv_bfloat16* dst = p.out + (size_t)row_token[i] * p.out_stride + (size_t)row_head[i] * HD;
 #pragma unroll
-      for (int d = 0; d < HD / 8; ++d)
-        *reinterpret_cast<uint32_t*>(dst + d * 8 + 2 * t4) = pack_bf16(o_acc[d][2 * i] * inv, o_acc[d][2 * i + 1] * inv);
+      for (int d = 0; d < HD / 8; ++d) {
+        float2 f = make_float2(inv, inv);
+        if (p.gate_elements) {
+          const float2 g = element_gates2(p, row_token[i], row_head[i], d * 8 + 2 * t4);
+          f = make_float2(inv * g.x, inv * g.y);
+        }
+        *reinterpret_cast<uint32_t*>(dst + d * 8 + 2 * t4) = pack_bf16(o_acc[d][2 * i] * f.x, o_acc[d][2 * i + 1] * f.y);
+      }
     } else {
       const size_t slot = ((size_t)split * p.total_tokens + row_token[i]) * p.heads + row_head[i];
       float* dst = p.partial_o + slot * HD;
@@ -1239,13 +1273,14 @@ __global__ void attention_merge_kernel(const float* __restrict__ partial_o, cons
                                        const int* __restrict__ positions, __nv_bfloat16* __restrict__ out,
                                        int out_stride, int total_tokens, int heads, int window, int split_tokens,
                                        int num_splits, int first_token, const float* __restrict__ sink, int keep_first,
-                                       const __nv_bfloat16* __restrict__ gate, int gate_stride) {
+                                       const __nv_bfloat16* __restrict__ gate, int gate_stride, int gate_elements) {
   pdl_trigger();
   const int t = blockIdx.x + first_token, h = blockIdx.y;
   const int pos = positions[t];                                     // given to the step: not the previous kernel's work
   const float sink_log2 = sink != nullptr ? sink[h] * LOG2E : -INFINITY;   // the sink joins the merged denominator once
   pdl_wait();
-  const float factor = gate != nullptr ? 1.0f / (1.0f + __expf(-__bfloat162float(gate[(size_t)t * gate_stride + h]))) : 1.0f;
+  const __nv_bfloat16* gates = gate != nullptr && gate_elements ? gate + (size_t)t * gate_stride + (size_t)h * DV : nullptr;
+  const float factor = gate != nullptr && !gate_elements ? gate_of(__bfloat162float(gate[(size_t)t * gate_stride + h])) : 1.0f;
   const size_t stride = (size_t)total_tokens * heads;               // slots per split
   const size_t slot0 = (size_t)t * heads + h;
   if (num_splits <= HELD) {
@@ -1282,7 +1317,7 @@ __global__ void attention_merge_kernel(const float* __restrict__ partial_o, cons
         acc += scale * o[i];
       }
       if (sink != nullptr) l += exp2f(sink_log2 - m_use);
-      out[(size_t)t * out_stride + (size_t)h * DV + d] = __float2bfloat16_rn(acc * (l > 0.0f ? 1.0f / l : 0.0f) * factor);
+      out[(size_t)t * out_stride + (size_t)h * DV + d] = __float2bfloat16_rn(acc * (l > 0.0f ? 1.0f / l : 0.0f) * (gates != nullptr ? gate_of(__bfloat162float(gates[d])) : factor));
     }
     return;
   }
@@ -1313,7 +1348,8 @@ __global__ void attention_merge_kernel(const float* __restrict__ partial_o, cons
       const size_t slot = (size_t)s * stride + slot0;
       acc += exp2f(partial_ml[slot * 2] - m_use) * partial_o[slot * DV + d];
     }
-    out[(size_t)t * out_stride + (size_t)h * DV + d] = __float2bfloat16_rn(acc * inv);
+    out[(size_t)t * out_stride + (size_t)h * DV + d] =
+        __float2bfloat16_rn(acc * inv * (gates != nullptr ? gate_of(__bfloat162float(gates[d])) : 1.0f));
   }
 }
 
@@ -1325,7 +1361,7 @@ void launch_merge(const AttnParams& p, const int* positions, int first_token, cu
   auto run = [&](auto kernel) {
     tge_launch(kernel, grid, threads, 0, stream, (const float*)p.partial_o, (const float*)p.partial_ml, positions, p.out, p.out_stride,
                p.total_tokens, p.heads, p.window, p.split_tokens, p.num_splits, first_token, p.sink, p.keep_first, p.gate,
-               p.gate_stride);
+               p.gate_stride, p.gate_elements);
   };
   if (p.num_splits <= 16) run(attention_merge_kernel<16>);
   else run(attention_merge_kernel<48>);
@@ -1370,7 +1406,8 @@ static int attention_dispatch(const void* q, int q_stride, const void* k_pages, 
                               int tokens, int max_q_len, int max_ctx_len, void* out, int out_stride, int heads,
                               int kv_heads, float scale, int window, int split_tokens, float* scratch, int* status,
                               int first_token, const float* sink, int leave_states, int v_pitch, const float* dist_bias,
-                              int dist_span, int keep_first, const void* gate, int gate_stride, cudaStream_t stream) {
+                              int dist_span, int keep_first, const void* gate, int gate_stride, int gate_elements,
+                              cudaStream_t stream) {
   TGE_REQUIRE(tokens >= 0 && num_seqs >= 0, "attention_mma: negative sizes");
   TGE_REQUIRE(dist_bias == nullptr || (dist_span > 0 && scale != 0.0f), "attention_mma: a bias by distance needs its span");
   TGE_REQUIRE(heads > 0 && kv_heads > 0 && heads % kv_heads == 0,
@@ -1390,11 +1427,13 @@ static int attention_dispatch(const void* q, int q_stride, const void* k_pages, 
   p.out = (__nv_bfloat16*)out; p.status = status; p.sink = sink;
   p.dist_bias = dist_bias; p.dist_span = dist_span; p.bias_to_raw = dist_bias != nullptr ? 1.0f / scale : 0.0f;
   p.leave_states = leave_states;
-  TGE_REQUIRE(keep_first >= 0 && (gate == nullptr || gate_stride >= heads), "attention_mma: %d kept positions, gate rows of %d for %d heads",
-              keep_first, gate_stride, heads);
+  TGE_REQUIRE(keep_first >= 0 && (gate == nullptr || gate_stride >= heads * (gate_elements ? DV : 1)),
+              "attention_mma: %d kept positions, gate rows of %d for %d heads", keep_first, gate_stride, heads);
+  TGE_REQUIRE(gate == nullptr || !gate_elements || (gate_stride % 8 == 0 && (uintptr_t)gate % 16 == 0),
+              "attention_mma: gates per element start on 16 bytes");
   TGE_REQUIRE(!leave_states || (keep_first == 0 && gate == nullptr), "attention_mma: kept first tokens and gates go without pooled blocks");
   p.keep_first = window > 0 ? keep_first : 0;
-  p.gate = (const __nv_bfloat16*)gate; p.gate_stride = gate_stride;
+  p.gate = (const __nv_bfloat16*)gate; p.gate_stride = gate_stride; p.gate_elements = gate != nullptr && gate_elements;
   if (v_pitch == 0) v_pitch = DV;
   TGE_REQUIRE(v_pitch >= DV && v_pitch % 8 == 0, "attention_mma: a value pitch of %d (values of %d) must be a multiple of 8", v_pitch, DV);
   TGE_REQUIRE(v_pitch == DV || !(TGE_TMA_KERNELS), "attention_mma: values inside the keys' entries are not served at equal sizes");
@@ -1596,7 +1635,7 @@ static int attention_dispatch(const void* q, int q_stride, const void* k_pages, 
 // key n positions back, entry min(n, dist_span - 1) of the head's row; every kernel adds it where it scales its scores.
 // `keep_first` (with a window): the first so many positions stay visible beside the window.  `gate` (bfloat16 [tokens,
 // gate_stride], or null): logits of one gate per token and head; whoever writes a head's output multiplies it by their
-// logistic function.
+// logistic function.  `gate_elements`: one gate per number of a head's output instead, [tokens, heads * DV].
 TGE_API int tge_attention_mma(const void* q, int q_stride, const void* k_pages, const void* v_pages,
                               const int* block_table, int max_pages, int num_pages, int page_size,
                               const int* q_start, const int* start_pos, const int* positions, int num_seqs,
@@ -1604,7 +1643,7 @@ TGE_API int tge_attention_mma(const void* q, int q_stride, const void* k_pages, 
                               int kv_heads, float scale, int window, int split_tokens, float* scratch, int* status,
                               int decode_prefix, int prefix_split_tokens, const float* sink, int leave_states,
                               int v_pitch, const float* dist_bias, int dist_span, int keep_first, const void* gate,
-                              int gate_stride, cudaStream_t stream) {
+                              int gate_stride, int gate_elements, cudaStream_t stream) {
   TGE_REQUIRE(decode_prefix >= 0 && decode_prefix <= num_seqs, "attention_mma: %d leading single tokens of %d sequences",
               decode_prefix, num_seqs);
   TGE_REQUIRE(prefix_split_tokens >= 0 && prefix_split_tokens % BKV == 0,
@@ -1612,16 +1651,16 @@ TGE_API int tge_attention_mma(const void* q, int q_stride, const void* k_pages, 
   if (decode_prefix == 0 || max_q_len <= 1 || decode_prefix == num_seqs || kv_heads <= 0 || heads / kv_heads > 16)
     return attention_dispatch(q, q_stride, k_pages, v_pages, block_table, max_pages, num_pages, page_size, q_start, start_pos,
                               positions, num_seqs, tokens, max_q_len, max_ctx_len, out, out_stride, heads, kv_heads, scale,
-                              window, split_tokens, scratch, status, 0, sink, leave_states, v_pitch, dist_bias, dist_span, keep_first, gate, gate_stride, stream);
+                              window, split_tokens, scratch, status, 0, sink, leave_states, v_pitch, dist_bias, dist_span, keep_first, gate, gate_stride, gate_elements, stream);
   const int first = attention_dispatch(q, q_stride, k_pages, v_pages, block_table, max_pages, num_pages, page_size, q_start,
                                        start_pos, positions, decode_prefix, decode_prefix, 1, max_ctx_len, out, out_stride,
                                        heads, kv_heads, scale, window, prefix_split_tokens, scratch, status, 0, sink, leave_states, v_pitch, dist_bias,
-                                       dist_span, keep_first, gate, gate_stride, stream);
+                                       dist_span, keep_first, gate, gate_stride, gate_elements, stream);
   if (first < 0) return first;
   const int rest = attention_dispatch(q, q_stride, k_pages, v_pages, block_table + (size_t)decode_prefix * max_pages, max_pages,
                                       num_pages, page_size, q_start + decode_prefix, start_pos + decode_prefix, positions,
                                       num_seqs - decode_prefix, tokens, max_q_len, max_ctx_len, out, out_stride, heads,
                                       kv_heads, scale, window, split_tokens, scratch, status, decode_prefix, sink, leave_states, v_pitch, dist_bias,
-                                      dist_span, keep_first, gate, gate_stride, stream);
+                                      dist_span, keep_first, gate, gate_stride, gate_elements, stream);
   return rest < 0 ? rest : first + rest;
 }

@@ -18,14 +18,15 @@
 // `dist_bias` [heads, span] (float32): a learned bias added to the scaled score of the key at distance n, entry
 // min(n, span - 1) of the head's row.  With a window and `keep_first` > 0 the first so many positions stay visible
 // beside the window.  `gate` [tokens, heads] (the run's format): logits of one gate per head; the output is multiplied by
-// their logistic function.
+// their logistic function; with `gate_elements` the logits are [tokens, heads * value_dim], one per number of the output.
 #include "common.cuh"
 
 namespace {
 
 constexpr int MAX_PER_LANE = 8;  // head_dim <= 256
+constexpr int WIDE_PER_LANE = 20; // entries of a latent cache may be up to 640 numbers
 
-template <typename T>
+template <typename T, int PER_LANE>
 __global__ void __launch_bounds__(128) attention_simt_kernel(
     const T* __restrict__ q, int q_stride, const T* __restrict__ k_pages, const T* __restrict__ v_pages,
     const int* __restrict__ block_table, int max_pages, int num_pages, int page_size,
@@ -33,7 +34,7 @@ __global__ void __launch_bounds__(128) attention_simt_kernel(
     int heads, int kv_heads, int head_dim, int value_dim, int v_pitch, const float* __restrict__ sink, float scale, int window,
     int pool, const T* __restrict__ kp_pages, const T* __restrict__ vp_pages, const int* __restrict__ pool_table,
     int pool_max_pages, int pool_num_pages, const float* __restrict__ dist_bias, int dist_span, int keep_first,
-    const T* __restrict__ gate, int gate_stride, int* status) {
+    const T* __restrict__ gate, int gate_stride, int gate_elements, int* status) {
   const int t = blockIdx.x;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int h = blockIdx.y * 4 + warp;
@@ -46,10 +47,10 @@ __global__ void __launch_bounds__(128) attention_simt_kernel(
   const int seq = seq_of_token[t];
   const int* table = block_table + (size_t)seq * max_pages;
 
-  float qv[MAX_PER_LANE], acc[MAX_PER_LANE];
+  float qv[PER_LANE], acc[PER_LANE];
   const T* qrow = q + (size_t)t * q_stride + (size_t)h * head_dim;
 #pragma unroll
-  for (int i = 0; i < MAX_PER_LANE; ++i) {
+  for (int i = 0; i < PER_LANE; ++i) {
     const int d = lane + 32 * i;
     qv[i] = d < head_dim ? to_float<T>(qrow[d]) : 0.0f;
     acc[i] = 0.0f;
@@ -70,7 +71,7 @@ __global__ void __launch_bounds__(128) attention_simt_kernel(
       const T* vrow = vp_pages + (((size_t)page * kv_heads + kvh) * page_size + entry % page_size) * value_dim;
       float dot = 0.0f;
 #pragma unroll
-      for (int i = 0; i < MAX_PER_LANE; ++i) {
+      for (int i = 0; i < PER_LANE; ++i) {
         const int d = lane + 32 * i;
         if (d < head_dim) dot = fmaf(qv[i], to_float<T>(krow[d]), dot);
       }
@@ -81,7 +82,7 @@ __global__ void __launch_bounds__(128) attention_simt_kernel(
       const float p = expf(s - m_new);
       l = l * corr + p;
 #pragma unroll
-      for (int i = 0; i < MAX_PER_LANE; ++i) {
+      for (int i = 0; i < PER_LANE; ++i) {
         const int d = lane + 32 * i;
         if (d < value_dim) acc[i] = fmaf(p, to_float<T>(vrow[d]), acc[i] * corr);
       }
@@ -115,7 +116,7 @@ __global__ void __launch_bounds__(128) attention_simt_kernel(
       const T* vrow = v_pages + vbase + (size_t)slot * v_pitch;
       float dot = 0.0f;
 #pragma unroll
-      for (int i = 0; i < MAX_PER_LANE; ++i) {
+      for (int i = 0; i < PER_LANE; ++i) {
         const int d = lane + 32 * i;
         if (d < head_dim) dot = fmaf(qv[i], to_float<T>(krow[d]), dot);
       }
@@ -127,7 +128,7 @@ __global__ void __launch_bounds__(128) attention_simt_kernel(
       const float p = expf(s - m_new);
       l = l * corr + p;
 #pragma unroll
-      for (int i = 0; i < MAX_PER_LANE; ++i) {
+      for (int i = 0; i < PER_LANE; ++i) {
         const int d = lane + 32 * i;
         if (d < value_dim) acc[i] = fmaf(p, to_float<T>(vrow[d]), acc[i] * corr);
       }
@@ -141,15 +142,19 @@ __global__ void __launch_bounds__(128) attention_simt_kernel(
     const float corr = expf(m - m_new);
     l = l * corr + expf(s - m_new);
 #pragma unroll
-    for (int i = 0; i < MAX_PER_LANE; ++i) acc[i] *= corr;
+    for (int i = 0; i < PER_LANE; ++i) acc[i] *= corr;
   }
   float inv = l > 0.0f ? 1.0f / l : 0.0f;
-  if (gate != nullptr) inv *= 1.0f / (1.0f + expf(-to_float<T>(gate[(size_t)t * gate_stride + h])));
+  if (gate != nullptr && !gate_elements) inv *= 1.0f / (1.0f + expf(-to_float<T>(gate[(size_t)t * gate_stride + h])));
   T* orow = out + (size_t)t * out_stride + (size_t)h * value_dim;
 #pragma unroll
-  for (int i = 0; i < MAX_PER_LANE; ++i) {
+  for (int i = 0; i < PER_LANE; ++i) {
     const int d = lane + 32 * i;
-    if (d < value_dim) orow[d] = from_float<T>(acc[i] * inv);
+    if (d < value_dim) {
+      float v = acc[i] * inv;
+      if (gate_elements) v *= 1.0f / (1.0f + expf(-to_float<T>(gate[(size_t)t * gate_stride + (size_t)h * value_dim + d])));
+      orow[d] = from_float<T>(v);
+    }
   }
 }
 
@@ -248,7 +253,7 @@ TGE_API int tge_attention_simt(const void* q, int q_stride, const void* k_pages,
                                int heads, int kv_heads, int head_dim, int value_dim, const float* sink, float scale,
                                int window, int is_bf16, int pool, const void* kp_pages, const void* vp_pages,
                                const int* pool_table, int pool_max_pages, int pool_num_pages, int v_pitch,
-                               const float* dist_bias, int dist_span, int keep_first, const void* gate, int gate_stride,
+                               const float* dist_bias, int dist_span, int keep_first, const void* gate, int gate_stride, int gate_elements,
                                int* status, cudaStream_t stream) {
   // v_pitch: numbers between the starts of two positions' values in `v_pages` (0: value_dim, values packed).  A cache
   // whose values are the leading part of its keys passes the keys' pages twice and the keys' size here.
@@ -257,14 +262,14 @@ TGE_API int tge_attention_simt(const void* q, int q_stride, const void* k_pages,
   TGE_REQUIRE(pool == 0 || v_pitch == value_dim, "attention: pooled blocks go with packed values");
   TGE_REQUIRE(tokens >= 0 && heads > 0 && kv_heads > 0 && heads % kv_heads == 0,
               "attention: heads %d must be a positive multiple of kv heads %d", heads, kv_heads);
-  TGE_REQUIRE(head_dim > 0 && head_dim <= 32 * MAX_PER_LANE, "attention: head_dim %d outside (0, %d]", head_dim,
-              32 * MAX_PER_LANE);
-  TGE_REQUIRE(value_dim > 0 && value_dim <= 32 * MAX_PER_LANE, "attention: value_dim %d outside (0, %d]", value_dim,
-              32 * MAX_PER_LANE);
+  TGE_REQUIRE(head_dim > 0 && head_dim <= 32 * WIDE_PER_LANE, "attention: head_dim %d outside (0, %d]", head_dim,
+              32 * WIDE_PER_LANE);
+  TGE_REQUIRE(value_dim > 0 && value_dim <= 32 * WIDE_PER_LANE, "attention: value_dim %d outside (0, %d]", value_dim,
+              32 * WIDE_PER_LANE);
   TGE_REQUIRE(page_size > 0 && max_pages > 0 && num_pages > 0, "attention: bad page geometry");
   TGE_REQUIRE(window >= 0 && keep_first >= 0, "attention: a window of %d with %d kept positions", window, keep_first);
   TGE_REQUIRE(pool == 0 || keep_first == 0, "attention: kept first tokens go without pooled blocks");
-  TGE_REQUIRE(gate == nullptr || gate_stride >= heads, "attention: gate rows of %d for %d heads", gate_stride, heads);
+  TGE_REQUIRE(gate == nullptr || gate_stride >= heads * (gate_elements ? value_dim : 1), "attention: gate rows of %d for %d heads", gate_stride, heads);
   if (window == 0) keep_first = 0;
   TGE_REQUIRE(dist_bias == nullptr || dist_span > 0, "attention: a bias by distance needs its span");
   TGE_REQUIRE(pool >= 0 && (pool == 0 || (window > 0 && kp_pages != nullptr && vp_pages != nullptr && pool_table != nullptr &&
@@ -272,18 +277,20 @@ TGE_API int tge_attention_simt(const void* q, int q_stride, const void* k_pages,
               "attention: pooled blocks need a window, their pages and their table");
   if (tokens == 0) return 0;
   dim3 grid(tokens, (heads + 3) / 4);
-  if (is_bf16)
-    attention_simt_kernel<__nv_bfloat16><<<grid, 128, 0, stream>>>(
-        (const __nv_bfloat16*)q, q_stride, (const __nv_bfloat16*)k_pages, (const __nv_bfloat16*)v_pages, block_table,
-        max_pages, num_pages, page_size, positions, seq_of_token, (__nv_bfloat16*)out, out_stride, heads, kv_heads,
-        head_dim, value_dim, v_pitch, sink, scale, window, pool, (const __nv_bfloat16*)kp_pages, (const __nv_bfloat16*)vp_pages,
-        pool_table, pool_max_pages, pool_num_pages, dist_bias, dist_span, keep_first, (const __nv_bfloat16*)gate, gate_stride, status);
-  else
-    attention_simt_kernel<float><<<grid, 128, 0, stream>>>(
-        (const float*)q, q_stride, (const float*)k_pages, (const float*)v_pages, block_table, max_pages, num_pages,
-        page_size, positions, seq_of_token, (float*)out, out_stride, heads, kv_heads, head_dim, value_dim, v_pitch, sink, scale,
-        window, pool, (const float*)kp_pages, (const float*)vp_pages, pool_table, pool_max_pages, pool_num_pages, dist_bias,
-        dist_span, keep_first, (const float*)gate, gate_stride, status);
+  if (gate == nullptr) gate_elements = 0;
+  auto run = [&](auto kernel, auto number) {
+    using T = decltype(number);
+    kernel<<<grid, 128, 0, stream>>>(
+        (const T*)q, q_stride, (const T*)k_pages, (const T*)v_pages, block_table, max_pages, num_pages, page_size, positions,
+        seq_of_token, (T*)out, out_stride, heads, kv_heads, head_dim, value_dim, v_pitch, sink, scale, window, pool,
+        (const T*)kp_pages, (const T*)vp_pages, pool_table, pool_max_pages, pool_num_pages, dist_bias, dist_span, keep_first,
+        (const T*)gate, gate_stride, gate_elements, status);
+  };
+  const bool wide = head_dim > 32 * MAX_PER_LANE || value_dim > 32 * MAX_PER_LANE;
+  if (is_bf16 && wide) run(attention_simt_kernel<__nv_bfloat16, WIDE_PER_LANE>, __nv_bfloat16());
+  else if (is_bf16) run(attention_simt_kernel<__nv_bfloat16, MAX_PER_LANE>, __nv_bfloat16());
+  else if (wide) run(attention_simt_kernel<float, WIDE_PER_LANE>, float());
+  else run(attention_simt_kernel<float, MAX_PER_LANE>, float());
   return tge_launched("attention_simt", 1);
 }
 

@@ -411,11 +411,21 @@ __global__ void __launch_bounds__(THREADS, 2) attention_prefill_tc_kernel(
       if (p.num_splits == 1) {
         uint4* dst = reinterpret_cast<uint4*>(p.out + (size_t)row_token * p.out_stride + (size_t)row_head * HD + c * 32);
 #pragma unroll
-        for (int e = 0; e < 4; ++e)
-          dst[e] = make_uint4(pack_bf16(__uint_as_float(o_bits[e * 8]) * inv, __uint_as_float(o_bits[e * 8 + 1]) * inv),
-                              pack_bf16(__uint_as_float(o_bits[e * 8 + 2]) * inv, __uint_as_float(o_bits[e * 8 + 3]) * inv),
-                              pack_bf16(__uint_as_float(o_bits[e * 8 + 4]) * inv, __uint_as_float(o_bits[e * 8 + 5]) * inv),
-                              pack_bf16(__uint_as_float(o_bits[e * 8 + 6]) * inv, __uint_as_float(o_bits[e * 8 + 7]) * inv));
+        for (int e = 0; e < 4; ++e) {
+          float f[8];
+          if (p.gate_elements) {
+            element_gates8(p, row_token, row_head, c * 32 + e * 8, f);
+#pragma unroll
+            for (int i = 0; i < 8; ++i) f[i] *= inv;
+          } else {
+#pragma unroll
+            for (int i = 0; i < 8; ++i) f[i] = inv;
+          }
+          dst[e] = make_uint4(pack_bf16(__uint_as_float(o_bits[e * 8]) * f[0], __uint_as_float(o_bits[e * 8 + 1]) * f[1]),
+                              pack_bf16(__uint_as_float(o_bits[e * 8 + 2]) * f[2], __uint_as_float(o_bits[e * 8 + 3]) * f[3]),
+                              pack_bf16(__uint_as_float(o_bits[e * 8 + 4]) * f[4], __uint_as_float(o_bits[e * 8 + 5]) * f[5]),
+                              pack_bf16(__uint_as_float(o_bits[e * 8 + 6]) * f[6], __uint_as_float(o_bits[e * 8 + 7]) * f[7]));
+        }
       } else {
         float4* dst = reinterpret_cast<float4*>(p.partial_o + slot * HD + c * 32);
 #pragma unroll

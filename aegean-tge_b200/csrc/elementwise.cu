@@ -8,34 +8,37 @@
 #include "common.cuh"
 
 // ---------------------------------------------------------------------------
-// embedding: x[t, :] = table[ids[t], :] * scale as float32
+// embedding: x[t, c, :] = table[ids[t], :] * scale as float32, for every copy c
 // ---------------------------------------------------------------------------
 template <typename T>
 __global__ void embedding_kernel(const T* __restrict__ table, const int* __restrict__ ids,
-                                 float* __restrict__ out, int hidden, int vocab, float scale, int* status) {
+                                 float* __restrict__ out, int hidden, int copies, int vocab, float scale, int* status) {
   pdl_trigger();
   pdl_wait();
   const int t = blockIdx.x;
   const int id = ids[t];
-  float* dst = out + (size_t)t * hidden;
+  float* dst = out + (size_t)t * copies * hidden;
   if (id < 0 || id >= vocab) {
     if (threadIdx.x == 0) atomicOr(status, TGE_STATUS_BAD_TOKEN);
-    for (int i = threadIdx.x; i < hidden; i += blockDim.x) dst[i] = 0.0f;
+    for (int i = threadIdx.x; i < copies * hidden; i += blockDim.x) dst[i] = 0.0f;
     return;
   }
   const T* src = table + (size_t)id * hidden;
-  for (int i = threadIdx.x; i < hidden; i += blockDim.x) dst[i] = to_float<T>(src[i]) * scale;
+  for (int i = threadIdx.x; i < hidden; i += blockDim.x) {
+    const float v = to_float<T>(src[i]) * scale;
+    for (int c = 0; c < copies; ++c) dst[(size_t)c * hidden + i] = v;
+  }
 }
 
 TGE_API int tge_embedding(const void* table, int is_bf16, const int* ids, float* out, int tokens,
-                          int hidden, int vocab, float scale, int* status, cudaStream_t stream) {
-  TGE_REQUIRE(tokens >= 0 && hidden > 0 && vocab > 0, "embedding: bad sizes tokens=%d hidden=%d vocab=%d",
-              tokens, hidden, vocab);
+                          int hidden, int copies, int vocab, float scale, int* status, cudaStream_t stream) {
+  TGE_REQUIRE(tokens >= 0 && hidden > 0 && copies > 0 && vocab > 0, "embedding: bad sizes tokens=%d hidden=%d copies=%d vocab=%d",
+              tokens, hidden, copies, vocab);
   if (tokens == 0) return 0;
   if (is_bf16)
-    tge_launch(embedding_kernel<__nv_bfloat16>, tokens, 256, 0, stream, (const __nv_bfloat16*)table, ids, out, hidden, vocab, scale, status);
+    tge_launch(embedding_kernel<__nv_bfloat16>, tokens, 256, 0, stream, (const __nv_bfloat16*)table, ids, out, hidden, copies, vocab, scale, status);
   else
-    tge_launch(embedding_kernel<float>, tokens, 256, 0, stream, (const float*)table, ids, out, hidden, vocab, scale, status);
+    tge_launch(embedding_kernel<float>, tokens, 256, 0, stream, (const float*)table, ids, out, hidden, copies, vocab, scale, status);
   return tge_launched("embedding", 1);
 }
 

@@ -1486,6 +1486,20 @@ TGE_API int tge_gemm_tcgen05_add_norm(const void* x, long long ldx, const void* 
   return tge_launched("splitk_add_norm", 2);
 }
 
+// The product of a small batch left as float32 partial sums [*splits_out, M, N] in scratch (at least max(1, k-splits) * M *
+// N floats), for a kernel of the caller's that adds them in their order.  At most 256 tokens; same return codes.
+TGE_API int tge_gemm_tcgen05_partials(const void* x, long long ldx, const void* w, long long ldw, int M, int N, int K,
+                                      float* scratch, long long scratch_floats, int* splits_out, int* status,
+                                      cudaStream_t stream) {
+  TGE_REQUIRE(M >= 0 && N > 0 && K > 0, "gemm partials: bad sizes M=%d N=%d K=%d", M, N, K);
+  TGE_REQUIRE(status != nullptr && splits_out != nullptr, "gemm partials: bad arguments");
+  *splits_out = 0;
+  if (M == 0) return 0;
+  if (M > FUSED_MAX_TOKENS || scratch == nullptr) return TGE_UNSUPPORTED;
+  return launch_product(x, ldx, w, ldw, nullptr, scratch, N, M, N, K, GEMM_STORE_F32, scratch, scratch_floats, 0, 0, true,
+                        status, stream, splits_out);
+}
+
 // The fused q/k/v product of an attention layer for a small batch: qkv = x . w^T + bias, q rotated into
 // `qkv` (bf16 [M, >= heads*head_dim]), k rotated and v copied into their pages.  Same conditions and
 // return codes as tge_gemm_tcgen05_add_norm; N must be (heads + 2 * kv_heads) * head_dim.

@@ -12,8 +12,9 @@
 //                         and the logistic gate (float32).
 //  * head_linear        - a product per head, out[t, n, :] = W_n x[t, n, :] (queries into the latent space, attended
 //                         latents to values), optionally times a gate per head or per element.
-//  * rotate_interleaved - rotation of neighbouring pairs (2i, 2i+1) by position * frequency_i, from cos/sin tables,
-//                         over `rot_dims` numbers of a run from a given place on; the rest is copied.
+//  * rotate_runs        - rotation of neighbouring pairs (2i, 2i+1), or of halves (i, i + rot_dims / 2), by position *
+//                         frequency_i, from cos/sin tables, over `rot_dims` numbers of a run from a given place on; the
+//                         rest is copied.
 //
 // Long prompt portions go another way: many queries meet every key, so it pays to give every head its own keys and
 // values again, [Wuk_n c | kr] and Wuv_n c, in pages of the step's own, and to run ordinary attention with as many
@@ -29,10 +30,16 @@
 
 namespace {
 
-// One number of a run after the rotation of neighbouring pairs; `e` indexes the run, `x` points at its start.
+// One number of a run after its rotation, in neighbouring pairs or (halves) with the number rot_dims / 2 away; `e` indexes
+// the run, `x` points at its start.
 __device__ __forceinline__ float rotated_pair_element(const float* x, int e, int rot_dims, const float* cos_row,
-                                                      const float* sin_row) {
+                                                      const float* sin_row, int halves) {
   if (e >= rot_dims) return x[e];
+  if (halves) {
+    const int half = rot_dims >> 1;
+    return e < half ? fmaf(x[e], cos_row[e], -x[e + half] * sin_row[e])
+                    : fmaf(x[e], cos_row[e - half], x[e - half] * sin_row[e - half]);
+  }
   const int pair = e >> 1;
   const float c = cos_row[pair], s = sin_row[pair];
   return (e & 1) ? fmaf(x[e], c, x[e - 1] * s) : fmaf(x[e], c, -x[e + 1] * s);
@@ -42,7 +49,7 @@ template <typename T>
 __global__ void __launch_bounds__(256) latent_prepare_kernel(
     const float* __restrict__ raw, long long ld_raw, int q_rank, int kv_rank, int rot, int gate_n, int has_kv,
     const float* __restrict__ q_weight, const float* __restrict__ kv_weight, float eps, const float* __restrict__ cos_table,
-    const float* __restrict__ sin_table, int rot_dims, int max_positions, const int* __restrict__ positions,
+    const float* __restrict__ sin_table, int rot_dims, int halves, int max_positions, const int* __restrict__ positions,
     const int* __restrict__ seq_of_token, const int* __restrict__ block_table, int max_pages, int num_pages, int page_size,
     T* __restrict__ pages, T* __restrict__ q_latent, float* __restrict__ gate, int* status) {
   __shared__ float scratch[32];
@@ -79,7 +86,7 @@ __global__ void __launch_bounds__(256) latent_prepare_kernel(
         const float* sin_row = sin_table + (size_t)pos * (rot_dims / 2);
         for (int base = 0; base < rot; base += 256) {
           const int e = base + threadIdx.x;
-          if (e < rot) entry[kv_rank + e] = from_float<T>(rotated_pair_element(kr, e, rot_dims, cos_row, sin_row));
+          if (e < rot) entry[kv_rank + e] = from_float<T>(rotated_pair_element(kr, e, rot_dims, cos_row, sin_row, halves));
         }
       }
     }
@@ -181,10 +188,10 @@ __global__ void __launch_bounds__(256) head_linear_rows_kernel(
 }
 
 template <typename T>
-__global__ void __launch_bounds__(256) rotate_interleaved_kernel(
+__global__ void __launch_bounds__(256) rotate_runs_kernel(
     const T* __restrict__ src, long long src_row, long long src_head, T* __restrict__ dst, long long dst_row,
     long long dst_head, const float* __restrict__ cos_table, const float* __restrict__ sin_table, int rot_dims,
-    int max_positions, const int* __restrict__ positions, int tokens, int heads, int width, int first, int* status) {
+    int max_positions, const int* __restrict__ positions, int tokens, int heads, int width, int first, int halves, int* status) {
   pdl_trigger();
   pdl_wait();
   const long long total = (long long)tokens * heads * width;
@@ -200,21 +207,23 @@ __global__ void __launch_bounds__(256) rotate_interleaved_kernel(
     const T* run = src + (size_t)t * src_row + (size_t)head * src_head;
     float v = to_float<T>(run[e]);
     if (e >= first && e < first + rot_dims) {
-      const int pair = (e - first) >> 1;
-      const float c = cos_table[(size_t)pos * (rot_dims / 2) + pair], s = sin_table[(size_t)pos * (rot_dims / 2) + pair];
-      v = ((e - first) & 1) ? fmaf(v, c, to_float<T>(run[e - 1]) * s) : fmaf(v, c, -to_float<T>(run[e + 1]) * s);
+      const int half = rot_dims >> 1, o = e - first;
+      const int pair = halves ? (o < half ? o : o - half) : o >> 1;
+      const float c = cos_table[(size_t)pos * half + pair], s = sin_table[(size_t)pos * half + pair];
+      if (halves) v = o < half ? fmaf(v, c, -to_float<T>(run[e + half]) * s) : fmaf(v, c, to_float<T>(run[e - half]) * s);
+      else v = (o & 1) ? fmaf(v, c, to_float<T>(run[e - 1]) * s) : fmaf(v, c, -to_float<T>(run[e + 1]) * s);
     }
     dst[(size_t)t * dst_row + (size_t)head * dst_head + e] = from_float<T>(v);
   }
 }
 
-// The same on pairs of bfloat16 (every size, stride and the first rotated place even, rows on 4 bytes): a thread owns
-// one pair, so a rotated pair is read once.
-__global__ void __launch_bounds__(256) rotate_interleaved_pairs_kernel(
+// The same on pairs of bfloat16 (every size, stride and the first rotated place even, rows on 4 bytes; of halves their
+// length even as well): a thread owns two neighbouring numbers, of halves it also reads the two they are rotated with.
+__global__ void __launch_bounds__(256) rotate_runs_pairs_kernel(
     const __nv_bfloat16* __restrict__ src, long long src_row, long long src_head, __nv_bfloat16* __restrict__ dst,
     long long dst_row, long long dst_head, const float* __restrict__ cos_table, const float* __restrict__ sin_table,
     int rot_dims, int max_positions, const int* __restrict__ positions, int tokens, int heads, int width, int first,
-    int* status) {
+    int halves, int* status) {
   pdl_trigger();
   pdl_wait();
   const int half = width >> 1;
@@ -230,8 +239,16 @@ __global__ void __launch_bounds__(256) rotate_interleaved_pairs_kernel(
       atomicOr(status, TGE_STATUS_BAD_ROW);
       continue;
     }
-    float2 v = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(src + (size_t)t * src_row + (size_t)head * src_head + e));
-    if (e >= first && e < first + rot_dims) {
+    const __nv_bfloat16* at = src + (size_t)t * src_row + (size_t)head * src_head + e;
+    float2 v = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(at));
+    if (halves && e >= first && e < first + rot_dims) {
+      const int half = rot_dims >> 1, o = e - first;
+      const bool low = o < half;
+      const size_t entry = (size_t)pos * half + (low ? o : o - half);
+      const float2 w = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(low ? at + half : at - half));
+      const float sx = low ? -sin_table[entry] : sin_table[entry], sy = low ? -sin_table[entry + 1] : sin_table[entry + 1];
+      v = make_float2(fmaf(v.x, cos_table[entry], w.x * sx), fmaf(v.y, cos_table[entry + 1], w.y * sy));
+    } else if (e >= first && e < first + rot_dims) {
       const int pair = (e - first) >> 1;
       const float c = cos_table[(size_t)pos * (rot_dims / 2) + pair], s = sin_table[(size_t)pos * (rot_dims / 2) + pair];
       v = make_float2(fmaf(v.x, c, -v.y * s), fmaf(v.y, c, v.x * s));
@@ -311,7 +328,7 @@ __global__ void __launch_bounds__(256) gate_rows_kernel(T* __restrict__ x, long 
 // cos/sin: float32 [max_positions, rot_dims / 2].  q_latent: run dtype [tokens, q_rank]; gate: float32 [tokens, gate_n].
 TGE_API int tge_latent_prepare(const float* raw, long long ld_raw, int q_rank, int kv_rank, int rot, int gate_n, int has_kv,
                                const float* q_weight, const float* kv_weight, float eps, const float* cos_table,
-                               const float* sin_table, int rot_dims, int max_positions, const int* positions,
+                               const float* sin_table, int rot_dims, int halves, int max_positions, const int* positions,
                                const int* seq_of_token, const int* block_table, int max_pages, int num_pages,
                                int page_size, void* pages, void* q_latent, float* gate, int is_bf16, int tokens,
                                int* status, cudaStream_t stream) {
@@ -325,12 +342,12 @@ TGE_API int tge_latent_prepare(const float* raw, long long ld_raw, int q_rank, i
   if (tokens == 0) return 0;
   if (is_bf16)
     tge_launch(latent_prepare_kernel<__nv_bfloat16>, dim3(tokens), dim3(256), 0, stream, raw, ld_raw, q_rank, kv_rank, rot,
-               gate_n, has_kv, q_weight, kv_weight, eps, cos_table, sin_table, rot_dims, max_positions, positions,
+               gate_n, has_kv, q_weight, kv_weight, eps, cos_table, sin_table, rot_dims, halves, max_positions, positions,
                seq_of_token, block_table, max_pages, num_pages, page_size, (__nv_bfloat16*)pages, (__nv_bfloat16*)q_latent,
                gate, status);
   else
     tge_launch(latent_prepare_kernel<float>, dim3(tokens), dim3(256), 0, stream, raw, ld_raw, q_rank, kv_rank, rot, gate_n,
-               has_kv, q_weight, kv_weight, eps, cos_table, sin_table, rot_dims, max_positions, positions, seq_of_token,
+               has_kv, q_weight, kv_weight, eps, cos_table, sin_table, rot_dims, halves, max_positions, positions, seq_of_token,
                block_table, max_pages, num_pages, page_size, (float*)pages, (float*)q_latent, gate, status);
   return tge_launched("latent_prepare", 1);
 }
@@ -365,34 +382,34 @@ TGE_API int tge_head_linear(const void* x, long long x_row, long long x_head, co
 }
 
 // src / dst: runs of `width` numbers per (token, head), at t * row + n * head (elements), two buffers.  The rotated
-// numbers are those from `first` on; the others are copied.
-TGE_API int tge_rotate_interleaved(const void* src, long long src_row, long long src_head, void* dst, long long dst_row,
+// numbers are the rot_dims from `first` on, in neighbouring pairs or as halves; the others are copied.
+TGE_API int tge_rotate_runs(const void* src, long long src_row, long long src_head, void* dst, long long dst_row,
                                    long long dst_head, const float* cos_table, const float* sin_table, int rot_dims,
                                    int max_positions, const int* positions, int tokens, int heads, int width, int first,
-                                   int is_bf16, int* status, cudaStream_t stream) {
-  TGE_REQUIRE(tokens >= 0 && heads > 0 && width > 0, "rotate_interleaved: bad shape");
+                                   int halves, int is_bf16, int* status, cudaStream_t stream) {
+  TGE_REQUIRE(tokens >= 0 && heads > 0 && width > 0, "rotate_runs: bad shape");
   TGE_REQUIRE(rot_dims >= 0 && rot_dims % 2 == 0 && first >= 0 && first + rot_dims <= width,
-              "rotate_interleaved: %d rotated numbers from %d on of %d", rot_dims, first, width);
-  TGE_REQUIRE(src != dst, "rotate_interleaved: a pair's second number is read after its first is written; give two buffers");
+              "rotate_runs: %d rotated numbers from %d on of %d", rot_dims, first, width);
+  TGE_REQUIRE(src != dst, "rotate_runs: a pair's second number is read after its first is written; give two buffers");
   if (tokens == 0) return 0;
   const long long total = (long long)tokens * heads * width;
   const int blocks = (int)((total + 255) / 256 > 65535 * 16 ? 65535 * 16 : (total + 255) / 256);
-  if (is_bf16 && ((width | first | src_row | src_head | dst_row | dst_head) & 1) == 0 && (((uintptr_t)src | (uintptr_t)dst) & 3) == 0) {
+  if (is_bf16 && ((width | first | src_row | src_head | dst_row | dst_head) & 1) == 0 && !(halves && rot_dims % 4 != 0) && (((uintptr_t)src | (uintptr_t)dst) & 3) == 0) {
     const int pair_blocks = (int)((total / 2 + 255) / 256 > 148 * 16 ? 148 * 16 : (total / 2 + 255) / 256);
-    tge_launch(rotate_interleaved_pairs_kernel, dim3(pair_blocks), dim3(256), 0, stream, (const __nv_bfloat16*)src, src_row,
+    tge_launch(rotate_runs_pairs_kernel, dim3(pair_blocks), dim3(256), 0, stream, (const __nv_bfloat16*)src, src_row,
                src_head, (__nv_bfloat16*)dst, dst_row, dst_head, cos_table, sin_table, rot_dims, max_positions, positions, tokens,
-               heads, width, first, status);
-    return tge_launched("rotate_interleaved", 1);
+               heads, width, first, halves, status);
+    return tge_launched("rotate_runs", 1);
   }
   if (is_bf16)
-    tge_launch(rotate_interleaved_kernel<__nv_bfloat16>, dim3(blocks), dim3(256), 0, stream, (const __nv_bfloat16*)src,
+    tge_launch(rotate_runs_kernel<__nv_bfloat16>, dim3(blocks), dim3(256), 0, stream, (const __nv_bfloat16*)src,
                src_row, src_head, (__nv_bfloat16*)dst, dst_row, dst_head, cos_table, sin_table, rot_dims, max_positions,
-               positions, tokens, heads, width, first, status);
+               positions, tokens, heads, width, first, halves, status);
   else
-    tge_launch(rotate_interleaved_kernel<float>, dim3(blocks), dim3(256), 0, stream, (const float*)src, src_row, src_head,
+    tge_launch(rotate_runs_kernel<float>, dim3(blocks), dim3(256), 0, stream, (const float*)src, src_row, src_head,
                (float*)dst, dst_row, dst_head, cos_table, sin_table, rot_dims, max_positions, positions, tokens, heads, width,
-               first, status);
-  return tge_launched("rotate_interleaved", 1);
+               first, halves, status);
+  return tge_launched("rotate_runs", 1);
 }
 
 // pages: the cache [num_pages, page_size, kv_rank + rot] found through table [seqs, max_pages]; the step's own pages:

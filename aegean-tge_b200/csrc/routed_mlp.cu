@@ -1,8 +1,9 @@
 // Kernels of a routed feed-forward (a mixture of small experts) and of activations that stand alone.
 //
 //  * router_topk      - from float32 router logits: softmax over all outputs or each output's logistic function, the
-//                       choice by score + correction inside the best groups of neighbouring outputs, the chosen
-//                       outputs' plain scores, over their sum or as they are.
+//                       choice by score + correction inside the best groups of neighbouring outputs (a group's value its
+//                       largest such number, or the sum of its two largest), the chosen outputs' plain scores, over their
+//                       sum or as they are, times a constant.
 //  * activation       - relu(z)^2, or the two-parameter form z > 0: softplus(p) z^2 + z/2, else
 //                       (1/2 + softplus(q)) (exp(z) - 1 - z) + z/2, in place on rows of the run dtype.
 //  * expert_up / expert_down_add - few tokens (a decode step): every (token, chosen expert) pair reads its expert's
@@ -47,8 +48,8 @@ __device__ __forceinline__ void warp_argmax(const float* values, int n, int lane
 // kept flags).
 __global__ void __launch_bounds__(128) router_topk_kernel(const float* __restrict__ logits, long long ld,
                                                           const float* __restrict__ correction, int tokens, int outputs,
-                                                          int top, int group_count, int group_keep, int logistic,
-                                                          int over_sum, int* __restrict__ ids,
+                                                          int top, int group_count, int group_keep, int group_pairs,
+                                                          int logistic, int over_sum, float factor, int* __restrict__ ids,
                                                           float* __restrict__ weights) {
   extern __shared__ float router_smem[];
   pdl_trigger();
@@ -65,8 +66,8 @@ __global__ void __launch_bounds__(128) router_topk_kernel(const float* __restric
     for (int i = lane; i < outputs; i += 32) {
       const float s = 1.0f / (1.0f + expf(-z[i]));
       score[i] = s;
-      // the logits order like the scores and do not saturate
-      choice[i] = correction != nullptr ? s + correction[i] : z[i];
+      // the logits order like the scores and do not saturate (sums of two do not order alike)
+      choice[i] = correction != nullptr ? s + correction[i] : (group_pairs ? s : z[i]);
     }
   } else {
     float m = -INFINITY;
@@ -90,9 +91,24 @@ __global__ void __launch_bounds__(128) router_topk_kernel(const float* __restric
   if (group_count > 1 && group_keep < group_count) {
     const int per = outputs / group_count;
     for (int g = 0; g < group_count; ++g) {
-      float best = -INFINITY;
-      for (int i = lane; i < per; i += 32) best = fmaxf(best, choice[g * per + i]);
-      best = warp_max(best);
+      float best = -INFINITY, second = -INFINITY;
+      for (int i = lane; i < per; i += 32) {
+        const float v = choice[g * per + i];
+        second = fmaxf(second, fminf(best, v));
+        best = fmaxf(best, v);
+      }
+      if (group_pairs) {
+        // the two largest of the group, added (a group of one has only the one)
+#pragma unroll
+        for (int offset = 16; offset > 0; offset >>= 1) {
+          const float other = __shfl_xor_sync(0xffffffffu, best, offset), third = __shfl_xor_sync(0xffffffffu, second, offset);
+          second = fmaxf(fminf(best, other), fmaxf(second, third));
+          best = fmaxf(best, other);
+        }
+        if (per > 1) best += second;
+      } else {
+        best = warp_max(best);
+      }
       if (lane == 0) { group_best[g] = best; kept[g] = 0.0f; }
     }
     __syncwarp();
@@ -122,7 +138,7 @@ __global__ void __launch_bounds__(128) router_topk_kernel(const float* __restric
   }
   chosen_sum = over_sum ? chosen_sum + 1e-20f : 1.0f;
   if (lane == 0)
-    for (int n = 0; n < top; ++n) weights[(size_t)t * top + n] = score[ids[(size_t)t * top + n]] / chosen_sum;
+    for (int n = 0; n < top; ++n) weights[(size_t)t * top + n] = score[ids[(size_t)t * top + n]] / chosen_sum * factor;
 }
 
 template <typename T>
@@ -217,6 +233,16 @@ __device__ __forceinline__ float warp_dot<__nv_bfloat16>(const __nv_bfloat16* __
   return warp_sum(acc);
 }
 
+// A gate per token on what a kernel adds to (the output of a feed-forward that every token uses): the logistic function of a
+// float32 logit found at z[token * ld].  Null: none.
+struct RowGate {
+  const float* z;
+  long long ld;
+};
+__device__ __forceinline__ float row_gate(const RowGate& gate, int token) {
+  return gate.z != nullptr ? 1.0f / (1.0f + expf(-gate.z[(size_t)token * gate.ld])) : 1.0f;
+}
+
 // What an expert applies between its matrices: relu(z)^2, or the clamped gate on interleaved (g, u).
 struct ExpertAct {
   int gated;
@@ -260,17 +286,18 @@ __global__ void __launch_bounds__(256) expert_up_kernel(const T* __restrict__ h,
   }
 }
 
-// x[token, n] += sum over the token's choices, in their order, of weight * (w_down[expert][n, :] . inner[pair, :]), or
-// weight * h[token, n] for an identity expert; null weights count as one.
+// x[token, n] <- gate * x[token, n] + sum over the token's choices, in their order, of weight * (w_down[expert][n, :] .
+// inner[pair, :]), or weight * h[token, n] for an identity expert; null weights and a null gate count as one.
 template <typename T>
 __global__ void __launch_bounds__(256) expert_down_add_kernel(const T* __restrict__ inner, const T* __restrict__ w_down,
                                                               const T* __restrict__ h, long long ld_h,
                                                               const int* __restrict__ ids, const float* __restrict__ weights,
                                                               float* __restrict__ x, int top, int experts, int width, int ff,
-                                                              long long down_expert, long long down_row) {
+                                                              long long down_expert, long long down_row, RowGate gate) {
   pdl_trigger();
   pdl_wait();
   const int t = blockIdx.x;
+  const float g = row_gate(gate, t);
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   for (int n = blockIdx.y * 8 + warp; n < width; n += gridDim.y * 8) {
     float acc = 0.0f;
@@ -283,7 +310,7 @@ __global__ void __launch_bounds__(256) expert_down_add_kernel(const T* __restric
       else
         acc = fmaf(weight, to_float<T>(h[(size_t)t * ld_h + n]), acc);
     }
-    if (lane == 0) x[(size_t)t * width + n] += acc;
+    if (lane == 0) x[(size_t)t * width + n] = fmaf(g, x[(size_t)t * width + n], acc);
   }
 }
 
@@ -353,10 +380,12 @@ __global__ void __launch_bounds__(256) expert_gather_kernel(const T* __restrict_
 template <typename T>
 __global__ void __launch_bounds__(256) expert_combine_add_kernel(const float* __restrict__ outputs, const int* __restrict__ place,
                                                                  const float* __restrict__ weights, const T* __restrict__ h,
-                                                                 long long ld_h, float* __restrict__ x, int top, int width) {
+                                                                 long long ld_h, float* __restrict__ x, int top, int width,
+                                                                 RowGate gate) {
   pdl_trigger();
   pdl_wait();
   const int t = blockIdx.x;
+  const float g = row_gate(gate, t);
   for (int n = blockIdx.y * blockDim.x + threadIdx.x; n < width; n += gridDim.y * blockDim.x) {
     float acc = 0.0f;
     for (int k = 0; k < top; ++k) {
@@ -365,7 +394,7 @@ __global__ void __launch_bounds__(256) expert_combine_add_kernel(const float* __
       const float v = row >= 0 ? outputs[(size_t)row * width + n] : to_float<T>(h[(size_t)t * ld_h + n]);
       acc = fmaf(weights != nullptr ? weights[pair] : 1.0f, v, acc);
     }
-    x[(size_t)t * width + n] += acc;
+    x[(size_t)t * width + n] = fmaf(g, x[(size_t)t * width + n], acc);
   }
 }
 
@@ -409,22 +438,32 @@ __global__ void __launch_bounds__(256) expert_dense_weigh_kernel(T* __restrict__
 
 // The dense path of gated experts: z [tokens, experts * 2 ff] (interleaved gate and up of every expert) -> out [tokens,
 // experts * ff], a chosen expert's activated values and zeros elsewhere.  `weigh_input`: the weight multiplies (g, u), else
-// the activated value.
+// the activated value.  `shared_ff` > 0: behind the experts' columns lie those of a feed-forward that every token uses
+// (2 shared_ff in z, shared_ff in out), its activated values times the token's gate; blocks with blockIdx.y == experts do it.
 template <typename T>
 __global__ void __launch_bounds__(256) expert_dense_gate_kernel(const T* __restrict__ z, const int* __restrict__ ids,
                                                                 const float* __restrict__ weights, T* __restrict__ out, int top,
-                                                                int experts, int ff, int weigh_input, ExpertAct act) {
+                                                                int experts, int expert_ff, int weigh_input, ExpertAct act,
+                                                                int shared_ff, RowGate gate) {
   pdl_trigger();
   pdl_wait();
   const int t = blockIdx.x, e = blockIdx.y;
   float w = 0.0f;
   bool chosen = false;
-  for (int k = 0; k < top; ++k)
-    if (ids[t * top + k] == e) { w = weights[t * top + k]; chosen = true; }
-  const T* src = z + ((size_t)t * experts + e) * 2 * ff;
-  T* dst = out + ((size_t)t * experts + e) * ff;
+  if (e == experts) {
+    w = row_gate(gate, t);
+    chosen = true;
+    weigh_input = 0;
+  } else {
+    for (int k = 0; k < top; ++k)
+      if (ids[t * top + k] == e) { w = weights[t * top + k]; chosen = true; }
+  }
+  const size_t row = (size_t)experts * expert_ff + shared_ff;
+  const int ff = e == experts ? shared_ff : expert_ff;
+  const T* src = z + ((size_t)t * row + (size_t)e * expert_ff) * 2;
+  T* dst = out + (size_t)t * row + (size_t)e * expert_ff;
   const float in = weigh_input ? w : 1.0f, after = weigh_input ? 1.0f : w;
-  if (sizeof(T) == 2 && ff % 4 == 0) {
+  if (sizeof(T) == 2 && expert_ff % 4 == 0 && shared_ff % 4 == 0) {
     // four values at a time: 16 bytes in, 8 bytes out (the buffers are the wrapper's own, so aligned)
     for (int j = threadIdx.x; j < ff / 4; j += blockDim.x) {
       uint2 packed = make_uint2(0u, 0u);
@@ -452,8 +491,8 @@ __global__ void __launch_bounds__(256) expert_dense_gate_kernel(const T* __restr
 
 // logits float32 [tokens, ld]; correction float32 [outputs] or null; ids int32 [tokens, top]; weights float32 [tokens, top].
 TGE_API int tge_router_topk(const float* logits, long long ld, const float* correction, int tokens, int outputs, int top,
-                            int group_count, int group_keep, int logistic, int over_sum, int* ids, float* weights,
-                            cudaStream_t stream) {
+                            int group_count, int group_keep, int group_pairs, int logistic, int over_sum, float factor,
+                            int* ids, float* weights, cudaStream_t stream) {
   TGE_REQUIRE(tokens >= 0 && outputs > 0 && outputs <= 1024, "router_topk: 1 to 1024 outputs, not %d", outputs);
   TGE_REQUIRE(top > 0 && top <= outputs, "router_topk: %d choices of %d outputs", top, outputs);
   TGE_REQUIRE(group_count > 0 && outputs % group_count == 0 && group_keep > 0 && group_keep <= group_count,
@@ -469,7 +508,7 @@ TGE_API int tge_router_topk(const float* logits, long long ld, const float* corr
     }
   }
   tge_launch(router_topk_kernel, dim3((tokens + 3) / 4), dim3(128), smem, stream, logits, ld, correction, tokens, outputs, top,
-             group_count, group_keep, logistic, over_sum, ids, weights);
+             group_count, group_keep, group_pairs, logistic, over_sum, factor, ids, weights);
   return tge_launched("router_topk", 1);
 }
 
@@ -500,11 +539,13 @@ TGE_API int tge_activation(void* rows, long long ld, int count, int width, int k
 TGE_API int tge_experts_direct(const void* h, long long ld_h, const void* w_up, const void* w_down, long long down_expert,
                                long long down_row, const int* ids, const float* weights, void* inner, float* x, int tokens,
                                int top, int experts, int width, int ff, int weigh_input, int gated, float limit,
-                               float alpha, float offset, int is_bf16, cudaStream_t stream) {
+                               float alpha, float offset, const float* x_gate, long long ld_gate, int is_bf16,
+                               cudaStream_t stream) {
   TGE_REQUIRE(tokens >= 0 && top > 0 && experts >= 0 && width > 0 && ff > 0, "experts: bad shape");
   TGE_REQUIRE(!gated || limit > 0.0f, "experts: the gate's limit must be positive");
   if (tokens == 0) return 0;
   const ExpertAct act{gated, limit, alpha, offset};
+  const RowGate gate{x_gate, ld_gate};
   const float* in_weights = weigh_input ? weights : nullptr;
   if (weigh_input) weights = nullptr;
   const int up_y = (ff + 7) / 8 < 64 ? (ff + 7) / 8 : 64;
@@ -514,12 +555,13 @@ TGE_API int tge_experts_direct(const void* h, long long ld_h, const void* w_up, 
                (const __nv_bfloat16*)w_up, ids, in_weights, (__nv_bfloat16*)inner, top, experts, width, ff, act);
     tge_launch(expert_down_add_kernel<__nv_bfloat16>, dim3(tokens, down_y), dim3(256), 0, stream, (const __nv_bfloat16*)inner,
                (const __nv_bfloat16*)w_down, (const __nv_bfloat16*)h, ld_h, ids, weights, x, top, experts, width, ff, down_expert,
-               down_row);
+               down_row, gate);
   } else {
     tge_launch(expert_up_kernel<float>, dim3(tokens * top, up_y), dim3(256), 0, stream, (const float*)h, ld_h,
                (const float*)w_up, ids, in_weights, (float*)inner, top, experts, width, ff, act);
     tge_launch(expert_down_add_kernel<float>, dim3(tokens, down_y), dim3(256), 0, stream, (const float*)inner,
-               (const float*)w_down, (const float*)h, ld_h, ids, weights, x, top, experts, width, ff, down_expert, down_row);
+               (const float*)w_down, (const float*)h, ld_h, ids, weights, x, top, experts, width, ff, down_expert, down_row,
+               gate);
   }
   return tge_launched("experts_direct", 2);
 }
@@ -543,16 +585,18 @@ TGE_API int tge_experts_group(const void* h, long long ld_h, const int* ids, con
 
 // The grouped path, second half: outputs float32 [tokens * top, width] in grouped order.
 TGE_API int tge_experts_combine_add(const float* outputs, const int* place, const float* weights, const void* h, long long ld_h,
-                                    float* x, int tokens, int top, int width, int is_bf16, cudaStream_t stream) {
+                                    float* x, int tokens, int top, int width, const float* x_gate, long long ld_gate,
+                                    int is_bf16, cudaStream_t stream) {
   TGE_REQUIRE(tokens >= 0 && top > 0 && width > 0, "experts: bad shape");
   if (tokens == 0) return 0;
+  const RowGate gate{x_gate, ld_gate};
   const int chunks = (width + 1023) / 1024;
   if (is_bf16)
     tge_launch(expert_combine_add_kernel<__nv_bfloat16>, dim3(tokens, chunks), dim3(256), 0, stream, outputs, place, weights,
-               (const __nv_bfloat16*)h, ld_h, x, top, width);
+               (const __nv_bfloat16*)h, ld_h, x, top, width, gate);
   else
     tge_launch(expert_combine_add_kernel<float>, dim3(tokens, chunks), dim3(256), 0, stream, outputs, place, weights,
-               (const float*)h, ld_h, x, top, width);
+               (const float*)h, ld_h, x, top, width, gate);
   return tge_launched("experts_combine_add", 1);
 }
 
@@ -570,19 +614,22 @@ TGE_API int tge_experts_dense_weigh(void* z, const int* ids, const float* weight
   return tge_launched("experts_dense_weigh", 1);
 }
 
-// The dense path of gated experts: z run dtype [tokens, experts * 2 ff] -> out [tokens, experts * ff] (see the kernel).
+// The dense path of gated experts: z run dtype [tokens, 2 (experts * ff + shared_ff)] -> out [tokens, experts * ff +
+// shared_ff] (see the kernel).
 TGE_API int tge_experts_dense_gate(const void* z, const int* ids, const float* weights, void* out, int tokens, int top,
-                                   int experts, int ff, int weigh_input, float limit, float alpha, float offset, int is_bf16,
-                                   cudaStream_t stream) {
-  TGE_REQUIRE(tokens >= 0 && top > 0 && experts > 0 && experts < 65535 && ff > 0 && limit > 0.0f, "experts: bad shape");
+                                   int experts, int ff, int weigh_input, float limit, float alpha, float offset, int shared_ff,
+                                   const float* shared_gate, long long ld_gate, int is_bf16, cudaStream_t stream) {
+  TGE_REQUIRE(tokens >= 0 && top > 0 && experts > 0 && experts < 65535 && ff > 0 && shared_ff >= 0 && limit > 0.0f, "experts: bad shape");
   TGE_REQUIRE(((uintptr_t)z & 15) == 0 && ((uintptr_t)out & 15) == 0, "experts: rows must start on 16 bytes");
   if (tokens == 0) return 0;
   const ExpertAct act{1, limit, alpha, offset};
+  const RowGate gate{shared_gate, ld_gate};
+  const dim3 grid(tokens, experts + (shared_ff > 0 ? 1 : 0));
   if (is_bf16)
-    tge_launch(expert_dense_gate_kernel<__nv_bfloat16>, dim3(tokens, experts), dim3(256), 0, stream, (const __nv_bfloat16*)z, ids,
-               weights, (__nv_bfloat16*)out, top, experts, ff, weigh_input, act);
+    tge_launch(expert_dense_gate_kernel<__nv_bfloat16>, grid, dim3(256), 0, stream, (const __nv_bfloat16*)z, ids,
+               weights, (__nv_bfloat16*)out, top, experts, ff, weigh_input, act, shared_ff, gate);
   else
-    tge_launch(expert_dense_gate_kernel<float>, dim3(tokens, experts), dim3(256), 0, stream, (const float*)z, ids, weights,
-               (float*)out, top, experts, ff, weigh_input, act);
+    tge_launch(expert_dense_gate_kernel<float>, grid, dim3(256), 0, stream, (const float*)z, ids, weights,
+               (float*)out, top, experts, ff, weigh_input, act, shared_ff, gate);
   return tge_launched("experts_dense_gate", 1);
 }

@@ -721,7 +721,8 @@ __global__ void __launch_bounds__(128) gated_norm_kernel(const float* __restrict
 // After the q/k/v product: the short convolution over time, the per-head norm of q and k, their rotation, and the
 // store.  One warp per (token, head of q, k or v).  `raw` holds the projections of this step's tokens [T, q | k | v];
 // inputs from before the portion come from the request's convolution state [slots, taps-1, channels] (oldest first),
-// which is zero for a request that starts.  q goes to `q_out`, k and v into their pages.
+// which is zero for a request that starts.  q goes to `q_out`, k and v into their pages.  `norm_last`: q and k are
+// normalised after their rotation instead of before it (weights may be null: none).
 constexpr int CNR_PER_LANE = 8;    // head sizes up to 256
 constexpr int MAX_TAPS = 16;
 
@@ -733,7 +734,7 @@ __global__ void __launch_bounds__(128) conv_norm_rope_store_kernel(
     const float* __restrict__ cos_table, const float* __restrict__ sin_table, int table_positions, int rotary,
     const int* __restrict__ positions, const int* __restrict__ seq_of_token, const int* __restrict__ block_table,
     int max_pages, T* __restrict__ k_pages, T* __restrict__ v_pages, int num_pages, int page_size,
-    T* __restrict__ q_out, long long ld_q, int heads, int kv_heads, int dim, int vdim, int store, int* status) {
+    T* __restrict__ q_out, long long ld_q, int heads, int kv_heads, int dim, int vdim, int store, int norm_last, int* status) {
   pdl_trigger();
   pdl_wait();
   __shared__ float staged[4][32 * CNR_PER_LANE];
@@ -773,7 +774,7 @@ __global__ void __launch_bounds__(128) conv_norm_rope_store_kernel(
     sum = fmaf(value, value, sum);
   }
   const float* norm_w = kind == 0 ? q_norm : (kind == 1 ? k_norm : nullptr);
-  if (norm_w != nullptr) {
+  if (norm_w != nullptr && !norm_last) {
     sum = warp_sum(sum);
     const float scale = 1.0f / sqrtf(sum / (float)size + eps);
 #pragma unroll
@@ -802,6 +803,17 @@ __global__ void __launch_bounds__(128) conv_norm_rope_store_kernel(
         const float other = staged[warp][e < half ? e + half : e - half];
         y[i] = e < half ? y[i] * cs - other * sn : y[i] * cs + other * sn;
       }
+    }
+  }
+  if (norm_last && kind != 2) {
+    float square = 0.0f;                                  // the rotation's tables may scale what they turn
+#pragma unroll
+    for (int i = 0; i < CNR_PER_LANE; ++i) square = fmaf(y[i], y[i], square);
+    const float scale = 1.0f / sqrtf(warp_sum(square) / (float)size + eps);
+#pragma unroll
+    for (int i = 0; i < CNR_PER_LANE; ++i) {
+      const int e = lane + 32 * i;
+      if (e < size) y[i] = y[i] * scale * (norm_w != nullptr ? norm_w[e] : 1.0f);
     }
   }
   if (kind == 0) {
@@ -1069,7 +1081,8 @@ TGE_API int tge_conv_norm_rope_store(const void* raw, int is_bf16, long long ld,
                                      int table_positions, int rotary, const int* positions, const int* seq_of_token,
                                      const int* block_table, int max_pages, void* k_pages, void* v_pages, int num_pages,
                                      int page_size, void* q_out, long long ld_q, int tokens, int num_seqs, int heads,
-                                     int kv_heads, int dim, int vdim, int store, int* status, cudaStream_t stream) {
+                                     int kv_heads, int dim, int vdim, int store, int norm_last, int* status,
+                                     cudaStream_t stream) {
   TGE_REQUIRE(heads > 0 && kv_heads > 0 && dim > 0 && vdim > 0 && dim <= 32 * CNR_PER_LANE && vdim <= 32 * CNR_PER_LANE,
               "conv_norm_rope_store: head sizes %d and %d outside (0, %d]", dim, vdim, 32 * CNR_PER_LANE);
   TGE_REQUIRE(taps >= 0 && taps <= MAX_TAPS, "conv_norm_rope_store: %d taps (at most %d)", taps, MAX_TAPS);
@@ -1088,12 +1101,12 @@ TGE_API int tge_conv_norm_rope_store(const void* raw, int is_bf16, long long ld,
     tge_launch(conv_norm_rope_store_kernel<__nv_bfloat16>, grid, dim3(128), 0, stream,
         (const __nv_bfloat16*)raw, ld, conv_w, taps, conv_state, slots, q_start, q_norm, k_norm, eps, cos_table, sin_table,
         table_positions, rotary, positions, seq_of_token, block_table, max_pages, (__nv_bfloat16*)k_pages,
-        (__nv_bfloat16*)v_pages, num_pages, page_size, (__nv_bfloat16*)q_out, ld_q, heads, kv_heads, dim, vdim, store, status);
+        (__nv_bfloat16*)v_pages, num_pages, page_size, (__nv_bfloat16*)q_out, ld_q, heads, kv_heads, dim, vdim, store, norm_last, status);
   } else {
     tge_launch(conv_norm_rope_store_kernel<float>, grid, dim3(128), 0, stream,
         (const float*)raw, ld, conv_w, taps, conv_state, slots, q_start, q_norm, k_norm, eps, cos_table, sin_table,
         table_positions, rotary, positions, seq_of_token, block_table, max_pages, (float*)k_pages, (float*)v_pages,
-        num_pages, page_size, (float*)q_out, ld_q, heads, kv_heads, dim, vdim, store, status);
+        num_pages, page_size, (float*)q_out, ld_q, heads, kv_heads, dim, vdim, store, norm_last, status);
   }
   if (int rc = tge_check_launch("conv_norm_rope_store")) return rc;
   if (taps > 1) {

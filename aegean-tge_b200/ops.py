@@ -56,7 +56,7 @@ def core() -> ctypes.CDLL:
         path = _build.build_core()
         lib = ctypes.CDLL(path)
         lib.tge_last_error.restype = ctypes.c_char_p
-        _declare(lib, "tge_embedding", [_c_ptr, _c_int, _c_ptr, _c_ptr, _c_int, _c_int, _c_int, _c_float, _c_ptr, _c_ptr])
+        _declare(lib, "tge_embedding", [_c_ptr, _c_int, _c_ptr, _c_ptr, _c_int, _c_int, _c_int, _c_int, _c_float, _c_ptr, _c_ptr])
         _declare(lib, "tge_rmsnorm", [_c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_int, _c_int, _c_int, _c_float,
                                       _c_ptr, _c_ptr])
         _declare(lib, "tge_add_to_stream", [_c_ptr, _c_ptr, _c_int, _c_ll, _c_float, _c_ptr])
@@ -93,7 +93,7 @@ def core() -> ctypes.CDLL:
         _declare(lib, "tge_attention_simt", [_c_ptr, _c_int, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_int, _c_int, _c_ptr,
                                              _c_ptr, _c_ptr, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_ptr,
                                              _c_float, _c_int, _c_int, _c_int, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_int,
-                                             _c_int, _c_ptr, _c_int, _c_int, _c_ptr, _c_int, _c_ptr, _c_ptr])
+                                             _c_int, _c_ptr, _c_int, _c_int, _c_ptr, _c_int, _c_int, _c_ptr, _c_ptr])
         _declare(lib, "tge_attention_pooled_merge", [_c_ptr, _c_int, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_int, _c_int, _c_ptr,
                                                      _c_ptr, _c_ptr, _c_ptr, _c_int, _c_int, _c_ptr, _c_int, _c_int, _c_int,
                                                      _c_int, _c_int, _c_int, _c_float, _c_int, _c_int, _c_ptr, _c_int, _c_ptr,
@@ -103,27 +103,34 @@ def core() -> ctypes.CDLL:
         _declare(lib, "tge_token_shift", [_c_ptr, _c_int, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_ptr, _c_ptr, _c_ptr, _c_ptr,
                                           _c_int, _c_int, _c_int, _c_int, _c_ptr, _c_ptr])
         _declare(lib, "tge_latent_prepare", [_c_ptr, _c_ll, _c_int, _c_int, _c_int, _c_int, _c_int, _c_ptr, _c_ptr, _c_float,
-                                             _c_ptr, _c_ptr, _c_int, _c_int, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_int, _c_int,
-                                             _c_ptr, _c_ptr, _c_ptr, _c_int, _c_int, _c_ptr, _c_ptr])
+                                             _c_ptr, _c_ptr, _c_int, _c_int, _c_int, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_int,
+                                             _c_int, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_int, _c_ptr, _c_ptr])
         _declare(lib, "tge_head_linear", [_c_ptr, _c_ll, _c_ll, _c_ptr, _c_ptr, _c_ll, _c_ll, _c_ptr, _c_int, _c_ll, _c_int,
                                           _c_int, _c_int, _c_int, _c_int, _c_ptr])
-        _declare(lib, "tge_rotate_interleaved", [_c_ptr, _c_ll, _c_ll, _c_ptr, _c_ll, _c_ll, _c_ptr, _c_ptr, _c_int, _c_int,
-                                                 _c_ptr, _c_int, _c_int, _c_int, _c_int, _c_int, _c_ptr, _c_ptr])
+        _declare(lib, "tge_rotate_runs", [_c_ptr, _c_ll, _c_ll, _c_ptr, _c_ll, _c_ll, _c_ptr, _c_ptr, _c_int, _c_int,
+                                          _c_ptr, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_ptr, _c_ptr])
         _declare(lib, "tge_latent_gather", [_c_ptr, _c_ptr, _c_int, _c_int, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_int, _c_int,
                                             _c_int, _c_int, _c_int, _c_ptr, _c_ptr, _c_int, _c_ptr, _c_ptr])
         _declare(lib, "tge_latent_scatter", [_c_ptr, _c_ll, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_ptr, _c_ptr,
                                              _c_int, _c_ptr])
         _declare(lib, "tge_gate_rows", [_c_ptr, _c_ll, _c_ptr, _c_ll, _c_int, _c_int, _c_int, _c_int, _c_int, _c_ptr])
-        _declare(lib, "tge_router_topk", [_c_ptr, _c_ll, _c_ptr, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int,
-                                          _c_ptr, _c_ptr, _c_ptr])
+        _declare(lib, "tge_router_topk", [_c_ptr, _c_ll, _c_ptr, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int,
+                                          _c_float, _c_ptr, _c_ptr, _c_ptr])
         _declare(lib, "tge_activation", [_c_ptr, _c_ll, _c_int, _c_int, _c_int, _c_ptr, _c_int, _c_ptr])
         _declare(lib, "tge_experts_direct", [_c_ptr, _c_ll, _c_ptr, _c_ptr, _c_ll, _c_ll, _c_ptr, _c_ptr, _c_ptr, _c_ptr,
                                              _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_float, _c_float,
-                                             _c_float, _c_int, _c_ptr])
+                                             _c_float, _c_ptr, _c_ll, _c_int, _c_ptr])
         _declare(lib, "tge_experts_dense_weigh", [_c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_ll, _c_ptr, _c_int, _c_int, _c_int,
                                                   _c_int, _c_int, _c_int, _c_ptr])
         _declare(lib, "tge_experts_dense_gate", [_c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_int, _c_int, _c_int, _c_int,
-                                                 _c_float, _c_float, _c_float, _c_int, _c_ptr])
+                                                 _c_float, _c_float, _c_float, _c_int, _c_ptr, _c_ll, _c_int, _c_ptr])
+        _declare(lib, "tge_streams_rows", [_c_ptr, _c_int, _c_int, _c_int, _c_int, _c_ptr, _c_ll, _c_ptr, _c_ptr, _c_ptr, _c_ptr,
+                                           _c_float, _c_ptr, _c_ptr, _c_int, _c_ptr, _c_ptr])
+        _declare(lib, "tge_streams_slices", [_c_int])
+        _declare(lib, "tge_streams_update_defer", [_c_ptr, _c_int, _c_int, _c_int, _c_ptr, _c_int, _c_ptr, _c_ptr, _c_ptr,
+                                                   _c_ptr, _c_ptr, _c_ptr, _c_ptr])
+        _declare(lib, "tge_gemm_tcgen05_partials", [_c_ptr, _c_ll, _c_ptr, _c_ll, _c_int, _c_int, _c_int, _c_ptr, _c_ll,
+                                                    ctypes.POINTER(_c_int), _c_ptr, _c_ptr])
         _declare(lib, "tge_mlstm_step", [_c_ptr, _c_int, _c_ll, _c_ptr, _c_ll, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_ptr,
                                          _c_ptr, _c_ll, _c_int, _c_int, _c_int, _c_int, _c_int, _c_float, _c_float, _c_float,
                                          _c_ptr])
@@ -135,7 +142,7 @@ def core() -> ctypes.CDLL:
         _declare(lib, "tge_experts_group", [_c_ptr, _c_ll, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_int, _c_int, _c_int,
                                             _c_int, _c_ptr])
         _declare(lib, "tge_experts_combine_add", [_c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_ll, _c_ptr, _c_int, _c_int, _c_int,
-                                                  _c_int, _c_ptr])
+                                                  _c_ptr, _c_ll, _c_int, _c_ptr])
         _declare(lib, "tge_to_run_dtype", [_c_ptr, _c_ptr, _c_int, _c_ll, _c_ptr])
         _declare(lib, "tge_scale_add_norm", [_c_ptr, _c_ptr, _c_ll, _c_ptr, _c_ptr, _c_int, _c_int, _c_int, _c_float,
                                              _c_float, _c_ptr])
@@ -147,7 +154,7 @@ def core() -> ctypes.CDLL:
         _declare(lib, "tge_conv_norm_rope_store", [_c_ptr, _c_int, _c_ll, _c_ptr, _c_int, _c_ptr, _c_ptr, _c_ptr, _c_ptr,
                                                    _c_ptr, _c_float, _c_ptr, _c_ptr, _c_int, _c_int, _c_ptr, _c_ptr,
                                                    _c_ptr, _c_int, _c_ptr, _c_ptr, _c_int, _c_int, _c_ptr, _c_ll, _c_int,
-                                                   _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_ptr, _c_ptr])
+                                                   _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_ptr, _c_ptr])
         _declare(lib, "tge_pool_kv", [_c_ptr, _c_ptr, _c_int, _c_ptr, _c_int, _c_int, _c_ptr, _c_ptr, _c_ptr, _c_int,
                                       _c_int, _c_int, _c_ptr, _c_ptr, _c_int, _c_int, _c_int, _c_int, _c_int, _c_ptr,
                                       _c_ptr])
@@ -191,7 +198,7 @@ def attention_lib(head_dim: int, value_dim: int = 0) -> ctypes.CDLL:
         _declare(lib, "tge_attention_mma", [_c_ptr, _c_int, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_int, _c_int, _c_ptr,
                                             _c_ptr, _c_ptr, _c_int, _c_int, _c_int, _c_int, _c_ptr, _c_int, _c_int,
                                             _c_int, _c_float, _c_int, _c_int, _c_ptr, _c_ptr, _c_int, _c_int, _c_ptr,
-                                            _c_int, _c_int, _c_ptr, _c_int, _c_int, _c_ptr, _c_int, _c_ptr])
+                                            _c_int, _c_int, _c_ptr, _c_int, _c_int, _c_ptr, _c_int, _c_int, _c_ptr])
         lib.tge_attention_mma_scratch_floats.argtypes = [_c_int, _c_int, _c_int]
         lib.tge_attention_mma_scratch_floats.restype = _c_ll
         if lib.tge_attention_mma_head_dim() != head_dim or lib.tge_attention_mma_value_dim() != value_dim:
@@ -321,18 +328,19 @@ def scratch_floats(count: int) -> torch.Tensor:
 # ----------------------------------------------------------------------------
 # kernels
 # ----------------------------------------------------------------------------
-def embedding(table: torch.Tensor, ids: torch.Tensor, out: Optional[torch.Tensor] = None, scale: float = 1.0) -> torch.Tensor:
-    """out[t, :] = float32(table[ids[t], :]) * scale"""
+def embedding(table: torch.Tensor, ids: torch.Tensor, out: Optional[torch.Tensor] = None, scale: float = 1.0,
+              copies: int = 0) -> torch.Tensor:
+    """out[t, :] = float32(table[ids[t], :]) * scale; with ``copies`` > 0 out [T, copies, hidden], every copy that row."""
     _want(table, "embedding table", _FLOAT)
     _want(ids, "token ids", torch.int32)
     vocab, hidden = table.shape
     tokens = ids.numel()
     if out is None:
-        out = torch.empty((tokens, hidden), dtype=torch.float32, device=table.device)
+        out = torch.empty((tokens, copies, hidden) if copies else (tokens, hidden), dtype=torch.float32, device=table.device)
     _want(out, "embedding output", torch.float32)
     lib = core()
     _check(lib.tge_embedding(table.data_ptr(), int(table.dtype == torch.bfloat16), ids.data_ptr(), out.data_ptr(),
-                             tokens, hidden, vocab, float(scale), status_word().data_ptr(), _stream()), lib)
+                             tokens, hidden, max(int(copies), 1), vocab, float(scale), status_word().data_ptr(), _stream()), lib)
     return out
 
 
@@ -787,7 +795,7 @@ def attention(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tensor, blo
     scales its scores.
     ``keep_first`` (with a window): the first so many positions of a request stay visible beside the window.
     ``gate`` (run dtype [T, heads], dense rows, any row stride): logits of one gate per head; whoever writes a head's
-    output multiplies it by their logistic function.
+    output multiplies it by their logistic function.  [T, heads * value_dim]: one gate per number of the output.
     """
     v_pitch = 0
     if values_in_keys:
@@ -842,12 +850,15 @@ def attention(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tensor, blo
     keep_first = int(keep_first) if window > 0 else 0
     if pool and (keep_first or gate is not None):
         raise KernelError("attention: kept first tokens and gates go without pooled blocks")
-    gate_stride = 0
+    gate_stride, gate_elements = 0, 0
     if gate is not None:
-        _want(gate, "head gates", q.dtype, contiguous=False)
-        gate_stride = _rows_2d(gate, "head gates")
-        if tuple(gate.shape) != (tokens, heads):
-            raise KernelError(f"attention: gates must be [{tokens}, {heads}], got {tuple(gate.shape)}")
+        _want(gate, "gates", q.dtype, contiguous=False)
+        gate_stride = _rows_2d(gate, "gates")
+        if tuple(gate.shape) not in ((tokens, heads), (tokens, heads * value_dim)):
+            raise KernelError(f"attention: gates must be [{tokens}, {heads}] or [{tokens}, {heads * value_dim}], got {tuple(gate.shape)}")
+        gate_elements = int(value_dim > 1 and gate.shape[1] == heads * value_dim)
+        if gate_elements:       # the tensor-core kernels read eight of them at a time
+            pairs_ok = pairs_ok and gate_stride % 8 == 0 and gate.data_ptr() % 16 == 0
     # what a query's keys span, for the choice of runs: with a window, the window's tiles and the kept tokens'
     span = max_ctx_len
     if window > 0 and not pool:
@@ -887,7 +898,7 @@ def attention(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tensor, blo
                                      max_ctx_len, out.data_ptr(), out_stride, heads, kv_heads, float(scale), window,
                                      split_tokens, _ptr(scratch), status_word().data_ptr(), prefix, prefix_split,
                                      _ptr(sink), int(bool(pool)), v_pitch, _ptr(dist_bias), dist_span,
-                                     keep_first, _ptr(gate), gate_stride, _stream()), lib)
+                                     keep_first, _ptr(gate), gate_stride, gate_elements, _stream()), lib)
         if pool:
             core_lib = core()
             states = scratch.data_ptr()
@@ -905,7 +916,7 @@ def attention(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tensor, blo
                                   seq_of_token.data_ptr(), out.data_ptr(), out_stride, tokens, heads, kv_heads,
                                   head_dim, value_dim, _ptr(sink), float(scale), window, int(q.dtype == torch.bfloat16),
                                   int(pool), _ptr(pooled_k), _ptr(pooled_v), _ptr(pool_table), pool_width, pool_pages,
-                                  v_pitch, _ptr(dist_bias), dist_span, keep_first, _ptr(gate), gate_stride,
+                                  v_pitch, _ptr(dist_bias), dist_span, keep_first, _ptr(gate), gate_stride, gate_elements,
                                   status_word().data_ptr(), _stream()), lib)
     return out
 
@@ -1021,13 +1032,15 @@ def conv_norm_rope_store(raw: torch.Tensor, conv_w: Optional[torch.Tensor], taps
                          k_norm: Optional[torch.Tensor], eps: float, cos: Optional[torch.Tensor],
                          sin: Optional[torch.Tensor], rotary: int, positions: torch.Tensor, seq_of_token: torch.Tensor,
                          block_table: Optional[torch.Tensor], k_pages: Optional[torch.Tensor],
-                         v_pages: Optional[torch.Tensor], heads: int, kv_heads: int, dim: int, vdim: int) -> torch.Tensor:
+                         v_pages: Optional[torch.Tensor], heads: int, kv_heads: int, dim: int, vdim: int,
+                         norm_last: bool = False) -> torch.Tensor:
     """What lies between the q/k/v product and the attention when the projections pass through a short causal
     convolution over time: y_t = sum_j w[:, j] u_(t - taps + 1 + j) on every channel (``conv_w`` float32 [channels,
     taps]; inputs from before the portion come from ``conv_state`` float32 [slots, taps-1, channels], which is then
     brought up to date), an RMS norm of each q and k head (weights float32 [dim], None: none), the rotation of their
     first ``rotary`` elements, and the store of k and v into their pages (None: nothing is stored).  ``raw`` [T, q | k
-    | v] in the run dtype.  Returns the queries [T, heads*dim].  ``taps`` 0: no convolution."""
+    | v] in the run dtype.  Returns the queries [T, heads*dim].  ``taps`` 0: no convolution.  ``norm_last``: the norm of q and k
+    comes after their rotation (and has no weights where they are None) instead of before it."""
     _want(raw, "projections", _FLOAT, contiguous=False)
     ld = _rows_2d(raw, "projections")
     tokens = raw.shape[0]
@@ -1076,7 +1089,7 @@ def conv_norm_rope_store(raw: torch.Tensor, conv_w: Optional[torch.Tensor], taps
                                         _ptr(cos) if rotary else None, _ptr(sin) if rotary else None, table_positions,
                                         rotary, positions.data_ptr(), seq_of_token.data_ptr(), _ptr(block_table), max_pages,
                                         _ptr(k_pages), _ptr(v_pages), num_pages, page_size, q_out.data_ptr(), heads * dim,
-                                        tokens, num_seqs, heads, kv_heads, dim, vdim, int(store),
+                                        tokens, num_seqs, heads, kv_heads, dim, vdim, int(store), int(norm_last),
                                         status_word().data_ptr(), _stream()), lib)
     return q_out
 
@@ -1290,12 +1303,13 @@ def token_shift(h: torch.Tensor, mu: torch.Tensor, state: torch.Tensor, slots: t
 def latent_prepare(raw: torch.Tensor, q_rank: int, kv_rank: int, rot: int, gate_n: int, has_kv: bool,
                    q_weight: torch.Tensor, kv_weight: Optional[torch.Tensor], eps: float, cos: Optional[torch.Tensor],
                    sin: Optional[torch.Tensor], rot_dims: int, positions: torch.Tensor, seq_of_token: torch.Tensor,
-                   block_table: Optional[torch.Tensor], pages: Optional[torch.Tensor], out_dtype: torch.dtype):
+                   block_table: Optional[torch.Tensor], pages: Optional[torch.Tensor], out_dtype: torch.dtype,
+                   halves: bool = False):
     """From the float32 rows ``raw`` = [query latent | kv latent | shared key part | gate logits] (the middle two only
     with ``has_kv``): the RMS-normed query latent (run dtype [T, q_rank]) and the logistic gate (float32 [T, gate_n]);
     with ``pages`` ([num_pages, 1, page_size, kv_rank + rot]) the RMS-normed kv latent and the shared key part, its
-    first ``rot_dims`` numbers rotated in neighbouring pairs by the float32 tables ``cos`` / ``sin`` [positions,
-    rot_dims / 2], are written into each token's entry."""
+    first ``rot_dims`` numbers rotated in neighbouring pairs (``halves``: number i with i + rot_dims / 2) by the float32
+    tables ``cos`` / ``sin`` [positions, rot_dims / 2], are written into each token's entry."""
     _want(raw, "latent rows", torch.float32, contiguous=False)
     ld = _rows_2d(raw, "latent rows")
     tokens = raw.shape[0]
@@ -1326,7 +1340,7 @@ def latent_prepare(raw: torch.Tensor, q_rank: int, kv_rank: int, rot: int, gate_
     gate = torch.empty((tokens, gate_n), dtype=torch.float32, device=raw.device)
     lib = core()
     _check(lib.tge_latent_prepare(raw.data_ptr(), ld, q_rank, kv_rank, rot, gate_n, int(has_kv), q_weight.data_ptr(),
-                                  _ptr(kv_weight), float(eps), _ptr(cos), _ptr(sin), rot_dims, max_positions,
+                                  _ptr(kv_weight), float(eps), _ptr(cos), _ptr(sin), rot_dims, int(halves), max_positions,
                                   positions.data_ptr(), seq_of_token.data_ptr(), _ptr(block_table), max_pages, num_pages,
                                   page_size, _ptr(pages) if has_kv else None, q_latent.data_ptr(), gate.data_ptr(),
                                   int(out_dtype == torch.bfloat16), tokens, status_word().data_ptr(), _stream()), lib)
@@ -1360,11 +1374,13 @@ def head_linear(x: torch.Tensor, x_head: int, w: torch.Tensor, out: torch.Tensor
     return out
 
 
-def rotate_interleaved(src: torch.Tensor, src_head: int, dst: torch.Tensor, dst_head: int, heads: int, width: int,
-                       cos: torch.Tensor, sin: torch.Tensor, rot_dims: int, positions: torch.Tensor, first: int = 0) -> torch.Tensor:
+def rotate_runs(src: torch.Tensor, src_head: int, dst: torch.Tensor, dst_head: int, heads: int, width: int,
+                cos: torch.Tensor, sin: torch.Tensor, rot_dims: int, positions: torch.Tensor, first: int = 0,
+                halves: bool = False) -> torch.Tensor:
     """dst[t, n * dst_head + e] = src[t, n * src_head + e] for e < width, with the ``rot_dims`` numbers of every
-    run from ``first`` on rotated in neighbouring pairs: (u, v) at position p -> (u cos a - v sin a, v cos a + u sin a),
-    a = p * f_i, from float32 tables [positions, rot_dims / 2].  Two buffers (or disjoint runs)."""
+    run from ``first`` on rotated in neighbouring pairs (``halves``: number i with i + rot_dims / 2): (u, v) at position
+    p -> (u cos a - v sin a, v cos a + u sin a), a = p * f_i, from float32 tables [positions, rot_dims / 2].  Two buffers
+    (or disjoint runs)."""
     _want(src, "rotation input", _FLOAT, contiguous=False)
     _want(dst, "rotation output", src.dtype, contiguous=False)
     _want(positions, "positions", torch.int32)
@@ -1374,14 +1390,14 @@ def rotate_interleaved(src: torch.Tensor, src_head: int, dst: torch.Tensor, dst_
         _want(cos, "cos table", torch.float32)
         _want(sin, "sin table", torch.float32)
         if cos.shape != sin.shape or cos.shape[1] != rot_dims // 2:
-            raise KernelError(f"rotate_interleaved: tables {tuple(cos.shape)} for {rot_dims} rotated numbers")
+            raise KernelError(f"rotate_runs: tables {tuple(cos.shape)} for {rot_dims} rotated numbers")
     if (heads - 1) * src_head + width > src.shape[1] or (heads - 1) * dst_head + width > dst.shape[1] or dst.shape[0] != tokens:
-        raise KernelError("rotate_interleaved: the runs do not fit the rows")
+        raise KernelError("rotate_runs: the runs do not fit the rows")
     lib = core()
-    _check(lib.tge_rotate_interleaved(src.data_ptr(), lds, int(src_head), dst.data_ptr(), ldd, int(dst_head), _ptr(cos) if rot_dims else None,
-                                      _ptr(sin) if rot_dims else None, int(rot_dims), cos.shape[0] if rot_dims else 2 ** 31 - 1,
-                                      positions.data_ptr(), tokens, int(heads), int(width), int(first),
-                                      int(src.dtype == torch.bfloat16), status_word().data_ptr(), _stream()), lib)
+    _check(lib.tge_rotate_runs(src.data_ptr(), lds, int(src_head), dst.data_ptr(), ldd, int(dst_head), _ptr(cos) if rot_dims else None,
+                               _ptr(sin) if rot_dims else None, int(rot_dims), cos.shape[0] if rot_dims else 2 ** 31 - 1,
+                               positions.data_ptr(), tokens, int(heads), int(width), int(first), int(halves),
+                               int(src.dtype == torch.bfloat16), status_word().data_ptr(), _stream()), lib)
     return dst
 
 
@@ -1448,15 +1464,20 @@ ACT_RELU_SQUARED, ACT_XIELU = 0, 1
 
 
 def router_topk(logits: torch.Tensor, correction: Optional[torch.Tensor], top: int, group_count: int = 1,
-                group_keep: int = 1, logistic: bool = False, over_sum: bool = True):
+                group_keep: int = 1, logistic: bool = False, over_sum: bool = True, group_pairs: bool = False,
+                factor: float = 1.0, outputs: int = 0):
     """(ids int32 [T, top], weights float32 [T, top]) from float32 router logits [T, outputs]: scores = softmax over
     all outputs; the ``top`` outputs with the largest score + correction are chosen (the lowest index among equals),
-    only inside the ``group_keep`` of ``group_count`` groups of neighbouring outputs whose best such value is largest;
-    weights = the chosen outputs' scores over their sum (+ 1e-20), or as they are without ``over_sum``.  ``logistic``: an
-    output's score is the logistic function of its own logit."""
+    only inside the ``group_keep`` of ``group_count`` groups of neighbouring outputs whose best such value is largest
+    (``group_pairs``: the sum of its two largest); weights = the chosen outputs' scores over their sum (+ 1e-20), or as they
+    are without ``over_sum``, times ``factor``.  ``logistic``: an output's score is the logistic function of its own logit.
+    ``outputs``: only the first so many columns of ``logits`` are router outputs (0: all)."""
     _want(logits, "router logits", torch.float32, contiguous=False)
     ld = _rows_2d(logits, "router logits")
-    tokens, outputs = logits.shape
+    tokens = logits.shape[0]
+    outputs = outputs or logits.shape[1]
+    if outputs > logits.shape[1]:
+        raise KernelError(f"router_topk: {outputs} outputs in rows of {logits.shape[1]}")
     if correction is not None:
         _want(correction, "router correction", torch.float32)
         if correction.numel() != outputs:
@@ -1465,7 +1486,7 @@ def router_topk(logits: torch.Tensor, correction: Optional[torch.Tensor], top: i
     weights = torch.empty((tokens, top), dtype=torch.float32, device=logits.device)
     lib = core()
     _check(lib.tge_router_topk(logits.data_ptr(), ld, _ptr(correction), tokens, outputs, int(top), int(group_count),
-                               int(group_keep), int(logistic), int(over_sum), ids.data_ptr(), weights.data_ptr(), _stream()), lib)
+                               int(group_keep), int(group_pairs), int(logistic), int(over_sum), float(factor), ids.data_ptr(), weights.data_ptr(), _stream()), lib)
     return ids, weights
 
 
@@ -1484,48 +1505,64 @@ def activation(rows: torch.Tensor, kind: int, params: Optional[torch.Tensor] = N
     return rows
 
 
+def _row_gate(gate: Optional[torch.Tensor], tokens: int):
+    """(pointer, stride) of one float32 logit per token, or of none."""
+    if gate is None:
+        return None, 0
+    _want(gate, "gate logits", torch.float32, contiguous=False)
+    if gate.dim() != 1 or gate.shape[0] != tokens:
+        raise KernelError(f"gate logits must be [{tokens}], got {tuple(gate.shape)}")
+    return gate.data_ptr(), gate.stride(0)
+
+
 def experts_direct(h: torch.Tensor, w_up: torch.Tensor, w_down: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor,
-                   x: torch.Tensor, gate=None, weigh_input: bool = False) -> None:
+                   x: torch.Tensor, gate=None, weigh_input: bool = False, x_gate: Optional[torch.Tensor] = None) -> None:
     """x[t] += sum_k weights[t, k] * (w_down[e] relu(w_up[e] h[t])^2 with e = ids[t, k], or h[t] itself when e is
     beyond the experts), every pair reading its expert's rows directly: for steps of few tokens.  w_up [experts, ff,
     width], w_down [width, experts, ff] (the experts' down matrices side by side), x float32 [T, width].
     ``gate`` (limit, alpha, offset): clamped gated experts instead, w_up [experts, 2 ff, width] with gate and up rows
-    interleaved.  ``weigh_input``: the weight multiplies the expert's input, not its output."""
+    interleaved.  ``weigh_input``: the weight multiplies the expert's input, not its output.  ``x_gate`` (float32 [T], any
+    stride): what ``x`` held is multiplied by the logistic function of its token's number.  The rows of ``w_down`` may lie
+    further apart than experts * ff."""
     _want(h, "expert input", _FLOAT, contiguous=False)
     _want(w_up, "expert up weights", h.dtype)
-    _want(w_down, "expert down weights", h.dtype)
+    _want(w_down, "expert down weights", h.dtype, contiguous=False)
     _want(ids, "expert ids", torch.int32)
     _want(weights, "expert weights", torch.float32)
     _want(x, "stream", torch.float32)
     tokens, width = x.shape
     experts, ff = w_up.shape[0], w_up.shape[1] // (1 if gate is None else 2)
     top = ids.shape[1]
-    if w_up.shape[2] != width or tuple(w_down.shape) != (width, experts, ff) or h.shape[0] != tokens or h.shape[1] != width:
+    if w_up.shape[2] != width or tuple(w_down.shape) != (width, experts, ff) or h.shape[0] != tokens or h.shape[1] != width or (
+            experts and (w_down.stride(2) != 1 or w_down.stride(1) != ff)):
         raise KernelError("experts: shapes do not agree")
     inner = torch.empty((tokens * top, ff), dtype=h.dtype, device=h.device)
     lib = core()
     _check(lib.tge_experts_direct(h.data_ptr(), _rows_2d(h, "expert input"), w_up.data_ptr(), w_down.data_ptr(), ff,
-                                  experts * ff, ids.data_ptr(), weights.data_ptr(), inner.data_ptr(), x.data_ptr(), tokens, top,
+                                  w_down.stride(0), ids.data_ptr(), weights.data_ptr(), inner.data_ptr(), x.data_ptr(), tokens, top,
                                   experts, width, ff, int(weigh_input), int(gate is not None),
-                                  *(float(v) for v in (gate or (1.0, 1.0, 1.0))), int(h.dtype == torch.bfloat16), _stream()), lib)
+                                  *(float(v) for v in (gate or (1.0, 1.0, 1.0))), *_row_gate(x_gate, tokens), int(h.dtype == torch.bfloat16), _stream()), lib)
 
 
 def experts_dense_gate(z: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor, experts: int, gate,
-                       weigh_input: bool) -> torch.Tensor:
+                       weigh_input: bool, shared_ff: int = 0, shared_gate: Optional[torch.Tensor] = None) -> torch.Tensor:
     """z [T, experts * 2 ff] (gate and up of every expert for every token, interleaved) -> [T, experts * ff]: for a token's
     chosen experts min(g, L) sigmoid(alpha min(g, L)) (clamp(u, -L, L) + offset) with ``gate`` = (L, alpha, offset), the
-    weight multiplying (g, u) with ``weigh_input`` and the value without; zeros for the other experts."""
+    weight multiplying (g, u) with ``weigh_input`` and the value without; zeros for the other experts.  ``shared_ff`` > 0:
+    z has 2 shared_ff more columns and the result shared_ff more, those of a feed-forward that every token uses, whose values
+    are multiplied by the logistic function of ``shared_gate`` (float32 [T], any stride; None: by one)."""
     _want(z, "expert rows", _FLOAT)
     _want(ids, "expert ids", torch.int32)
     _want(weights, "expert weights", torch.float32)
     tokens, columns = z.shape
-    if columns % (2 * experts) or ids.shape[0] != tokens or weights.shape != ids.shape:
+    ff = (columns // 2 - shared_ff) // experts
+    if columns != 2 * (experts * ff + shared_ff) or ff <= 0 or ids.shape[0] != tokens or weights.shape != ids.shape:
         raise KernelError("experts: shapes do not agree")
     out = torch.empty((tokens, columns // 2), dtype=z.dtype, device=z.device)
     lib = core()
     _check(lib.tge_experts_dense_gate(z.data_ptr(), ids.data_ptr(), weights.data_ptr(), out.data_ptr(), tokens, ids.shape[1],
-                                      int(experts), columns // (2 * experts), int(weigh_input), *(float(v) for v in gate),
-                                      int(z.dtype == torch.bfloat16), _stream()), lib)
+                                      int(experts), ff, int(weigh_input), *(float(v) for v in gate), int(shared_ff),
+                                      *_row_gate(shared_gate, tokens), int(z.dtype == torch.bfloat16), _stream()), lib)
     return out
 
 
@@ -1572,9 +1609,9 @@ def experts_group(h: torch.Tensor, ids: torch.Tensor, experts: int, in_weights: 
 
 
 def experts_combine_add(outputs: torch.Tensor, place: torch.Tensor, weights: Optional[torch.Tensor], h: torch.Tensor,
-                        x: torch.Tensor) -> None:
+                        x: torch.Tensor, x_gate: Optional[torch.Tensor] = None) -> None:
     """x[t] += sum_k weights[t, k] * (outputs[place[t, k]] or, where place is -1, h[t]); outputs float32 grouped rows;
-    ``weights`` None: all one."""
+    ``weights`` None: all one.  ``x_gate`` as in :func:`experts_direct`."""
     _want(outputs, "expert outputs", torch.float32)
     _want(place, "expert places", torch.int32)
     if weights is not None:
@@ -1585,7 +1622,7 @@ def experts_combine_add(outputs: torch.Tensor, place: torch.Tensor, weights: Opt
     top = place.numel() // max(tokens, 1)
     lib = core()
     _check(lib.tge_experts_combine_add(outputs.data_ptr(), place.data_ptr(), _ptr(weights), h.data_ptr(),
-                                       _rows_2d(h, "expert input"), x.data_ptr(), tokens, top, width,
+                                       _rows_2d(h, "expert input"), x.data_ptr(), tokens, top, width, *_row_gate(x_gate, tokens),
                                        int(h.dtype == torch.bfloat16), _stream()), lib)
 
 
@@ -1845,3 +1882,98 @@ def concat_rows(a: torch.Tensor, b: torch.Tensor, out_dtype: torch.dtype) -> tor
     _check(lib.tge_concat_rows(a.data_ptr(), b.data_ptr(), out.data_ptr(), int(out_dtype == torch.bfloat16), a.shape[0],
                                a.shape[1], _stream()), lib)
     return out
+
+
+# ----------------------------------------------------------------------------
+# a residual made of several streams
+# ----------------------------------------------------------------------------
+def _streams_of(x: torch.Tensor) -> Tuple[int, int, int]:
+    _want(x, "residual streams", torch.float32)
+    if x.dim() != 3:
+        raise KernelError(f"residual streams must be [T, streams, width], got {tuple(x.shape)}")
+    return tuple(x.shape)
+
+
+def _connection(streams: int, width: int, mix, out, into, gain) -> None:
+    for name, t, count in (("stream matrix", mix, streams * streams), ("stream outputs", out, streams), ("stream inputs", into, streams),
+                           ("norm weight", gain, width)):
+        if t is not None:
+            _want(t, name, torch.float32)
+            if t.numel() != count:
+                raise KernelError(f"{name}: {t.numel()} numbers for {streams} streams of width {width}")
+
+
+def streams_norm(x: torch.Tensor, into: Optional[torch.Tensor], gain: torch.Tensor, eps: float, out_dtype: torch.dtype,
+                 rows: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """What a sublayer reads of the streams ``x`` (float32 [T, S, width]): RMS norm of sum_s into[s] x_s (None: all one) times
+    ``gain``, in ``out_dtype``; optionally of the rows that ``rows`` names only."""
+    tokens, streams, width = _streams_of(x)
+    _connection(streams, width, None, None, into, gain)
+    if rows is not None:
+        _want(rows, "norm row index", torch.int32)
+    count = tokens if rows is None else rows.numel()
+    h = torch.empty((count, width), dtype=out_dtype, device=x.device)
+    lib = core()
+    _check(lib.tge_streams_rows(x.data_ptr(), count, tokens, streams, width, None, 0, None, None, _ptr(into), gain.data_ptr(),
+                                float(eps), _ptr(rows), h.data_ptr(), int(out_dtype == torch.bfloat16), status_word().data_ptr(),
+                                _stream()), lib)
+    return h
+
+
+def streams_update(x: torch.Tensor, y: torch.Tensor, mix: torch.Tensor, out: torch.Tensor, following=None,
+                   out_dtype: Optional[torch.dtype] = None) -> Optional[torch.Tensor]:
+    """The streams after a sublayer, in place: x_t <- sum_s mix[s, t] x_s + out[t] y (y float32 [T, width]).  ``following``
+    (into, gain, eps): also what the next sublayer reads (:func:`streams_norm` of the new streams), from the same kernel."""
+    tokens, streams, width = _streams_of(x)
+    _want(y, "sublayer output", torch.float32, contiguous=False)
+    if tuple(y.shape) != (tokens, width):
+        raise KernelError(f"sublayer output must be [{tokens}, {width}], got {tuple(y.shape)}")
+    into, gain, eps = following if following is not None else (None, None, 1.0)
+    _connection(streams, width, mix, out, into, gain)
+    h = torch.empty((tokens, width), dtype=out_dtype, device=x.device) if following is not None else None
+    lib = core()
+    _check(lib.tge_streams_rows(x.data_ptr(), tokens, tokens, streams, width, y.data_ptr(), _rows_2d(y, "sublayer output"),
+                                mix.data_ptr(), out.data_ptr(), _ptr(into), _ptr(gain), float(eps), None, _ptr(h),
+                                int(out_dtype == torch.bfloat16), status_word().data_ptr(), _stream()), lib)
+    return h
+
+
+def streams_defer(x: torch.Tensor, following, partial: Optional[torch.Tensor] = None, splits: int = 0,
+                  mix: Optional[torch.Tensor] = None, out: Optional[torch.Tensor] = None) -> Optional[DeferredRows]:
+    """For up to ``DEFER_MAX_TOKENS`` tokens in bfloat16, a row spread over many blocks: the update with the sublayer's output
+    as ``splits`` partial sums [splits, T, width] (``partial`` None: no update), and what the next sublayer reads as rows
+    without their norm factor (``following`` None: nothing)."""
+    tokens, streams, width = _streams_of(x)
+    into, gain, eps = following if following is not None else (None, None, 1.0)
+    _connection(streams, width, mix, out, into, gain)
+    lib = core()
+    rows = sums = None
+    if following is not None:
+        rows = torch.empty((tokens, width), dtype=torch.bfloat16, device=x.device)
+        sums = torch.empty((lib.tge_streams_slices(width), tokens), dtype=torch.float32, device=x.device)
+    if partial is not None:
+        _want(partial, "partial sums", torch.float32)
+        if partial.numel() < splits * tokens * width:
+            raise KernelError("streams: the partial sums are too few")
+    _check(lib.tge_streams_update_defer(x.data_ptr(), tokens, streams, width, _ptr(partial), int(splits), _ptr(mix), _ptr(out),
+                                        _ptr(into), _ptr(gain), _ptr(rows), _ptr(sums), _stream()), lib)
+    return DeferredRows(rows, sums, width, eps) if following is not None else None
+
+
+def linear_partials(x: torch.Tensor, w: torch.Tensor) -> Optional[Tuple[torch.Tensor, int]]:
+    """x . w^T of a small bfloat16 batch as float32 partial sums [splits, M, N] in the scratch buffer, not yet added up:
+    (buffer, splits), to be read by the next kernel of the stream.  None: not a product for this path."""
+    M, K = x.shape
+    N = w.shape[0]
+    if not (x.dtype == torch.bfloat16 and USE_TCGEN05 and M <= DEFER_MAX_TOKENS):
+        return None
+    _want(x, "linear input", torch.bfloat16, contiguous=False)
+    _want(w, "linear weight", torch.bfloat16, contiguous=False)
+    if w.shape[1] != K:
+        raise KernelError(f"linear: input has {K} columns, weight has {w.shape[1]}")
+    lib = core()
+    scratch = scratch_floats(max(lib.tge_gemm_tcgen05_scratch_floats(M, N, K), M * N))
+    splits = _c_int(0)
+    rc = lib.tge_gemm_tcgen05_partials(x.data_ptr(), _rows_2d(x, "linear input"), w.data_ptr(), _rows_2d(w, "linear weight"), M, N, K,
+                                       scratch.data_ptr(), scratch.numel(), ctypes.byref(splits), status_word().data_ptr(), _stream())
+    return None if _check(rc, lib) == UNSUPPORTED else (scratch, splits.value)

@@ -48,6 +48,10 @@ tokens of the request stay visible; one gate per head (``head_gate``), the logis
 input, that multiplies the head's output where the attention writes it; and a layer that has no keys and values of its own
 (``own_kv: False``) because it reads an earlier layer's cache.  The gate's rows lie below q, k and v in the one input
 product; one kernel normalises and stores, and the attention adds the bias and applies the gate.
+
+On the general path, too: the norm of q and k after their rotation, with or without weights (``qk_norm`` with
+``"after_rotation": True``); a sink whose score is a constant and not learned (``sink_score``); and one gate per number of
+the output (``output_gate``), the logistic function of a projection of the same input, applied where the attention writes.
 """
 from __future__ import annotations
 
@@ -77,8 +81,10 @@ class GQAttention(Mixer):
     or ``{"coef": c, "every": n}``), ``distance_bias`` (None or ``{"far": D}``; weight ``rel`` float32 [rows, heads], the
     rows taken from the tensor).
     The separate path: ``distance_bias`` with values of their own, ``qk_norm`` ``{"scope": "head", "eps": e, "weight": False}``
-    (no ``q_norm.weight`` / ``k_norm.weight``), ``keep_first`` (0, or with a window how many first tokens stay visible),
+    (no ``q_norm.weight`` / ``k_norm.weight``; on the general path also with ``"after_rotation": True``), ``keep_first`` (0, or with a window how many first tokens stay visible),
     ``head_gate`` (bool; ``gate.weight`` [heads, hidden]), ``own_kv`` (default True; False: no ``k.weight`` / ``v.weight``).
+    More of the general path: ``sink_score`` (None, or every head's sink as a constant), ``output_gate`` (bool; ``gate.weight``
+    [heads * value_dim, hidden]).
     """
     graph_safe = True
     can_defer_norm = True
@@ -122,6 +128,11 @@ class GQAttention(Mixer):
         if self.q_temp is not None and not self.values_are_keys:
             raise ValueError("attention: a query temperature is built for values that are the keys")
         self.norm_weights = norm is None or bool(norm.get("weight", True))
+        self.norm_last = norm is not None and bool(norm.get("after_rotation", False))
+        self.sink_score = None if p.get("sink_score") is None else float(p["sink_score"])
+        if self.sinks and self.sink_score is not None:
+            raise ValueError("attention: a sink is learned or a constant, not both")
+        self.output_gate = bool(p.get("output_gate", False))
         self.keep_first = int(p.get("keep_first") or 0)
         self.head_gate = bool(p.get("head_gate", False))
         self.own_kv = bool(p.get("own_kv", True))
@@ -153,8 +164,13 @@ class GQAttention(Mixer):
                                  "or none, and neither convolution, pooled blocks nor value mixing")
             self.v_dim = 0
         # the general path: convolution, per-head norm, rotation and store in one kernel, pooled blocks
-        self.general = bool(p.get("prepare_in_one_kernel") or self.taps or self.pool
+        self.general = bool(p.get("prepare_in_one_kernel") or self.taps or self.pool or self.norm_last or self.output_gate
                             or (self.value_dim != self.head_dim and self.rotates))
+        if self.general and (self.values_are_keys or (not self.norm_weights and not self.norm_last)):
+            raise ValueError("attention: gates per number, a norm after the rotation and the like go with values of their own, and a "
+                             "norm without weights comes after the rotation there")
+        if self.output_gate and self.pool:
+            raise ValueError("attention: gates per number of the output go without pooled blocks")
         if self.general:
             if self.value_mix is not None or self.qkv_bias or (self.qk_norm is not None and self.qk_norm[0] != "head"):
                 raise ValueError("attention: a short convolution, pooled blocks, or a rotation with values of their own "
@@ -162,7 +178,7 @@ class GQAttention(Mixer):
             if tables is None:
                 raise ValueError("attention: the general path rotates by tables, or not at all")
         # the separate path: one kernel normalises and stores behind the product, the attention does the rest
-        self.separate = not self.values_are_keys and (self.dist_far is not None or not self.norm_weights or self.keep_first > 0
+        self.separate = not self.values_are_keys and not (self.norm_last or self.output_gate) and (self.dist_far is not None or not self.norm_weights or self.keep_first > 0
                                                       or self.head_gate or not self.own_kv)
         if self.separate:
             if (self.general or self.rotates or self.value_mix is not None or self.qkv_bias
@@ -170,13 +186,17 @@ class GQAttention(Mixer):
                 raise ValueError("attention: a bias by distance, kept first tokens, a gate per head or borrowed keys and values go "
                                  "with no rotation, a per-head q/k norm or none, and neither convolution, pooled blocks, biases on "
                                  "q, k, v nor value mixing")
-        elif self.keep_first or self.head_gate or not self.own_kv or not self.norm_weights:
-            raise ValueError("attention: values that are the keys go without kept first tokens, gates or borrowed keys")
+        elif (self.keep_first or self.head_gate or not self.own_kv or (not self.norm_weights and not self.general)
+              or (self.general and self.dist_far is not None)):
+            raise ValueError("attention: values that are the keys, and the general path, go without kept first tokens, gates per head, "
+                             "borrowed keys or (the general path) a bias by distance")
         # rows of the gate inside the input product, padded with zero rows so that a product's row stays a multiple of 16 bytes
         self.gate_rows = 0
         if self.head_gate:
             kv = self.kv_dim + self.v_dim if self.own_kv else 0
             self.gate_rows = self.heads + -(self.q_dim + kv + self.heads) % 16
+        elif self.output_gate:
+            self.gate_rows = self.o_dim + -(self.q_dim + self.kv_dim + self.v_dim + self.o_dim) % 16
         self.conv_w: Optional[torch.Tensor] = None
         self.q_norm_w: Optional[torch.Tensor] = None
         self.k_norm_w: Optional[torch.Tensor] = None
@@ -202,6 +222,8 @@ class GQAttention(Mixer):
             del specs["k.weight"], specs["v.weight"]
         if self.head_gate:
             specs["gate.weight"] = ParamSpec((self.heads, self.hidden))
+        if self.output_gate:
+            specs["gate.weight"] = ParamSpec((self.o_dim, self.hidden))
         if self.dist_far is not None:
             specs["rel"] = ParamSpec((-1, self.heads), role="vector")
         if self.qk_norm is not None and self.norm_weights:
@@ -231,9 +253,9 @@ class GQAttention(Mixer):
         # rows of q, then k, then v: one product serves all three
         rows = ("q", "k") if self.values_are_keys else ("q", "k", "v") if self.own_kv else ("q",)
         blocks = [tensors[f"{t}.weight"] for t in rows]
-        if self.head_gate:
+        if self.head_gate or self.output_gate:
             gate = tensors["gate.weight"]
-            blocks += [gate, gate.new_zeros((self.gate_rows - self.heads, self.hidden))]
+            blocks += [gate, gate.new_zeros((self.gate_rows - gate.shape[0], self.hidden))]
         self.w_qkv = torch.cat(blocks, dim=0).contiguous()
         if self.qkv_bias:
             self.b_qkv = torch.cat([tensors[f"{t}.bias"] for t in rows]).contiguous()
@@ -241,13 +263,17 @@ class GQAttention(Mixer):
             self.dist_table = self.expand_distance_bias(tensors["rel"], self.dist_far)
         self.w_o = tensors["o.weight"].contiguous()
         self.b_o = tensors["o.bias"].contiguous() if self.o_bias else None
-        if self.qk_norm is not None and not self.norm_weights:
+        if self.norm_last and not self.norm_weights:
+            pass                                          # nothing to multiply by
+        elif self.qk_norm is not None and not self.norm_weights:
             self.q_norm_w = self.k_norm_w = torch.ones(self.head_dim, dtype=torch.float32, device=self.w_o.device)
         elif self.qk_norm is not None:
             self.q_norm_w = tensors["q_norm.weight"].contiguous()
             self.k_norm_w = tensors["k_norm.weight"].contiguous()
         if self.sinks:
             self.sink = tensors["sink"].contiguous()
+        elif self.sink_score is not None:
+            self.sink = torch.full((self.heads,), self.sink_score, dtype=torch.float32, device=self.w_o.device)
         if self.taps:
             self.conv_w = torch.cat([tensors["q.conv.weight"], tensors["k.conv.weight"], tensors["v.conv.weight"]],
                                     dim=0).contiguous()
@@ -282,8 +308,9 @@ class GQAttention(Mixer):
 
     def flops(self, tokens: int, pairs: float) -> float:
         kv = self.kv_dim + self.v_dim if self.own_kv else 0
-        products = 2.0 * tokens * (self.q_dim + kv + self.o_dim + (self.heads if self.head_gate else 0)) * self.hidden
-        if self.separate and self.window is not None:
+        products = 2.0 * tokens * (self.q_dim + kv + self.o_dim + (self.heads if self.head_gate else 0)
+                                   + (self.o_dim if self.output_gate else 0)) * self.hidden
+        if (self.separate or (self.general and not self.pool)) and self.window is not None:
             # a query meets at most the window's keys and the kept ones
             limit = int(self.window) + self.keep_first
             if 2.0 * pairs == tokens * (tokens + 1.0):                    # a whole prompt
@@ -365,7 +392,9 @@ class GQAttention(Mixer):
                                      ctx.num_seqs, self.q_norm_w, self.k_norm_w, self.qk_norm[1] if self.qk_norm else 1.0,
                                      cos, sin, rotary, ctx.positions, ctx.seq_of_token, table,
                                      k_pages if cache.owner else None, v_pages if cache.owner else None,
-                                     self.heads, self.kv_heads, self.head_dim, self.value_dim)
+                                     self.heads, self.kv_heads, self.head_dim, self.value_dim, norm_last=self.norm_last)
+        first = self.q_dim + self.kv_dim + self.v_dim
+        gate = raw[:, first:first + self.o_dim] if self.output_gate else None
         pooled = {}
         if self.pool:
             more = cache.more["pooled"]
@@ -378,7 +407,7 @@ class GQAttention(Mixer):
                              ctx.num_seqs, ctx.max_q_len, ctx.max_ctx_len, self.heads, self.kv_heads, self.head_dim,
                              self.scale, window=int(self.window or 0), split_tokens=ctx.attn_split_tokens,
                              typical_ctx_len=ctx.typical_ctx_len, decode_prefix=ctx.decode_prefix, sink=self.sink,
-                             out=out, **pooled)
+                             out=out, gate=gate, **pooled)
 
     def share_input_projection(self, rows: torch.Tensor) -> Optional[torch.Tensor]:
         """A block offers the rows of another product over the same input (a feed-forward's up weight) to be

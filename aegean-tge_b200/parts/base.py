@@ -316,6 +316,19 @@ class FeedForward(Part):
     def output_projection(self) -> Optional[Tuple[torch.Tensor, Optional[torch.Tensor]]]:
         return None
 
+    def takes_deferred_at(self, tokens: int) -> bool:
+        """Whether, in a step of so many tokens, the rows may come without their norm's factor at no cost."""
+        return self.takes_deferred_rows
+
+    def last_product(self, h: torch.Tensor, ctx: StepContext) -> Optional[Tuple[torch.Tensor, torch.Tensor]]:
+        """(rows, weight) of a plain product whose result is this feed-forward's whole output in this step, for a caller
+        that runs it itself; None: ask :meth:`forward_f32`."""
+        projection = self.output_projection()
+        if projection is None or projection[1] is not None:
+            return None
+        rows = self.inner(h, ctx)
+        return None if rows is None else (rows, projection[0])
+
     def forward_f32(self, h: torch.Tensor, ctx: StepContext) -> torch.Tensor:
         """The feed-forward's output in float32 [T, H] (see ``Mixer.forward_f32``)."""
         out = torch.zeros((h.shape[0], self.env.hidden_size), dtype=torch.float32, device=h.device)
@@ -358,6 +371,7 @@ class Block:
         raise NotImplementedError
 
     passes_deferred_rows = False
+    streams = False               # True: the stream is several rows per token, [T, streams, width]
 
     def parts(self) -> Dict[str, Part]:
         named = {"mixer_norm": self.mixer_norm, "mixer": self.mixer,

@@ -173,3 +173,43 @@ class PostNormBlock(Block):
         elif second is not None:
             h = ops.scale_add_norm(x, torch.zeros_like(x), self.alpha, second[0], second[1], self.env.dtype)
         return h
+
+
+@BLOCKS.register("hyper_connected")
+class HyperConnectedBlock(Block):
+    """Each sublayer reads one combination of several streams and writes all of them (parts/stream.py); both norms are
+    ``connected_rmsnorm`` parts.  The feed-forward may be absent; a second norm is then read by nothing.
+
+    A sublayer that ends in a plain product hands it out, so that for few tokens the kernel that adds up the product's
+    partial sums also updates the streams and combines them for the next norm."""
+
+    passes_deferred_rows = True
+    streams = True
+
+    def __init__(self, mixer, feed_forward, mixer_norm, ffn_norm, env, params=None):
+        super().__init__(mixer, feed_forward, mixer_norm, ffn_norm, env, params)
+        for norm in (mixer_norm,) + ((ffn_norm,) if feed_forward is not None else ()):
+            if not getattr(norm, "connected", False):
+                raise ValueError("hyper_connected block: a sublayer needs a norm with a connection to the streams")
+
+    def forward(self, x, ctx: StepContext, cache: LayerCache, h=None, next_norm=None, next_takes_deferred=False):
+        tokens = x.shape[0]
+        if h is None:
+            h = self.mixer_norm.forward(x, defer=self.mixer.takes_deferred_rows)
+        if next_norm is not None and not hasattr(next_norm, "reads"):
+            next_norm = None
+        if self.feed_forward is None:
+            following, defer = next_norm, next_takes_deferred
+        else:
+            following, defer = self.ffn_norm, self.feed_forward.takes_deferred_at(tokens)
+        projection = self.mixer.output_projection()
+        if projection is not None and projection[1] is None:
+            h = self.mixer_norm.update_product(x, self.mixer.inner(h, ctx, cache), projection[0], following, defer)
+        else:
+            h = self.mixer_norm.update(x, self.mixer.forward_f32(h, ctx, cache), following, defer)
+        if self.feed_forward is None:
+            return h
+        last = self.feed_forward.last_product(h, ctx)
+        if last is not None:
+            return self.ffn_norm.update_product(x, last[0], last[1], next_norm, next_takes_deferred)
+        return self.ffn_norm.update(x, self.feed_forward.forward_f32(h, ctx), next_norm, next_takes_deferred)

@@ -18,7 +18,8 @@ from .base import EMBEDDINGS, HEADS, NORMS, ParamSpec, Part, build_part
 class TokenEmbedding(Part):
     """params: ``vocab_size``, ``hidden_size``; optional ``norm`` (a norm's PartSpec: the looked-up rows are
     normalised before they become the stream; the norm needs ``forward_stream``), ``scale`` (a factor on the looked-up
-    rows, default 1; a head that shares the table reads it unscaled).  weights: ``weight`` and, with a
+    rows, default 1; a head that shares the table reads it unscaled), ``streams`` (the stream is that many copies of the
+    rows, [T, streams, hidden], and goes without a norm; default: one, [T, hidden]).  weights: ``weight`` and, with a
     norm, its parameters as ``norm.<name>``."""
     graph_safe = True
 
@@ -28,6 +29,9 @@ class TokenEmbedding(Part):
         self.hidden = int(spec.params["hidden_size"])
         self.scale = float(spec.params.get("scale", 1.0))
         self.weight: Optional[torch.Tensor] = None
+        self.streams = int(spec.params.get("streams", 0))
+        if self.streams < 0 or (self.streams and spec.params.get("norm") is not None):
+            raise ValueError("token_embedding: several streams go without a norm of the embedding")
         norm = spec.params.get("norm")
         self.norm = build_part(NORMS, norm, env) if norm is not None else None
         if self.norm is not None and not hasattr(self.norm, "forward_stream"):
@@ -48,7 +52,7 @@ class TokenEmbedding(Part):
         return 0        # a step reads the rows of its tokens, not the table
 
     def forward(self, token_ids: torch.Tensor) -> torch.Tensor:
-        x = self.ops.embedding(self.weight, token_ids, scale=self.scale)
+        x = self.ops.embedding(self.weight, token_ids, scale=self.scale, copies=self.streams)
         return x if self.norm is None else self.norm.forward_stream(x)
 
 

@@ -5,7 +5,7 @@
     cq = rms(Wdq h) gq                     q = Wuq cq              per head [dim plain | rot rotated]
     [c_raw | kr] = Wdkv h                  c = rms(c_raw) gkv      kr: one rotated key part for all heads
     k_n = [Wuk_n c | kr]                   v_n = Wuv_n c
-    s_ij = scale (q_i . k_j),  j <= i      softmax, o = sum_j p_ij v_j
+    s_ij = scale (q_i . k_j),  j <= i      softmax, o = sum_j p_ij v_j    (with a window w: 0 <= i - j < w)
     out = Wo (gate * o)                    gate = sigmoid(Wg h), one per head or one per element, or none
 
 A token keeps only ``[c | kr]`` (kv_rank + rot numbers, one cache entry, whatever the head count).  The keys and
@@ -13,12 +13,12 @@ values are never materialised: the query's plain part is carried into the latent
 s_ij = scale (q~_n . c_j + qr_n . kr_j), the paged attention kernels run with ONE key/value head whose keys are the
 entries and whose values are the entries' first kv_rank numbers, and the attended latent returns through Wuv_n.  The
 kernels between the products: ``latent_prepare`` (both norms, rotation and store of the shared key part, gate),
-``head_linear`` (the two per-head products, the second with the gate), ``rotate_interleaved`` (the queries'
-rotated part).
+``head_linear`` (the two per-head products, the second with the gate), ``rotate_runs`` (the queries'
+rotated part; pairs are neighbours or halves, as the position encoding says).
 
 Long prompt portions go another way (``expand_keys``): there many queries meet every key, and attention with one
 key/value head of kv_rank + rot numbers costs more per pair than attention with every head's own keys of dim + rot
-and values of vdim.  So the latents of all positions the step's requests hold are gathered from the cache
+and values of vdim.  So the latents of all positions the step's queries may read are gathered from the cache
 (``latent_gather``), one product with [Wuk; Wuv] gives every head's plain key parts and values, ``latent_scatter`` puts
 them into pages of the step's own beside the shared key part, and the ordinary paged attention runs with as many
 key/value heads as heads; the queries then need no Wuk and the attended rows no Wuv, only the gate (``gate_rows``).
@@ -54,12 +54,14 @@ def _sm_count(device) -> int:
 class LatentAttention(Mixer):
     """params: ``hidden_size``, ``heads``, ``head_dim`` (plain query/key numbers per head), ``rope_dim`` (rotated
     ones), ``value_dim``, ``q_rank``, ``kv_rank``, ``scale``, ``eps`` (of the two latent norms), ``gate`` (``"none"``,
-    ``"head"`` or ``"element"``), ``position`` (a PartSpec that offers ``pair_tables()``: the rotation of the rope_dim
-    part), ``shared_kv`` (bool: the entries are another layer's), ``expand_keys`` (``"auto"``: every head's own keys
+    ``"head"`` or ``"element"``), ``position`` (a PartSpec that offers ``pair_tables()`` or ``rotary_tables()``: the
+    rotation of the rope_dim part, of neighbouring pairs or of halves), ``window`` (None, or how many most recent positions a
+    query reads, its own included), ``shared_kv`` (bool: the entries are another layer's), ``expand_keys`` (``"auto"``: every head's own keys
     and values for steps with long portions, where the tensor-core attention takes the sizes; ``"never"``;
     ``"always"``).
     weights: ``dq|uq|dkv|uk|uv|g|o.weight``, ``dq_norm.weight``, ``dkv_norm.weight`` (float32)."""
     graph_safe = True
+    takes_deferred_rows = True
 
     def __init__(self, spec, env):
         super().__init__(spec, env)
@@ -84,15 +86,20 @@ class LatentAttention(Mixer):
             raise ValueError(f"latent_attention: gate {self.gate!r} is none of 'none', 'head', 'element'")
         if not self.eps > 0.0:
             raise ValueError("latent_attention: eps must be positive")
-        if self.kv_rank + self.rot > 256:
-            raise ValueError(f"latent_attention: entries of {self.kv_rank} + {self.rot} numbers exceed the 256 the "
+        if self.kv_rank + self.rot > 640:
+            raise ValueError(f"latent_attention: entries of {self.kv_rank} + {self.rot} numbers exceed the 640 the "
                              f"attention kernels take")
+        self.window = None if p.get("window") is None else int(p["window"])
+        if self.window is not None and self.window <= 0:
+            raise ValueError("latent_attention: a window must be positive")
         position: PartSpec = p.get("position", PartSpec("none"))
         self.position = build_part(POSITIONS, position, env)
-        tables = getattr(self.position, "pair_tables", None)
-        if self.rot and tables is None and position.kind != "none":
-            raise ValueError(f"latent_attention: position encoding '{position.kind}' offers no tables of neighbouring pairs")
-        self.cos, self.sin, self.rot_dims = tables() if (tables is not None and self.rot) else (None, None, 0)
+        pairs = getattr(self.position, "pair_tables", None)
+        tables = pairs() if pairs is not None else self.position.rotary_tables()
+        if self.rot and tables is None:
+            raise ValueError(f"latent_attention: position encoding '{position.kind}' offers no tables")
+        self.halves = pairs is None
+        self.cos, self.sin, self.rot_dims = tables if self.rot else (None, None, 0)
         if self.rot_dims > self.rot:
             raise ValueError("latent_attention: more rotated numbers than the rotated part holds")
         self.graph_safe = bool(self.position.graph_safe)
@@ -142,11 +149,15 @@ class LatentAttention(Mixer):
         in_rows = self.q_rank + (0 if self.shared_kv else self.entry) + self.gate_n
         products = 2.0 * tokens * (in_rows * self.hidden + self.heads * (self.dim + self.rot) * self.q_rank
                                    + self.heads * self.kv_rank * (self.dim + self.vdim) + self.heads * self.vdim * self.hidden)
+        if self.window is not None:
+            if 2.0 * pairs == tokens * (tokens + 1.0):                    # a whole prompt
+                pairs -= max(tokens - self.window, 0) * (tokens - self.window + 1.0) / 2.0
+            pairs = min(pairs, float(tokens) * self.window)
         # per query-key pair: every head's own keys and values (what long portions run) or the entries as one head
         return products + 2.0 * self.heads * min(self.entry + self.kv_rank, self.dim + self.rot + self.vdim) * pairs
 
     def cache_spec(self) -> Optional[PagedCacheSpec]:
-        return PagedCacheSpec(entries=(("kv", (1, self.entry)),), window=None)
+        return PagedCacheSpec(entries=(("kv", (1, self.entry)),), window=self.window)
 
     def attend(self, h: torch.Tensor, ctx: StepContext, cache: LayerCache, out: Optional[torch.Tensor] = None) -> torch.Tensor:
         """Everything up to, not including, the output projection: the gated heads [T, heads * value_dim]."""
@@ -159,7 +170,8 @@ class LatentAttention(Mixer):
         raw = ops.linear(h, self.w_in, None, ops.GEMM_STORE_F32)
         q_latent, gate = ops.latent_prepare(raw, self.q_rank, self.kv_rank, self.rot, self.gate_n, own, self.q_norm_w,
                                             self.kv_norm_w, self.eps, self.cos, self.sin, self.rot_dims, ctx.positions,
-                                            ctx.seq_of_token, table, pages if (own and cache.owner) else None, dtype)
+                                            ctx.seq_of_token, table, pages if (own and cache.owner) else None, dtype,
+                                            halves=self.halves)
         q = ops.linear(q_latent, self.w_uq, None, ops.GEMM_STORE)
         per_head = self.dim + self.rot
         if self.expands(ctx, pages):
@@ -167,8 +179,8 @@ class LatentAttention(Mixer):
         queries = torch.empty((tokens, self.heads * self.entry), dtype=dtype, device=h.device)
         ops.head_linear(q, per_head, self.w_uk_t, queries, self.entry)
         if self.rot:
-            ops.rotate_interleaved(q[:, self.dim:], per_head, queries[:, self.kv_rank:], self.entry, self.heads, self.rot,
-                                   self.cos, self.sin, self.rot_dims, ctx.positions)
+            ops.rotate_runs(q[:, self.dim:], per_head, queries[:, self.kv_rank:], self.entry, self.heads, self.rot,
+                                   self.cos, self.sin, self.rot_dims, ctx.positions, halves=self.halves)
         # single tokens: the decode kernels take the heads that share a key/value head as the rows of one tile of 16,
         # so more heads than that go in equal runs of up to 16 (the entries are few bytes; reading them twice is cheap)
         single = ctx.max_q_len <= 1 and dtype == torch.bfloat16
@@ -179,6 +191,8 @@ class LatentAttention(Mixer):
             # entries this wide leave room for one block of the decode kernel per SM, so the keys are cut into just
             # enough runs to give every SM a block, not into the many short ones that suit narrow heads
             bound = max(ctx.typical_ctx_len or ctx.max_ctx_len, 1)
+            if self.window is not None:
+                bound = min(bound, (-(-self.window // 64) + 1) * 64)
             want = max(_sm_count(h.device) // max(ctx.num_seqs, 1), 1)
             split = max(64 * -(-(-(-bound // want)) // 64), 128)
         attended = torch.empty((tokens, self.heads * self.kv_rank), dtype=dtype, device=h.device)
@@ -186,7 +200,7 @@ class LatentAttention(Mixer):
             n = min(size, self.heads - lo)
             ops.attention(queries[:, lo * self.entry:(lo + n) * self.entry], pages, None, table, ctx.q_start, ctx.start_pos,
                           ctx.positions, ctx.seq_of_token, ctx.num_seqs, ctx.max_q_len, ctx.max_ctx_len, n, 1, self.entry,
-                          self.scale, split_tokens=split, typical_ctx_len=ctx.typical_ctx_len,
+                          self.scale, window=self.window or 0, split_tokens=split, typical_ctx_len=ctx.typical_ctx_len,
                           decode_prefix=ctx.decode_prefix, values_in_keys=self.kv_rank,
                           out=attended[:, lo * self.kv_rank:(lo + n) * self.kv_rank])
         if out is None:
@@ -202,23 +216,29 @@ class LatentAttention(Mixer):
             return False
         if self.expand_keys == "always":
             return True
-        held = sum(s + n for s, n in zip(ctx.host_start_pos, ctx.host_q_lens))
+        held = sum(s - self.first_read(s) + n for s, n in zip(ctx.host_start_pos, ctx.host_q_lens))
         return (self.env.dtype == torch.bfloat16 and ctx.max_q_len >= 32 and held <= 16 * ctx.num_tokens
                 and self.ops.mma_attention_supports(self.dim + self.rot, self.heads, self.heads, pages.shape[2], self.vdim))
 
+    def first_read(self, position: int) -> int:
+        """The first position that a query at ``position`` reads."""
+        return 0 if self.window is None else max(position - self.window + 1, 0)
+
     def own_pages(self, ctx: StepContext, page_size: int, device):
-        """The step's own pages, one run per request: (page owners, page indices, block table [S, most], count); made
-        once per step and shared by the model's layers of this kind."""
-        key = ("latent_own_pages", page_size)
+        """The step's own pages, one run per request, from the page of the first position its queries read on: (page
+        owners, page indices, block table [S, most], count); made once per step and shared by the model's layers of this
+        kind and window."""
+        key = ("latent_own_pages", page_size, self.window)
         if key not in ctx.scratch:
+            skipped = [self.first_read(s) // page_size for s in ctx.host_start_pos]
             counts = [-(-(s + n) // page_size) for s, n in zip(ctx.host_start_pos, ctx.host_q_lens)]
             most = max(counts)
             owners, indices, rows, first = [], [], [], 0
-            for seq, count in enumerate(counts):
-                owners += [seq] * count
-                indices += list(range(count))
-                rows.append(list(range(first, first + count)) + [-1] * (most - count))
-                first += count
+            for seq, (skip, count) in enumerate(zip(skipped, counts)):
+                owners += [seq] * (count - skip)
+                indices += list(range(skip, count))
+                rows.append([-1] * skip + list(range(first, first + count - skip)) + [-1] * (most - count))
+                first += count - skip
             make = lambda values: torch.tensor(values, dtype=torch.int32).to(device, non_blocking=True)
             ctx.scratch[key] = (make(owners), make(indices), make(rows), first)
         return ctx.scratch[key]
@@ -244,11 +264,11 @@ class LatentAttention(Mixer):
         expanded = ops.linear(latents, self.w_ukv, None, ops.GEMM_STORE)
         ops.latent_scatter(expanded, count, self.dim, keys, values)
         queries = torch.empty_like(q)
-        ops.rotate_interleaved(q, per, queries, per, self.heads, per, self.cos, self.sin, self.rot_dims, ctx.positions,
-                               first=self.dim)
+        ops.rotate_runs(q, per, queries, per, self.heads, per, self.cos, self.sin, self.rot_dims, ctx.positions,
+                        first=self.dim, halves=self.halves)
         attended = ops.attention(queries, keys, values, own_table, ctx.q_start, ctx.start_pos, ctx.positions, ctx.seq_of_token,
                                  ctx.num_seqs, ctx.max_q_len, ctx.max_ctx_len, self.heads, self.heads, per, self.scale,
-                                 split_tokens=ctx.attn_split_tokens, typical_ctx_len=ctx.typical_ctx_len,
+                                 window=self.window or 0, split_tokens=ctx.attn_split_tokens, typical_ctx_len=ctx.typical_ctx_len,
                                  decode_prefix=ctx.decode_prefix, out=out)
         mode = {"none": 0, "head": 1, "element": 2}[self.gate]
         return ops.gate_rows(attended, gate, self.heads, mode) if mode else attended

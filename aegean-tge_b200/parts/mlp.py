@@ -46,6 +46,14 @@ class SwiGLU(FeedForward):
     def flops(self, tokens: int, pairs: float) -> float:
         return 2.0 * tokens * 3 * self.inner * self.hidden
 
+    def gated_matrices(self):
+        """(gate and up rows interleaved [2 inner, hidden], down [hidden, inner]), for a part that runs them with its own."""
+        return self.w_gate_up, self.w_down
+
+    def adopt_matrices(self, gate_up: torch.Tensor, down: torch.Tensor) -> None:
+        """The matrices now live inside tensors of another part's (same values): use those."""
+        self.w_gate_up, self.w_down = gate_up, down
+
     def forward(self, h: torch.Tensor, ctx: StepContext) -> torch.Tensor:
         a = self.ops.linear(h, self.w_gate_up, None, self.ops.GEMM_SWIGLU)
         return self.ops.linear(a, self.w_down, None, self.ops.GEMM_STORE)

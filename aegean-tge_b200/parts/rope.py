@@ -34,21 +34,41 @@ def rescale_by_wavelength(freq: torch.Tensor, factor: float, low: float, high: f
     return torch.where(wavelength < original / high, freq, out)
 
 
+def stretch_by_turns(freq: torch.Tensor, theta: float, dims: int, factor: float, fast: float, slow: float,
+                     original: float) -> torch.Tensor:
+    """Frequencies (float64) for contexts ``factor`` times ``original`` positions: pair i turns t(i) = original f_i / (2 pi)
+    times over the original positions, and i as a function of t is dims ln(original / (2 pi t)) / (2 ln theta).  Pairs up to
+    that place for ``fast`` turns (rounded down, at least 0) keep their frequency, those from the place for ``slow`` turns
+    (rounded up, at most dims - 1) on have it divided by ``factor``, and between the two places the blend is linear."""
+    def place(turns: float) -> float:
+        return dims * math.log(original / (2.0 * math.pi * turns)) / (2.0 * math.log(theta))
+    lo = max(math.floor(place(fast)), 0)
+    hi = min(math.ceil(place(slow)), dims - 1)
+    ramp = ((torch.arange(freq.numel(), dtype=torch.float64) - lo) / max(hi - lo, 0.001)).clamp(0.0, 1.0)
+    return freq / factor * ramp + freq * (1.0 - ramp)
+
+
 def rotary_tables(theta: float, rotary: int, positions: int,
                   scaling: Optional[Tuple[float, float, float, float]] = None,
-                  precise: bool = False) -> Tuple[torch.Tensor, torch.Tensor]:
+                  precise: bool = False,
+                  stretch: Optional[Tuple[float, float, float, float]] = None) -> Tuple[torch.Tensor, torch.Tensor]:
     """cos and sin of position * frequency, float32 [positions, rotary/2].  By default the exponent, the
     frequency and the angle are each rounded to float32 as described above; with ``precise`` all of it is
     float64 and only the cosine and the sine are rounded (an angle of a thousand radians in float32 is already
-    off by 6e-5)."""
+    off by 6e-5).  ``stretch`` (factor, fast, slow, original; with ``precise``): frequencies by :func:`stretch_by_turns`,
+    cosine and sine times 0.1 ln(factor) + 1."""
     half = rotary // 2
     if precise:
         index = torch.arange(half, dtype=torch.float64)
         freq = torch.pow(torch.tensor(theta, dtype=torch.float64), -2.0 * index / float(rotary))
         if scaling is not None:
             freq = rescale_by_wavelength(freq, *scaling)
+        amplitude = 1.0
+        if stretch is not None:
+            freq = stretch_by_turns(freq, theta, rotary, *stretch)
+            amplitude = 0.1 * math.log(stretch[0]) + 1.0
         angle = torch.arange(positions, dtype=torch.float64)[:, None] * freq[None, :]
-        return torch.cos(angle).float(), torch.sin(angle).float()
+        return (amplitude * torch.cos(angle)).float(), (amplitude * torch.sin(angle)).float()
     index = torch.arange(half, dtype=torch.float32)
     exponent = (-2.0 * index) / torch.tensor(float(rotary), dtype=torch.float32)          # float32
     theta32 = torch.tensor(theta, dtype=torch.float32)
@@ -67,7 +87,9 @@ _TABLES: dict = {}
 class RotaryNeoX(PositionEncoding):
     """params: ``head_dim``, ``theta``, optional ``rotary_dim`` (default head_dim), optional ``scaling``
     (``{"factor", "low", "high", "original"}``: frequencies rescaled by wavelength, see
-    :func:`rescale_by_wavelength`), optional ``precise`` (tables from float64 angles)."""
+    :func:`rescale_by_wavelength`), optional ``stretch`` (``{"factor", "fast", "slow", "original"}``: frequencies stretched
+    for long contexts, see :func:`stretch_by_turns`; the rotation then also scales what it turns; goes with ``precise``),
+    optional ``precise`` (tables from float64 angles)."""
     graph_safe = True
 
     def __init__(self, spec, env):
@@ -88,11 +110,17 @@ class RotaryNeoX(PositionEncoding):
                 raise ValueError(f"rope: scaling {scaling!r} needs factor > 0, original > 0 and high > low >= 0")
         # layers with the same base, width and length share one pair of tables
         self.precise = bool(spec.params.get("precise", False))
-        key = (self.theta, self.rotary, env.max_positions, str(env.device), self.scaling, self.precise)
+        stretch = spec.params.get("stretch")
+        self.stretch = None
+        if stretch is not None:
+            self.stretch = tuple(float(stretch[name]) for name in ("factor", "fast", "slow", "original"))
+            if not min(self.stretch) > 0 or self.theta == 1.0 or not self.precise or self.scaling is not None:
+                raise ValueError(f"rope: stretch {stretch!r} needs positive numbers, theta other than 1, precise tables and no scaling")
+        key = (self.theta, self.rotary, env.max_positions, str(env.device), self.scaling, self.precise, self.stretch)
         if key not in _TABLES:
             if len(_TABLES) >= 8:
                 _TABLES.pop(next(iter(_TABLES)))
-            cos, sin = rotary_tables(self.theta, self.rotary, env.max_positions, self.scaling, self.precise)
+            cos, sin = rotary_tables(self.theta, self.rotary, env.max_positions, self.scaling, self.precise, self.stretch)
             _TABLES[key] = (cos.to(env.device).contiguous(), sin.to(env.device).contiguous())
         self.cos, self.sin = _TABLES[key]
 
@@ -150,7 +178,7 @@ class RotaryInterleaved(PositionEncoding):
                 # a view into a wider row (q or k inside a q/k/v row): rows stay dense, heads follow one another
                 flat = t.as_strided((tokens, heads * dim), (t.stride(0), 1))
             before = flat.clone()
-            self.ops.rotate_interleaved(before, dim, flat, dim, heads, dim, self.cos, self.sin, self.rotary, positions)
+            self.ops.rotate_runs(before, dim, flat, dim, heads, dim, self.cos, self.sin, self.rotary, positions)
 
 
 @POSITIONS.register("none")

@@ -8,10 +8,13 @@ With h the input, R = experts + identity router outputs:
     w_k = s_k / (sum of the chosen s + 1e-20)
     out = sum_k w_k E_k(h)      E_e(h) = Wdown_e relu(Wup_e h)^2 for an expert, h itself for an identity output
 
-Parameters change four things: the scores may be each output's own logistic function instead of the softmax; the weights
-the chosen scores as they are instead of over their sum; a weight may multiply its expert's INPUT, E(w h), instead of the
-output; and an expert may be a clamped gated feed-forward, Wdown (g sigmoid(alpha g) (u + offset)) with g = min(Wgate h, L)
-and u = clamp(Wup h, -L, L), its gate and up rows interleaved in one matrix.
+Parameters change six things: the scores may be each output's own logistic function instead of the softmax; the weights
+the chosen scores as they are instead of over their sum, and all times a constant; a weight may multiply its expert's INPUT,
+E(w h), instead of the output; a group's value may be the sum of its two largest choice values; an expert may be a gated
+feed-forward, Wdown (silu(Wgate h) Wup h), or a clamped gated one, Wdown (g sigmoid(alpha g) (u + offset)) with g =
+min(Wgate h, L) and u = clamp(Wup h, -L, L), gate and up rows interleaved in one matrix (the plain gate is the clamped one
+with L infinite, alpha 1 and offset 0); and the feed-forward that every token uses may be multiplied by one gate per token,
+sigmoid(wg h).  That gate's row lies below the router's in one matrix.
 
 The correction steers the choice only; the weights use the plain scores.  Identity outputs are the last ``identity``
 router outputs and have no tensors.  The sum over a token's choices is formed in float32 in the order of the choice
@@ -28,10 +31,14 @@ both can be captured into a CUDA graph.  A step of many tokens groups the pairs 
 expert and projection over that expert's block of rows (``experts_group`` -> products ->
 ``experts_combine_add``); the host reads the group sizes, which a step with prompt portions may do.
 
+On the dense path a gated feed-forward that every token uses is one expert more: its rows lie below the experts' in the up
+matrix and beside them in the down matrix, and the kernel between the products multiplies its values by the token's gate.
+
 The down matrices are kept side by side, [hidden, experts, inner]: expert e's matrix is the strided view [:, e, :].
 """
 from __future__ import annotations
 
+import math
 from typing import Dict, List, Optional
 
 import torch
@@ -47,8 +54,9 @@ class RoutedExperts(FeedForward):
     """params: ``hidden_size``, ``intermediate_size`` (an expert's inner width), ``experts``, ``top``, optional
     ``identity`` (default 0), ``group_count`` / ``group_keep`` (default 1 / 1: no groups), ``correction`` (bool,
     default True: the checkpoint holds a correction of the choice), ``activation`` (``"relu_squared"`` or
-    ``"clamped_glu"``, the latter with ``limit`` and optionally ``alpha``, default 1.702, and ``up_offset``, default 1),
-    ``score`` (``"softmax"`` or ``"logistic"``), ``weights_over_sum`` (bool, default True), ``weigh`` (``"output"`` or
+    ``"clamped_glu"``, the latter with ``limit`` and optionally ``alpha``, default 1.702, and ``up_offset``, default 1, or
+    ``"swiglu"``), ``group_value`` (``"best"`` or ``"two_best"``), ``weights_scale`` (default 1), ``shared_gate`` (bool, default
+    False: one logistic gate per token on the shared feed-forward; parameter ``shared_gate.weight`` [1, hidden]), ``score`` (``"softmax"`` or ``"logistic"``), ``weights_over_sum`` (bool, default True), ``weigh`` (``"output"`` or
     ``"input"``; the latter without identity experts), ``router_bias`` (bool, default False: a bias added to the router's logits, so it
     steers the choice and the weights alike), ``shared`` (None, or the PartSpec of a feed-forward that every token
     uses and whose output is added; its parameters are this part's under ``shared.<local name>``).
@@ -75,6 +83,15 @@ class RoutedExperts(FeedForward):
         self.shared: Optional[FeedForward] = build_part(FEED_FORWARDS, shared, env) if shared is not None else None
         if self.shared is not None:
             self.graph_safe = bool(self.shared.graph_safe)
+        self.shared_gate = bool(p.get("shared_gate", False))
+        if self.shared_gate and self.shared is None:
+            raise ValueError("routed_experts: a gate on the shared feed-forward needs one")
+        group_value = str(p.get("group_value", "best"))
+        if group_value not in ("best", "two_best"):
+            raise ValueError(f"routed_experts: group_value {group_value!r} is 'best' or 'two_best'")
+        self.group_pairs = group_value == "two_best"
+        self.weights_scale = float(p.get("weights_scale", 1.0))
+        self.shared_inner = 0                  # inner width of a shared feed-forward that runs as one expert more
         self.router_bias: Optional[torch.Tensor] = None
         self.outputs = self.experts + self.identity
         activation = str(p.get("activation", "relu_squared"))
@@ -83,6 +100,8 @@ class RoutedExperts(FeedForward):
             self.gate = (float(p["limit"]), float(p.get("alpha", 1.702)), float(p.get("up_offset", 1.0)))
             if not self.gate[0] > 0.0:
                 raise ValueError("routed_experts: the limit must be positive")
+        elif activation == "swiglu":
+            self.gate = (math.inf, 1.0, 0.0)
         elif activation != "relu_squared":
             raise ValueError(f"routed_experts: unknown activation '{p.get('activation')}'")
         self.matrices = 2 if self.gate is None else 3
@@ -106,6 +125,8 @@ class RoutedExperts(FeedForward):
         self.correction: Optional[torch.Tensor] = None
         self.w_up: Optional[torch.Tensor] = None         # [experts, inner, hidden]; gated: [experts, 2 inner, hidden]
         self.w_down: Optional[torch.Tensor] = None       # [hidden, experts, inner]
+        self.up_rows: Optional[torch.Tensor] = None      # all up (and gate) rows, a joined shared feed-forward's last
+        self.down_columns: Optional[torch.Tensor] = None # all down matrices side by side, likewise
 
     def param_specs(self) -> Dict[str, ParamSpec]:
         specs = {"router.weight": ParamSpec((self.outputs, self.hidden))}
@@ -113,6 +134,8 @@ class RoutedExperts(FeedForward):
             specs["correction"] = ParamSpec((self.outputs,), role="vector")
         if self.has_router_bias:
             specs["router.bias"] = ParamSpec((self.outputs,), role="vector")
+        if self.shared_gate:
+            specs["shared_gate.weight"] = ParamSpec((1, self.hidden))
         if self.shared is not None:
             specs.update({f"shared.{local}": param for local, param in self.shared.param_specs().items()})
         for e in range(self.experts):
@@ -124,8 +147,15 @@ class RoutedExperts(FeedForward):
 
     def load(self, tensors: Dict[str, torch.Tensor]) -> None:
         self.w_router = tensors["router.weight"].contiguous()
+        if self.shared_gate:
+            # the gate's row below the router's, and rows of zeros up to a multiple of four (rows of logits on 16 bytes)
+            gate = tensors["shared_gate.weight"]
+            spare = gate.new_zeros((-(self.outputs + 1) % 4, self.hidden))
+            self.w_router = torch.cat([self.w_router, gate, spare], dim=0).contiguous()
         self.correction = tensors["correction"].contiguous() if self.has_correction else None
         self.router_bias = tensors["router.bias"].contiguous() if self.has_router_bias else None
+        if self.router_bias is not None and self.shared_gate:
+            self.router_bias = torch.cat([self.router_bias, self.router_bias.new_zeros(self.w_router.shape[0] - self.outputs)])
         if self.shared is not None:
             self.shared.load({name[len("shared."):]: t for name, t in tensors.items() if name.startswith("shared.")})
         if self.experts:
@@ -135,9 +165,26 @@ class RoutedExperts(FeedForward):
                 self.w_up = torch.stack([torch.stack([tensors[f"experts.{e}.gate.weight"], tensors[f"experts.{e}.up.weight"]], dim=1)
                                          .reshape(2 * self.inner_size, self.hidden) for e in range(self.experts)]).contiguous()
             self.w_down = torch.stack([tensors[f"experts.{e}.down.weight"] for e in range(self.experts)], dim=1).contiguous()
+            self.up_rows = self.w_up.view(-1, self.hidden)
+            self.down_columns = self.w_down.view(self.hidden, -1)
+            self.join_shared()
         else:
             self.w_up = torch.empty((0, self.inner_size, self.hidden), dtype=self.w_router.dtype, device=self.w_router.device)
             self.w_down = torch.empty((self.hidden, 0, self.inner_size), dtype=self.w_router.dtype, device=self.w_router.device)
+
+    def join_shared(self) -> None:
+        """A gated feed-forward that every token uses becomes the last block of the experts' matrices."""
+        matrices = getattr(self.shared, "gated_matrices", None)
+        if matrices is None or self.gate is None or self.gate[1:] != (1.0, 0.0) or self.weigh_input:
+            return
+        gate_up, down = matrices()
+        routed = self.experts * self.inner_size
+        self.shared_inner = down.shape[1]
+        self.up_rows = torch.cat([self.up_rows, gate_up], dim=0).contiguous()
+        self.down_columns = torch.cat([self.down_columns, down], dim=1).contiguous()
+        self.w_up = self.up_rows[:2 * routed].view(self.experts, 2 * self.inner_size, self.hidden)
+        self.w_down = self.down_columns[:, :routed].unflatten(1, (self.experts, self.inner_size))
+        self.shared.adopt_matrices(self.up_rows[2 * routed:], self.down_columns[:, routed:])
 
     def param_bytes(self) -> int:
         """What one token's step reads: the router and the chosen experts (a large batch touches more of them)."""
@@ -166,12 +213,34 @@ class RoutedExperts(FeedForward):
         complete = getattr(h, "complete", None)
         if complete is not None:
             h = complete()
+        return (h, *self.choose(h)[:2])
+
+    def choose(self, h: torch.Tensor):
+        """(ids, weights, the gate logits of the shared feed-forward [T] or None); the rows may lack their norm factor."""
         logits = self.ops.linear(h, self.w_router, self.router_bias, self.ops.GEMM_STORE_F32)
         ids, weights = self.ops.router_topk(logits, self.correction, self.top, self.group_count, self.group_keep,
-                                            logistic=self.logistic, over_sum=self.over_sum)
-        return h, ids, weights
+                                            logistic=self.logistic, over_sum=self.over_sum, group_pairs=self.group_pairs,
+                                            factor=self.weights_scale, outputs=self.outputs)
+        return ids, weights, logits[:, self.outputs] if self.shared_gate else None
+
+    def takes_deferred_at(self, tokens: int) -> bool:
+        # on the dense path two products read the rows, and nothing else does
+        return self.gate is not None and self.dense(tokens) and (self.shared is None or self.shared_inner > 0)
+
+    def last_product(self, h: torch.Tensor, ctx: StepContext):
+        """On the dense path of gated experts everything ends in one product with all down matrices."""
+        ops, tokens = self.ops, h.shape[0]
+        if not self.takes_deferred_at(tokens):
+            return None
+        ids, weights, gate = self.choose(h)
+        z = ops.linear(h, self.up_rows, None, ops.GEMM_STORE)
+        a = ops.experts_dense_gate(z, ids, weights, self.experts, self.gate, self.weigh_input, self.shared_inner, gate)
+        return a, self.down_columns
 
     def forward_add(self, h: torch.Tensor, x: torch.Tensor, ctx: StepContext, next_norm=None):
+        if self.shared_gate:
+            self.ops.add_to_stream(x, self.forward_f32(h, ctx))
+            return None
         h = self.add_routed(h, x, ctx)
         if self.shared is not None:
             # the feed-forward every token uses adds last, and with it whatever it can do for the next norm
@@ -179,35 +248,43 @@ class RoutedExperts(FeedForward):
         return None
 
     def add_routed(self, h: torch.Tensor, x: torch.Tensor, ctx: StepContext) -> torch.Tensor:
-        """Adds the chosen experts' weighted outputs into ``x``; returns the rows as the experts read them."""
+        """Adds the chosen experts' weighted outputs into ``x`` (with a gate on the shared feed-forward, whose output ``x``
+        then holds: into gate * x); returns the rows as the experts read them."""
         ops = self.ops
-        h, ids, weights = self.route(h)
+        complete = getattr(h, "complete", None)
+        h = h if complete is None else complete()
+        ids, weights, x_gate = self.choose(h)
         tokens = h.shape[0]
         few = ctx.max_q_len <= 1 or tokens <= DIRECT_MAX_TOKENS
-        if self.dense(tokens) and self.gate is not None:
+        if self.dense(tokens) and self.gate is not None and x_gate is None:
             z = ops.linear(h, self.w_up.view(self.experts * 2 * self.inner_size, self.hidden), None, ops.GEMM_STORE)
             a = ops.experts_dense_gate(z, ids, weights, self.experts, self.gate, self.weigh_input)
             ops.linear(a, self.w_down.view(self.hidden, self.experts * self.inner_size), None, ops.GEMM_ADD_F32, out=x)
             return h
-        if self.dense(tokens):
+        if self.dense(tokens) and self.gate is None and x_gate is None:
             z = ops.linear(h, self.w_up.view(self.experts * self.inner_size, self.hidden), None, ops.GEMM_STORE)
             ops.experts_dense_weigh(z, ids, weights, h, x, self.experts)
             ops.linear(z, self.w_down.view(self.hidden, self.experts * self.inner_size), None, ops.GEMM_ADD_F32, out=x)
             return h
         if few or self.experts == 0:
-            ops.experts_direct(h, self.w_up, self.w_down, ids, weights, x, gate=self.gate, weigh_input=self.weigh_input)
+            ops.experts_direct(h, self.w_up, self.w_down, ids, weights, x, gate=self.gate, weigh_input=self.weigh_input,
+                               x_gate=x_gate)
             return h
         place, offsets, grouped = ops.experts_group(h, ids, self.experts, in_weights=weights if self.weigh_input else None)
         bounds: List[int] = offsets.tolist()             # the host learns the group sizes: not a captured step
         rows = bounds[-1]
         inner = torch.empty((max(rows, 1), self.inner_size), dtype=h.dtype, device=h.device)
         outputs = torch.empty((max(rows, 1), self.hidden), dtype=torch.float32, device=h.device)
-        fused = self.gate is not None and self.gate[1:] == (1.702, 1.0)      # the gate is the product's own epilogue
+        # the gate is the product's own epilogue, where it has it
+        fused = {(1.702, 1.0): ops.GEMM_GLU_CLAMPED, (1.0, 0.0): ops.GEMM_SWIGLU}.get(self.gate[1:] if self.gate else None)
+        if fused == ops.GEMM_SWIGLU and self.gate[0] != math.inf:
+            fused = None
         for e in range(self.experts):
             lo, hi = bounds[e], bounds[e + 1]
             if hi > lo:
-                if fused:
-                    ops.linear(grouped[lo:hi], self.w_up[e], None, ops.GEMM_GLU_CLAMPED, out=inner[lo:hi], alpha=self.gate[0])
+                if fused is not None:
+                    ops.linear(grouped[lo:hi], self.w_up[e], None, fused, out=inner[lo:hi],
+                               alpha=self.gate[0] if fused == ops.GEMM_GLU_CLAMPED else 1.0)
                 elif self.gate is not None:
                     both = ops.linear(grouped[lo:hi], self.w_up[e], None, ops.GEMM_STORE_F32)
                     ops.gated_clamp_act(both, *self.gate, self.env.dtype, out=inner[lo:hi])
@@ -219,10 +296,13 @@ class RoutedExperts(FeedForward):
             lo, hi = bounds[e], bounds[e + 1]
             if hi > lo:
                 ops.linear(inner[lo:hi], self.w_down[:, e, :], None, ops.GEMM_STORE_F32, out=outputs[lo:hi])
-        ops.experts_combine_add(outputs, place, None if self.weigh_input else weights, h, x)
+        ops.experts_combine_add(outputs, place, None if self.weigh_input else weights, h, x, x_gate=x_gate)
         return h
 
     def forward_f32(self, h: torch.Tensor, ctx: StepContext) -> torch.Tensor:
+        last = self.last_product(h, ctx) if self.shared_inner else None
+        if last is not None:
+            return self.ops.linear(last[0], last[1], None, self.ops.GEMM_STORE_F32)
         if self.shared is not None:
             # the feed-forward every token uses writes the rows, the chosen experts add to them
             complete = getattr(h, "complete", None)

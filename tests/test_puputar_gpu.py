@@ -311,7 +311,7 @@ def test_rotation_of_neighbouring_pairs(ops, dtype, heads, width, dims, base):
     src = torch.randn(len(positions), heads * stride, generator=gen).to(TORCH[dtype])
     cos, sin = pair_tables(base, dims, 2000)
     dst = torch.zeros(len(positions), heads * width, dtype=TORCH[dtype], device=DEV)
-    ops.rotate_interleaved(src.to(DEV)[:, 5:], stride, dst, width, heads, width, cos.to(DEV), sin.to(DEV), dims, _i32(positions))
+    ops.rotate_runs(src.to(DEV)[:, 5:], stride, dst, width, heads, width, cos.to(DEV), sin.to(DEV), dims, _i32(positions))
     runs = src.double().view(len(positions), heads, stride)[:, :, 5:]
     ref = torch.from_numpy(plain.rotate_pairs(runs.numpy(), positions, base, dims)).reshape(len(positions), heads * width)
     assert rel_error(dst, ref) < KERNEL_TOL[dtype]
@@ -323,7 +323,7 @@ def test_rotation_of_neighbouring_pairs(ops, dtype, heads, width, dims, base):
         moved = torch.cat([runs[..., dims:], runs[..., :dims]], dim=-1).to(TORCH[dtype])
         want = torch.cat([ref.view(len(positions), heads, width)[..., dims:], ref.view(len(positions), heads, width)[..., :dims]], dim=-1)
         back = torch.zeros(len(positions), heads * width, dtype=TORCH[dtype], device=DEV)
-        ops.rotate_interleaved(moved.reshape(len(positions), -1).to(DEV), width, back, width, heads, width, cos.to(DEV), sin.to(DEV), dims,
+        ops.rotate_runs(moved.reshape(len(positions), -1).to(DEV), width, back, width, heads, width, cos.to(DEV), sin.to(DEV), dims,
                                _i32(positions), first=lead)
         assert rel_error(back, want.reshape(len(positions), -1)) < KERNEL_TOL[dtype]
     # the halves-paired rotation is another function: it must differ
