@@ -231,7 +231,28 @@ def paired_configs(width: int, heads: int, kv_heads: int, head_dim: int, gated_i
     return {"qwen2": qwen2, "lepizen": lepizen, "mozepel": mozepel_config(width, heads, kv_heads, head_dim, gated_inner, layers, vocab),
             "puputar": puputar_config(width, heads, head_dim, gated_inner, layers, vocab),
             "kokolorn": kokolorn_config(width, heads, kv_heads, head_dim, gated_inner, layers, vocab),
-            "fesorax": fesorax_config(width, heads, kv_heads, head_dim, gated_inner, layers, vocab)}
+            "fesorax": fesorax_config(width, heads, kv_heads, head_dim, gated_inner, layers, vocab),
+            "tazizen": tazizen_config(width, heads, kv_heads, head_dim, gated_inner, layers, vocab)}
+
+
+def tazizen_config(width: int, heads: int, kv_heads: int, head_dim: int, gated_inner: int, layers: int, vocab: int,
+                   experts: int = 16, top: int = 4, streams: int = 4, window: int = 1024) -> dict:
+    """A Tazizen config.json with the width, heads, kv heads, head size and layer count of a Qwen2 shape: ``streams`` residual
+    streams; layers by turns latent attention (as in :func:`puputar_config`) and attention (the shape's GQA, half of each head
+    rotated with stretched frequencies), both over a window; every layer with ``experts`` gated experts in four groups of
+    which two are kept, three sixteenths of the gated inner width each, of which ``top`` are used, and a shared one of a
+    quarter of it: as many multiplications per token as the dense feed-forward; one pass over all layers."""
+    unit, rot = max(gated_inner // 16 // 64 * 64, 64), head_dim // 2
+    moe = {"kind": "moe", "expert": {"ff": 3 * unit}, "shared": {"ff": 4 * unit},
+           "router": {"experts": experts, "top": top, "scale": 2.0, "groups": {"count": 4, "keep": 2}}}
+    latent = {"heads": heads, "dim": head_dim - rot, "rot_dim": rot, "vdim": head_dim, "q_rank": max(width // 4 // 64 * 64, 64),
+              "kv_rank": 192, "scale": head_dim ** -0.5, "rot": {"base": 500000.0, "dims": rot}, "mask": {"size": window}}
+    attention = {"heads": heads, "kv_heads": kv_heads, "dim": head_dim, "vdim": head_dim, "scale": head_dim ** -0.5,
+                 "rot": {"base": 500000.0, "dims": rot, "scaling": {"factor": 8.0, "original": 4096, "fast": 32.0, "slow": 1.0}},
+                 "mask": {"size": window}}
+    kinds = [{"type": "latent_attention", "mixer": latent, "mlp": moe}, {"type": "attention", "mixer": attention, "mlp": moe}]
+    return {"architecture": "Tazizen", "vocab": vocab, "width": width, "streams": streams, "norm": {"eps": 1e-6},
+            "layers": [kinds[n % 2] for n in range(layers)]}
 
 
 def fesorax_config(width: int, heads: int, kv_heads: int, head_dim: int, gated_inner: int, layers: int, vocab: int,

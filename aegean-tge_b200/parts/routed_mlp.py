@@ -208,15 +208,9 @@ class RoutedExperts(FeedForward):
         extra = self.shared.flops(tokens, pairs) if self.shared is not None else 0.0
         return 2.0 * tokens * (self.outputs * self.hidden + self.top * self.matrices * self.inner_size * self.hidden) + extra
 
-    def route(self, h: torch.Tensor):
-        """(ids int32 [T, top], weights float32 [T, top]); the logits are a float32 product of the rows as given."""
-        complete = getattr(h, "complete", None)
-        if complete is not None:
-            h = complete()
-        return (h, *self.choose(h)[:2])
-
-    def choose(self, h: torch.Tensor):
-        """(ids, weights, the gate logits of the shared feed-forward [T] or None); the rows may lack their norm factor."""
+    def route(self, h):
+        """(ids int32 [T, top], weights float32 [T, top], the gate logits of the shared feed-forward [T] or None); the logits
+        are a float32 product of the rows as given, which may lack their norm's factor."""
         logits = self.ops.linear(h, self.w_router, self.router_bias, self.ops.GEMM_STORE_F32)
         ids, weights = self.ops.router_topk(logits, self.correction, self.top, self.group_count, self.group_keep,
                                             logistic=self.logistic, over_sum=self.over_sum, group_pairs=self.group_pairs,
@@ -232,7 +226,7 @@ class RoutedExperts(FeedForward):
         ops, tokens = self.ops, h.shape[0]
         if not self.takes_deferred_at(tokens):
             return None
-        ids, weights, gate = self.choose(h)
+        ids, weights, gate = self.route(h)
         z = ops.linear(h, self.up_rows, None, ops.GEMM_STORE)
         a = ops.experts_dense_gate(z, ids, weights, self.experts, self.gate, self.weigh_input, self.shared_inner, gate)
         return a, self.down_columns
@@ -253,7 +247,7 @@ class RoutedExperts(FeedForward):
         ops = self.ops
         complete = getattr(h, "complete", None)
         h = h if complete is None else complete()
-        ids, weights, x_gate = self.choose(h)
+        ids, weights, x_gate = self.route(h)
         tokens = h.shape[0]
         few = ctx.max_q_len <= 1 or tokens <= DIRECT_MAX_TOKENS
         if self.dense(tokens) and self.gate is not None and x_gate is None:

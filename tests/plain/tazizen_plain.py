@@ -156,35 +156,42 @@ def group_values(choice: np.ndarray, count: int) -> np.ndarray:
 
 
 def route(h: np.ndarray, router: np.ndarray, correction: np.ndarray, top: int, count: int, keep: int, scale: float,
-          margins: Optional[List[float]] = None):
-    """-> (ids [T, top], weights [T, top]).  ``margins`` receives per token how far the choice is from another one."""
+          margins: Optional[List[float]] = None, choices: Optional[np.ndarray] = None):
+    """-> (ids [T, top], weights [T, top]).  ``margins`` receives per token how far the choice is from another one.
+    ``choices`` [T, top]: these experts instead, with their own scores; a margin is then negative by how much the choice
+    scores (or group values) would have to move for it."""
     s = sigmoid(h @ router.T)
     ids, weights = [], []
     for t in range(h.shape[0]):
         choice = s[t] + correction
         per = choice.size // count
         values = group_values(choice, count)
-        order = np.argsort(-values, kind="stable")
+        order = list(np.argsort(-values, kind="stable"))
+        if choices is not None:
+            taken = {int(e) // per for e in choices[t]}
+            order.sort(key=lambda g: g not in taken)               # the groups of the experts taken first
         allowed = np.full(choice.size, -np.inf)
         for g in order[:keep]:
             allowed[g * per:(g + 1) * per] = choice[g * per:(g + 1) * per]
-        chosen = np.argsort(-allowed, kind="stable")
-        ids.append(chosen[:top])
-        w = s[t, chosen[:top]]
+        chosen = np.argsort(-allowed, kind="stable")[:top] if choices is None else np.asarray(choices[t], dtype=np.int64)
+        ids.append(chosen)
+        w = s[t, chosen]
         weights.append(w / (w.sum() + 1e-20) * scale)
         if margins is not None:
-            gap = np.inf if keep >= count else values[order[keep - 1]] - values[order[keep]]
-            if top < keep * per:
-                gap = min(gap, allowed[chosen[top - 1]] - allowed[chosen[top]])
+            gap = np.inf if keep >= count else values[order[:keep]].min() - values[order[keep:]].max()
+            left = np.delete(allowed, chosen)
+            if left.size and np.isfinite(left.max()):
+                gap = min(gap, allowed[chosen].min() - left.max())
             margins.append(float(gap))
     return np.array(ids), np.array(weights)
 
 
-def experts(h: np.ndarray, W: Dict[str, np.ndarray], p: str, mlp: dict, margins: Optional[List[float]] = None) -> np.ndarray:
+def experts(h: np.ndarray, W: Dict[str, np.ndarray], p: str, mlp: dict, margins: Optional[List[float]] = None,
+            choices: Optional[np.ndarray] = None) -> np.ndarray:
     r = mlp["router"]
     groups = r.get("groups") or {"count": 1, "keep": 1}
     ids, weights = route(h, W[p + "router"], W[p + "correction"], r["top"], groups["count"], groups["keep"], r.get("scale", 1.0),
-                         margins)
+                         margins, choices)
     out = np.zeros_like(h)
     for e in range(r["experts"]):
         rows, places = np.nonzero(ids == e)
@@ -204,13 +211,15 @@ def run_order(config: dict) -> List[int]:
     return list(range(loop["start"])) + once * loop["times"] + list(range(loop["stop"], n))
 
 
-def forward(config: dict, weights: Dict[str, np.ndarray], tokens, return_layers: bool = False, margins: Optional[list] = None):
+def forward(config: dict, weights: Dict[str, np.ndarray], tokens, return_layers: bool = False, margins: Optional[list] = None,
+            choices: Optional[list] = None):
     """Logits [T, vocab] of a whole sequence (and, on request, the sum of the streams after every layer run [runs, T,
-    width]).  ``margins``: a list that receives the [T] choice margins of every routed layer run."""
+    width]).  ``margins``: a list that receives the [T] choice margins of every routed layer run; ``choices``: the experts
+    every routed layer run takes, [T, top] each."""
     W = {name: np.asarray(t, dtype=F) for name, t in weights.items()}
     eps = config["norm"]["eps"]
     X = np.repeat(W["embed"][np.asarray(tokens)][:, None, :], config["streams"], axis=1)
-    kept = []
+    kept, routed = [], 0
     for n in run_order(config):
         layer, p = config["layers"][n], f"l{n}."
         mixer = {"attention": attention, "latent_attention": latent_attention}[layer["type"]]
@@ -218,7 +227,9 @@ def forward(config: dict, weights: Dict[str, np.ndarray], tokens, return_layers:
         X = streams_out(X, y, W[p + "hc1.mix"], W[p + "hc1.out"])
         if layer.get("mlp") is not None:
             found = None if margins is None else []
-            y = experts(norm_around_one(streams_in(X, W[p + "hc2.in"]), W[p + "norm2"], eps), W, p + "mlp.", layer["mlp"], found)
+            y = experts(norm_around_one(streams_in(X, W[p + "hc2.in"]), W[p + "norm2"], eps), W, p + "mlp.", layer["mlp"], found,
+                        None if choices is None else choices[routed])
+            routed += 1
             X = streams_out(X, y, W[p + "hc2.mix"], W[p + "hc2.out"])
             if margins is not None:
                 margins.append(np.array(found))

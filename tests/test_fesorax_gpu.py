@@ -218,9 +218,9 @@ class _Run:
         seen, route = [], RoutedExperts.route
 
         def recording(part, h):
-            h, ids, weights = route(part, h)
-            seen.append(ids.cpu().numpy())
-            return h, ids, weights
+            chosen = route(part, h)
+            seen.append(chosen[0].cpu().numpy())
+            return chosen
         if self.record:
             RoutedExperts.route = recording
         try:
