@@ -71,6 +71,9 @@ struct AttnParams {
   int early_tiles;           // decode: key tiles of settled positions asked for before the dependency wait (0: none)
   int heads, kv_heads, group, bq;
   int window, split_tokens, num_splits;
+  int window_runs;           // single tokens over a window: the key runs are counted from the window's start, not from position 0
+  int kv_pool;               // key/value heads of the pages: kv_heads, or 1 when all runs of heads read the same one
+  int v_in_keys;             // a position's value is the leading part of its key
   int keep_first;            // with a window: the first so many positions stay visible (0: none)
   const __nv_bfloat16* gate; // null, or [tokens, heads] logits: a head's output is multiplied by their logistic function
   int gate_stride;
@@ -85,6 +88,10 @@ __device__ __forceinline__ float distance_bias(const AttnParams& p, int head, in
   return p.dist_bias[(size_t)head * p.dist_span + min(max(distance, 0), p.dist_span - 1)] * LOG2E;
 }
 
+// Where the key runs of a single token at `pos` start counting: at the tile that holds its window's first position (no
+// window given: at position 0).
+__device__ __forceinline__ int run_base(int window, int pos) { return window > 0 ? max(pos - window + 1, 0) / BKV * BKV : 0; }
+
 // The keys a block visits, in its run [first, last) of positions (the whole request when the keys are not cut): the tiles
 // of the kept first tokens, then those from the start of the window (of the block's first query) on.
 struct KeyTiles {
@@ -94,7 +101,7 @@ struct KeyTiles {
   __device__ __forceinline__ KeyTiles(const AttnParams& p, int pos0, int q_count, int split) {
     int first = 0, last = 0x7fffffff;
     if (p.num_splits > 1) {
-      first = split * p.split_tokens;
+      first = run_base(p.window_runs ? p.window : 0, pos0) + split * p.split_tokens;
       last = first + p.split_tokens;
     }
     lo = max(p.window > 0 ? max(pos0 - p.window + 1, 0) : 0, first);
@@ -191,7 +198,7 @@ __device__ __forceinline__ void load_tile(const AttnParams& p, const __nv_bfloat
       const int page_index = kpos >> p.page_shift;
       const int page = page_index < p.max_pages ? table[page_index] : -1;
       if (page >= 0 && page < p.num_pages) {
-        src = pages + ((((size_t)page * p.kv_heads + kvh) << p.page_shift) + (kpos & (p.page_size - 1))) * (size_t)pitch + part * 8;
+        src = pages + ((((size_t)page * p.kv_pool + (p.kv_pool == 1 ? 0 : kvh)) << p.page_shift) + (kpos & (p.page_size - 1))) * (size_t)pitch + part * 8;
         bytes = 16;
       } else {
         bad_page = true;
@@ -429,6 +436,7 @@ __global__ void __launch_bounds__(NWARPS * 32) attention_mma_kernel(const AttnPa
 constexpr int DEC_WARPS = 4;
 constexpr int DEC_STAGES = 3;
 constexpr int STAGE_ELEMS = BKV * (ROW_ELEMS + V_ROW_ELEMS);   // K tile then V tile
+constexpr int KEYS_STAGE_ELEMS = BKV * ROW_ELEMS;              // values inside the keys: the K tile is both
 
 __global__ void __launch_bounds__(DEC_WARPS * 32) attention_decode_kernel(const AttnParams p) {
   extern __shared__ __align__(16) unsigned char smem_raw[];
@@ -447,7 +455,9 @@ __global__ void __launch_bounds__(DEC_WARPS * 32) attention_decode_kernel(const 
 
   // The page ids of this block's key range, fetched once: the copy loops then index shared memory.
   // (The staged row is addressed like the global one, so ids before first_page are never read.)
-  int* local_table = reinterpret_cast<int*>(smem_raw + (size_t)DEC_STAGES * STAGE_ELEMS * sizeof(__nv_bfloat16));
+  const int stage_elems = p.v_in_keys ? KEYS_STAGE_ELEMS : STAGE_ELEMS;
+  const int v_row = p.v_in_keys ? ROW_ELEMS : V_ROW_ELEMS;
+  int* local_table = reinterpret_cast<int*>(smem_raw + (size_t)DEC_STAGES * stage_elems * sizeof(__nv_bfloat16));
   const int first_page = keys.probe(keys.start(0)) >> p.page_shift, last_page = (hi - 1) >> p.page_shift;
   for (int i = first_page + tid; i <= last_page; i += DEC_WARPS * 32)
     local_table[i - first_page] = i < p.max_pages ? p.block_table[(size_t)seq * p.max_pages + i] : -1;
@@ -479,8 +489,9 @@ __global__ void __launch_bounds__(DEC_WARPS * 32) attention_decode_kernel(const 
 #pragma unroll
   for (int s = 0; s < DEC_STAGES - 1; ++s) {
     if (s < num_tiles) {
-      load_tile<DEC_WARPS>(p, p.k_pages, table, kvh, stages + s * STAGE_ELEMS, keys.start(s), keys, bad_page);
-      load_tile<DEC_WARPS, DV>(p, p.v_pages, table, kvh, stages + s * STAGE_ELEMS + BKV * ROW_ELEMS, keys.start(s), keys, bad_page, p.v_pitch);
+      load_tile<DEC_WARPS>(p, p.k_pages, table, kvh, stages + s * stage_elems, keys.start(s), keys, bad_page);
+      if (!p.v_in_keys)
+        load_tile<DEC_WARPS, DV>(p, p.v_pages, table, kvh, stages + s * stage_elems + BKV * ROW_ELEMS, keys.start(s), keys, bad_page, p.v_pitch);
     }
     cp_async_commit();
   }
@@ -490,14 +501,15 @@ __global__ void __launch_bounds__(DEC_WARPS * 32) attention_decode_kernel(const 
     {
       const int next = it + DEC_STAGES - 1;
       if (next < num_tiles) {
-        __nv_bfloat16* dst = stages + (next % DEC_STAGES) * STAGE_ELEMS;
+        __nv_bfloat16* dst = stages + (next % DEC_STAGES) * stage_elems;
         load_tile<DEC_WARPS>(p, p.k_pages, table, kvh, dst, keys.start(next), keys, bad_page);
-        load_tile<DEC_WARPS, DV>(p, p.v_pages, table, kvh, dst + BKV * ROW_ELEMS, keys.start(next), keys, bad_page, p.v_pitch);
+        if (!p.v_in_keys)
+          load_tile<DEC_WARPS, DV>(p, p.v_pages, table, kvh, dst + BKV * ROW_ELEMS, keys.start(next), keys, bad_page, p.v_pitch);
       }
       cp_async_commit();
     }
-    const __nv_bfloat16* tK = stages + (it % DEC_STAGES) * STAGE_ELEMS;
-    const __nv_bfloat16* tV = tK + BKV * ROW_ELEMS;
+    const __nv_bfloat16* tK = stages + (it % DEC_STAGES) * stage_elems;
+    const __nv_bfloat16* tV = p.v_in_keys ? tK : tK + BKV * ROW_ELEMS;
     const int k0 = keys.start(it) + warp * 16;          // this warp's 16 positions
     if (k0 >= hi || (k0 + 16 <= lo && k0 >= keys.keep)) continue;   // nothing visible in this slice (warp-uniform)
 
@@ -570,7 +582,7 @@ __global__ void __launch_bounds__(DEC_WARPS * 32) attention_decode_kernel(const 
       const int key = warp * 16 + (mi & 1) * 8 + (lane & 7);
       const int d = (dt + (mi >> 1)) * 8;
       uint32_t r0, r1, r2, r3;
-      ldmatrix_x4_trans(smem_u32(tV + key * V_ROW_ELEMS + d), r0, r1, r2, r3);
+      ldmatrix_x4_trans(smem_u32(tV + key * v_row + d), r0, r1, r2, r3);
       mma_bf16(o_acc[dt], pf, r0, r1);
       mma_bf16(o_acc[dt + 1], pf, r2, r3);
     }
@@ -1273,7 +1285,8 @@ __global__ void attention_merge_kernel(const float* __restrict__ partial_o, cons
                                        const int* __restrict__ positions, __nv_bfloat16* __restrict__ out,
                                        int out_stride, int total_tokens, int heads, int window, int split_tokens,
                                        int num_splits, int first_token, const float* __restrict__ sink, int keep_first,
-                                       const __nv_bfloat16* __restrict__ gate, int gate_stride, int gate_elements) {
+                                       const __nv_bfloat16* __restrict__ gate, int gate_stride, int gate_elements,
+                                       int window_runs) {
   pdl_trigger();
   const int t = blockIdx.x + first_token, h = blockIdx.y;
   const int pos = positions[t];                                     // given to the step: not the previous kernel's work
@@ -1292,9 +1305,10 @@ __global__ void attention_merge_kernel(const float* __restrict__ partial_o, cons
     for (int i = 0; i < HELD; ++i)
       ml[i] = i < num_splits ? *reinterpret_cast<const float2*>(partial_ml + ((size_t)i * stride + slot0) * 2)
                              : make_float2(-INFINITY, 0.0f);
+    const int base = run_base(window_runs ? window : 0, pos);
     const int first_key = window > 0 ? max(pos - window + 1, 0) : 0;
-    const int s_lo = first_key / split_tokens;
-    const int s_hi = min(pos / split_tokens, num_splits - 1);
+    const int s_lo = (first_key - base) / split_tokens;
+    const int s_hi = min((pos - base) / split_tokens, num_splits - 1);
     for (int d = threadIdx.x; d < DV; d += blockDim.x) {
       float o[HELD];
 #pragma unroll
@@ -1321,9 +1335,10 @@ __global__ void attention_merge_kernel(const float* __restrict__ partial_o, cons
     }
     return;
   }
+  const int base = run_base(window_runs ? window : 0, pos);
   const int first_key = window > 0 ? max(pos - window + 1, 0) : 0;
-  const int s_lo = first_key / split_tokens;
-  const int s_hi = min(pos / split_tokens, num_splits - 1);
+  const int s_lo = (first_key - base) / split_tokens;
+  const int s_hi = min((pos - base) / split_tokens, num_splits - 1);
   // the runs of the kept first tokens, then those of the window
   const int kept_runs = min(s_lo, (keep_first + split_tokens - 1) / split_tokens);
   const int skipped = s_lo - kept_runs;
@@ -1361,7 +1376,7 @@ void launch_merge(const AttnParams& p, const int* positions, int first_token, cu
   auto run = [&](auto kernel) {
     tge_launch(kernel, grid, threads, 0, stream, (const float*)p.partial_o, (const float*)p.partial_ml, positions, p.out, p.out_stride,
                p.total_tokens, p.heads, p.window, p.split_tokens, p.num_splits, first_token, p.sink, p.keep_first, p.gate,
-               p.gate_stride, p.gate_elements);
+               p.gate_stride, p.gate_elements, p.window_runs);
   };
   if (p.num_splits <= 16) run(attention_merge_kernel<16>);
   else run(attention_merge_kernel<48>);
@@ -1407,7 +1422,7 @@ static int attention_dispatch(const void* q, int q_stride, const void* k_pages, 
                               int kv_heads, float scale, int window, int split_tokens, float* scratch, int* status,
                               int first_token, const float* sink, int leave_states, int v_pitch, const float* dist_bias,
                               int dist_span, int keep_first, const void* gate, int gate_stride, int gate_elements,
-                              cudaStream_t stream) {
+                              int shared_keys, cudaStream_t stream) {
   TGE_REQUIRE(tokens >= 0 && num_seqs >= 0, "attention_mma: negative sizes");
   TGE_REQUIRE(dist_bias == nullptr || (dist_span > 0 && scale != 0.0f), "attention_mma: a bias by distance needs its span");
   TGE_REQUIRE(heads > 0 && kv_heads > 0 && heads % kv_heads == 0,
@@ -1438,6 +1453,11 @@ static int attention_dispatch(const void* q, int q_stride, const void* k_pages, 
   TGE_REQUIRE(v_pitch >= DV && v_pitch % 8 == 0, "attention_mma: a value pitch of %d (values of %d) must be a multiple of 8", v_pitch, DV);
   TGE_REQUIRE(v_pitch == DV || !(TGE_TMA_KERNELS), "attention_mma: values inside the keys' entries are not served at equal sizes");
   p.v_pitch = v_pitch;
+  p.v_in_keys = v_pitch != DV && k_pages == v_pages;
+  // keys that all runs of heads share are a latent cache's entries, read by single tokens
+  const bool single = max_q_len <= 1 && tokens == num_seqs && group <= 16;
+  TGE_REQUIRE(!shared_keys || (single && p.v_in_keys), "attention_mma: runs of heads over the same keys are for single tokens and values inside the keys");
+  p.kv_pool = shared_keys ? 1 : kv_heads;
   p.q_stride = q_stride; p.out_stride = out_stride;
   p.max_pages = max_pages; p.num_pages = num_pages; p.page_size = page_size;
   p.page_shift = 0;
@@ -1449,8 +1469,11 @@ static int attention_dispatch(const void* q, int q_stride, const void* k_pages, 
   p.window = window;
   p.scale_log2 = scale * 1.4426950408889634f;
   int num_splits = 1;
-  if (split_tokens > 0 && max_ctx_len > split_tokens) num_splits = (max_ctx_len + split_tokens - 1) / split_tokens;
-  p.split_tokens = split_tokens > 0 ? split_tokens : max_ctx_len;
+  // a single token's window covers so many positions from the start of its first tile on, wherever it lies
+  p.window_runs = single && window > 0 && p.keep_first == 0 && !leave_states;
+  const int key_span = p.window_runs && window < max_ctx_len - (BKV - 1) ? window + BKV - 1 : max_ctx_len;
+  if (split_tokens > 0 && key_span > split_tokens) num_splits = (key_span + split_tokens - 1) / split_tokens;
+  p.split_tokens = num_splits > 1 ? split_tokens : max_ctx_len;
   p.num_splits = num_splits;
   TGE_REQUIRE(num_splits == 1 || scratch != nullptr, "attention_mma: %d splits need scratch memory", num_splits);
   TGE_REQUIRE(!leave_states || num_splits > 1, "attention_mma: states are left unmerged only when the keys are cut");
@@ -1462,7 +1485,7 @@ static int attention_dispatch(const void* q, int q_stride, const void* k_pages, 
     const CUtensorMap* map_k = pool_map(k_pages, num_pages, kv_heads, page_size);
     const CUtensorMap* map_v = pool_map(v_pages, num_pages, kv_heads, page_size);
     if (!map_k || !map_v) return -3;
-    const int range = (num_splits > 1 ? p.split_tokens : max_ctx_len) + 2 * BKV;
+    const int range = (num_splits > 1 ? p.split_tokens : key_span) + 2 * BKV;
     // No more blocks than SMs, each with many keys: a block has its SM to itself and runs two groups of warps on
     // alternate tiles (batch 32 at context 2,048, not cut: 3.82 -> 3.66 ms per step).  With few tiles per block the
     // second group only adds to what has to be set up and merged (batch 4, nine splits of 256 keys: 2.95 -> 3.10).
@@ -1471,7 +1494,7 @@ static int attention_dispatch(const void* q, int q_stride, const void* k_pages, 
       return 1024 + (size_t)ring * TMA_STAGE_BYTES + 64 + ((size_t)(range >> p.page_shift) + 2) * sizeof(int);
     };
     const bool two_groups = two_ok && (long long)num_seqs * kv_heads * num_splits <= tge_sm_count() &&
-                            (num_splits > 1 ? p.split_tokens : max_ctx_len) >= 1536 && smem_of(4) <= 227 * 1024;
+                            (num_splits > 1 ? p.split_tokens : key_span) >= 1536 && smem_of(4) <= 227 * 1024;
     const int stages = two_groups ? 4 : DEC_STAGES;
     const size_t smem = smem_of(stages);
     TGE_REQUIRE(smem <= 227 * 1024, "attention_decode: %d keys per block need %zu bytes of shared memory; use smaller splits", range, smem);
@@ -1502,8 +1525,9 @@ static int attention_dispatch(const void* q, int q_stride, const void* k_pages, 
 #endif
   if (max_q_len <= 1 && tokens == num_seqs && group <= 16) {
     // stages, then one page id per page of the longest key range a block can own
-    const int range = num_splits > 1 ? p.split_tokens : max_ctx_len;
-    const size_t smem = (size_t)DEC_STAGES * STAGE_ELEMS * sizeof(__nv_bfloat16) + ((size_t)(range >> p.page_shift) + 2) * sizeof(int);
+    const int range = (num_splits > 1 ? p.split_tokens : key_span) + BKV;
+    const size_t smem = (size_t)DEC_STAGES * (p.v_in_keys ? KEYS_STAGE_ELEMS : STAGE_ELEMS) * sizeof(__nv_bfloat16) +
+                        ((size_t)(range >> p.page_shift) + 2) * sizeof(int);
     TGE_REQUIRE(smem <= 227 * 1024, "attention_decode: %d keys per block need %zu bytes of shared memory; use smaller splits", range, smem);
     static size_t configured = 0;
     if (smem > configured) {
@@ -1635,7 +1659,9 @@ static int attention_dispatch(const void* q, int q_stride, const void* k_pages, 
 // key n positions back, entry min(n, dist_span - 1) of the head's row; every kernel adds it where it scales its scores.
 // `keep_first` (with a window): the first so many positions stay visible beside the window.  `gate` (bfloat16 [tokens,
 // gate_stride], or null): logits of one gate per token and head; whoever writes a head's output multiplies it by their
-// logistic function.  `gate_elements`: one gate per number of a head's output instead, [tokens, heads * DV].
+// logistic function.  `shared_keys`: for single tokens whose values lie inside the keys, all kv_heads runs of heads read the one
+// key/value head that the pages hold.  Single tokens over a window (without kept first positions): split_tokens cuts the window's
+// span, from its first tile on.  `gate_elements`: one gate per number of a head's output instead, [tokens, heads * DV].
 TGE_API int tge_attention_mma(const void* q, int q_stride, const void* k_pages, const void* v_pages,
                               const int* block_table, int max_pages, int num_pages, int page_size,
                               const int* q_start, const int* start_pos, const int* positions, int num_seqs,
@@ -1643,7 +1669,7 @@ TGE_API int tge_attention_mma(const void* q, int q_stride, const void* k_pages, 
                               int kv_heads, float scale, int window, int split_tokens, float* scratch, int* status,
                               int decode_prefix, int prefix_split_tokens, const float* sink, int leave_states,
                               int v_pitch, const float* dist_bias, int dist_span, int keep_first, const void* gate,
-                              int gate_stride, int gate_elements, cudaStream_t stream) {
+                              int gate_stride, int gate_elements, int shared_keys, cudaStream_t stream) {
   TGE_REQUIRE(decode_prefix >= 0 && decode_prefix <= num_seqs, "attention_mma: %d leading single tokens of %d sequences",
               decode_prefix, num_seqs);
   TGE_REQUIRE(prefix_split_tokens >= 0 && prefix_split_tokens % BKV == 0,
@@ -1651,16 +1677,16 @@ TGE_API int tge_attention_mma(const void* q, int q_stride, const void* k_pages, 
   if (decode_prefix == 0 || max_q_len <= 1 || decode_prefix == num_seqs || kv_heads <= 0 || heads / kv_heads > 16)
     return attention_dispatch(q, q_stride, k_pages, v_pages, block_table, max_pages, num_pages, page_size, q_start, start_pos,
                               positions, num_seqs, tokens, max_q_len, max_ctx_len, out, out_stride, heads, kv_heads, scale,
-                              window, split_tokens, scratch, status, 0, sink, leave_states, v_pitch, dist_bias, dist_span, keep_first, gate, gate_stride, gate_elements, stream);
+                              window, split_tokens, scratch, status, 0, sink, leave_states, v_pitch, dist_bias, dist_span, keep_first, gate, gate_stride, gate_elements, shared_keys, stream);
   const int first = attention_dispatch(q, q_stride, k_pages, v_pages, block_table, max_pages, num_pages, page_size, q_start,
                                        start_pos, positions, decode_prefix, decode_prefix, 1, max_ctx_len, out, out_stride,
                                        heads, kv_heads, scale, window, prefix_split_tokens, scratch, status, 0, sink, leave_states, v_pitch, dist_bias,
-                                       dist_span, keep_first, gate, gate_stride, gate_elements, stream);
+                                       dist_span, keep_first, gate, gate_stride, gate_elements, shared_keys, stream);
   if (first < 0) return first;
   const int rest = attention_dispatch(q, q_stride, k_pages, v_pages, block_table + (size_t)decode_prefix * max_pages, max_pages,
                                       num_pages, page_size, q_start + decode_prefix, start_pos + decode_prefix, positions,
                                       num_seqs - decode_prefix, tokens, max_q_len, max_ctx_len, out, out_stride, heads,
                                       kv_heads, scale, window, split_tokens, scratch, status, decode_prefix, sink, leave_states, v_pitch, dist_bias,
-                                      dist_span, keep_first, gate, gate_stride, gate_elements, stream);
+                                      dist_span, keep_first, gate, gate_stride, gate_elements, shared_keys, stream);
   return rest < 0 ? rest : first + rest;
 }

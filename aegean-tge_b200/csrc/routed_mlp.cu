@@ -90,40 +90,87 @@ __global__ void __launch_bounds__(128) router_topk_kernel(const float* __restric
   __syncwarp();
   if (group_count > 1 && group_keep < group_count) {
     const int per = outputs / group_count;
-    for (int g = 0; g < group_count; ++g) {
-      float best = -INFINITY, second = -INFINITY;
-      for (int i = lane; i < per; i += 32) {
-        const float v = choice[g * per + i];
-        second = fmaxf(second, fminf(best, v));
-        best = fmaxf(best, v);
-      }
-      if (group_pairs) {
-        // the two largest of the group, added (a group of one has only the one)
-#pragma unroll
-        for (int offset = 16; offset > 0; offset >>= 1) {
-          const float other = __shfl_xor_sync(0xffffffffu, best, offset), third = __shfl_xor_sync(0xffffffffu, second, offset);
-          second = fmaxf(fminf(best, other), fmaxf(second, third));
-          best = fmaxf(best, other);
+    if (per <= 32) {
+      // small groups: a lane takes a group, and keeps it if fewer than group_keep others come before it
+      for (int g = lane; g < group_count; g += 32) {
+        float best = -INFINITY, second = -INFINITY;
+        for (int i = 0; i < per; ++i) {
+          const float v = choice[g * per + i];
+          second = fmaxf(second, fminf(best, v));
+          best = fmaxf(best, v);
         }
-        if (per > 1) best += second;
-      } else {
-        best = warp_max(best);
+        group_best[g] = group_pairs && per > 1 ? best + second : best;
       }
-      if (lane == 0) { group_best[g] = best; kept[g] = 0.0f; }
-    }
-    __syncwarp();
-    for (int n = 0; n < group_keep; ++n) {
-      float best;
-      int where;
-      warp_argmax(group_best, group_count, lane, best, where);
-      if (lane == 0 && where < group_count) { kept[where] = 1.0f; group_best[where] = -INFINITY; }
       __syncwarp();
+      for (int g = lane; g < group_count; g += 32) {
+        const float own = group_best[g];
+        int before = 0;
+        for (int other = 0; other < group_count; ++other) {
+          const float v = group_best[other];
+          before += v > own || (v == own && other < g);
+        }
+        kept[g] = before < group_keep ? 1.0f : 0.0f;
+      }
+      __syncwarp();
+    } else {
+      for (int g = 0; g < group_count; ++g) {
+        float best = -INFINITY, second = -INFINITY;
+        for (int i = lane; i < per; i += 32) {
+          const float v = choice[g * per + i];
+          second = fmaxf(second, fminf(best, v));
+          best = fmaxf(best, v);
+        }
+        if (group_pairs) {
+          // the two largest of the group, added (a group of one has only the one)
+#pragma unroll
+          for (int offset = 16; offset > 0; offset >>= 1) {
+            const float other = __shfl_xor_sync(0xffffffffu, best, offset), third = __shfl_xor_sync(0xffffffffu, second, offset);
+            second = fmaxf(fminf(best, other), fmaxf(second, third));
+            best = fmaxf(best, other);
+          }
+          if (per > 1) best += second;
+        } else {
+          best = warp_max(best);
+        }
+        if (lane == 0) { group_best[g] = best; kept[g] = 0.0f; }
+      }
+      __syncwarp();
+      for (int n = 0; n < group_keep; ++n) {
+        float best;
+        int where;
+        warp_argmax(group_best, group_count, lane, best, where);
+        if (lane == 0 && where < group_count) { kept[where] = 1.0f; group_best[where] = -INFINITY; }
+        __syncwarp();
+      }
     }
     for (int i = lane; i < outputs; i += 32)
       if (kept[i / per] == 0.0f) choice[i] = -INFINITY;
     __syncwarp();
   }
   float chosen_sum = 0.0f;
+  if (outputs <= 64) {
+    // few outputs: every lane counts how many come before its own; the chosen ones meet in order of their rank
+    int* order = reinterpret_cast<int*>(group_best);               // the groups are settled
+    for (int n = lane; n < top; n += 32) order[n] = 0;
+    __syncwarp();
+    for (int i = lane; i < outputs; i += 32) {
+      const float own = choice[i];
+      int before = 0;
+      for (int other = 0; other < outputs; ++other) {
+        const float v = choice[other];
+        before += v > own || (v == own && other < i);
+      }
+      if (before < top) order[before] = i;
+    }
+    __syncwarp();
+    for (int n = 0; n < top; ++n) chosen_sum += score[order[n]];
+    chosen_sum = over_sum ? chosen_sum + 1e-20f : 1.0f;
+    for (int n = lane; n < top; n += 32) {
+      ids[(size_t)t * top + n] = order[n];
+      weights[(size_t)t * top + n] = score[order[n]] / chosen_sum * factor;
+    }
+    return;
+  }
   for (int n = 0; n < top; ++n) {
     float best;
     int where;

@@ -1075,6 +1075,109 @@ TGE_API int tge_gated_norm(const float* o, const void* gate, int is_bf16, long l
   return tge_launched("gated_norm", 1);
 }
 
+namespace {
+
+constexpr int NRV_THREADS = 256;
+
+// The same without a convolution, on eight bfloat16 at a time (head sizes and row strides multiples of 8, half the rotated
+// numbers as well): `lanes` lanes (a power of two, one per 16 bytes of a head) share a head; the number a rotated one is
+// paired with comes from the lane half / 8 away.
+__global__ void __launch_bounds__(NRV_THREADS) norm_rope_store_vec_kernel(
+    const __nv_bfloat16* __restrict__ raw, long long ld, const float* __restrict__ q_norm, const float* __restrict__ k_norm,
+    float eps, const float* __restrict__ cos_table, const float* __restrict__ sin_table, int table_positions, int rotary,
+    const int* __restrict__ positions, const int* __restrict__ seq_of_token, const int* __restrict__ block_table, int max_pages,
+    __nv_bfloat16* __restrict__ k_pages, __nv_bfloat16* __restrict__ v_pages, int num_pages, int page_size,
+    __nv_bfloat16* __restrict__ q_out, long long ld_q, int heads, int kv_heads, int dim, int vdim, int store_kv, int norm_last,
+    int lanes, int* status) {
+  pdl_trigger();
+  const int t = blockIdx.x;
+  const int pos = positions[t];
+  bool store = store_kv != 0;
+  size_t k_base = 0, v_base = 0;
+  if (store) {
+    const int page_index = pos / page_size;
+    const int page = (pos >= 0 && page_index < max_pages) ? block_table[(size_t)seq_of_token[t] * max_pages + page_index] : -1;
+    if (page < 0 || page >= num_pages) {
+      if (threadIdx.x == 0) atomicOr(status, TGE_STATUS_BAD_PAGE);
+      store = false;
+    } else {
+      k_base = ((size_t)page * kv_heads * page_size + (pos % page_size)) * dim;
+      v_base = ((size_t)page * kv_heads * page_size + (pos % page_size)) * vdim;
+    }
+  }
+  int at = pos;
+  if (rotary > 0 && (pos < 0 || pos >= table_positions)) {
+    if (threadIdx.x == 0) atomicOr(status, TGE_STATUS_BAD_ROW);
+    at = 0;
+  }
+  const int per_head = dim / 8, total = heads + kv_heads;
+  const int mine = threadIdx.x & (lanes - 1), groups = NRV_THREADS / lanes;
+  const int half = rotary >> 1, away = half >> 3;
+  const bool turns = mine * 8 < rotary, low = mine < away;
+  // a lane turns the same pairs in every head: its cosines and sines are read once
+  float cs[8], sn[8];
+  if (turns) {
+    const size_t entry = (size_t)at * half + (low ? mine : mine - away) * 8;
+#pragma unroll
+    for (int e = 0; e < 8; e += 4) {
+      const float4 c = *reinterpret_cast<const float4*>(cos_table + entry + e), s = *reinterpret_cast<const float4*>(sin_table + entry + e);
+      cs[e] = c.x; cs[e + 1] = c.y; cs[e + 2] = c.z; cs[e + 3] = c.w;
+      sn[e] = s.x; sn[e + 1] = s.y; sn[e + 2] = s.z; sn[e + 3] = s.w;
+    }
+  }
+  pdl_wait();
+  const uint4* row = reinterpret_cast<const uint4*>(raw + (size_t)t * ld);
+  for (int base = 0; base < total; base += groups) {
+    const int unit = base + (int)threadIdx.x / lanes;
+    const bool valid = unit < total && mine < per_head;
+    uint4 packed = valid ? row[unit * per_head + mine] : make_uint4(0u, 0u, 0u, 0u);
+    __nv_bfloat162* two = reinterpret_cast<__nv_bfloat162*>(&packed);
+    float f[8];
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      const float2 v = __bfloat1622float2(two[e]);
+      f[2 * e] = v.x;
+      f[2 * e + 1] = v.y;
+    }
+    const float* weight = unit < heads ? q_norm : k_norm;
+    auto norm = [&](bool wanted) {
+      float sum = 0.0f;
+#pragma unroll
+      for (int e = 0; e < 8; ++e) sum = fmaf(f[e], f[e], sum);
+      for (int step = lanes >> 1; step > 0; step >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, step);
+      const float scale = 1.0f / sqrtf(sum / (float)dim + eps);
+      if (wanted && valid) {
+#pragma unroll
+        for (int e = 0; e < 8; ++e) f[e] *= scale * (weight != nullptr ? weight[mine * 8 + e] : 1.0f);
+      }
+    };
+    if (!norm_last && (q_norm != nullptr || k_norm != nullptr)) norm(weight != nullptr);      // the same for the whole block
+    if (rotary > 0) {
+      const int group_first = (threadIdx.x & 31) & ~(lanes - 1);
+      const int from = group_first + (turns ? (low ? mine + away : mine - away) : mine);
+#pragma unroll
+      for (int e = 0; e < 8; ++e) {
+        const float other = __shfl_sync(0xffffffffu, f[e], from);
+        if (turns) f[e] = low ? f[e] * cs[e] - other * sn[e] : f[e] * cs[e] + other * sn[e];
+      }
+    }
+    if (norm_last) norm(true);
+    if (!valid) continue;
+#pragma unroll
+    for (int e = 0; e < 4; ++e) two[e] = __floats2bfloat162_rn(f[2 * e], f[2 * e + 1]);
+    if (unit < heads) *reinterpret_cast<uint4*>(q_out + (size_t)t * ld_q + (size_t)unit * dim + mine * 8) = packed;
+    else if (store) *reinterpret_cast<uint4*>(k_pages + k_base + (size_t)(unit - heads) * page_size * dim + mine * 8) = packed;
+  }
+  if (!store) return;
+  const uint4* v_row = row + total * per_head;
+  for (int u = threadIdx.x; u < kv_heads * vdim / 8; u += NRV_THREADS) {
+    const int h = u * 8 / vdim, d = u * 8 - h * vdim;
+    *reinterpret_cast<uint4*>(v_pages + v_base + (size_t)h * page_size * vdim + d) = v_row[u];
+  }
+}
+
+}  // namespace
+
 TGE_API int tge_conv_norm_rope_store(const void* raw, int is_bf16, long long ld, const float* conv_w, int taps,
                                      float* conv_state, const int* slots, const int* q_start, const float* q_norm,
                                      const float* k_norm, float eps, const float* cos_table, const float* sin_table,
@@ -1097,6 +1200,16 @@ TGE_API int tge_conv_norm_rope_store(const void* raw, int is_bf16, long long ld,
   const int channels = (heads + kv_heads) * dim + kv_heads * vdim;
   dim3 grid(tokens, (units + 3) / 4);
   int launched = 1;
+  if (is_bf16 && taps == 0 && dim % 8 == 0 && vdim % 8 == 0 && rotary % 16 == 0 && ld % 8 == 0 && ld_q % 8 == 0 &&
+      (((uintptr_t)raw | (uintptr_t)q_out | (uintptr_t)k_pages | (uintptr_t)v_pages | (uintptr_t)cos_table | (uintptr_t)sin_table) & 15) == 0) {
+    int lanes = 1;
+    while (lanes * 8 < dim) lanes *= 2;
+    tge_launch(norm_rope_store_vec_kernel, dim3(tokens), dim3(NRV_THREADS), 0, stream, (const __nv_bfloat16*)raw, ld, q_norm, k_norm,
+               eps, cos_table, sin_table, table_positions, rotary, positions, seq_of_token, block_table, max_pages,
+               (__nv_bfloat16*)k_pages, (__nv_bfloat16*)v_pages, num_pages, page_size, (__nv_bfloat16*)q_out, ld_q, heads, kv_heads,
+               dim, vdim, store, norm_last, lanes, status);
+    return tge_launched("norm_rope_store_vec", 1);
+  }
   if (is_bf16) {
     tge_launch(conv_norm_rope_store_kernel<__nv_bfloat16>, grid, dim3(128), 0, stream,
         (const __nv_bfloat16*)raw, ld, conv_w, taps, conv_state, slots, q_start, q_norm, k_norm, eps, cos_table, sin_table,

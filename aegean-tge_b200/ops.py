@@ -198,7 +198,7 @@ def attention_lib(head_dim: int, value_dim: int = 0) -> ctypes.CDLL:
         _declare(lib, "tge_attention_mma", [_c_ptr, _c_int, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_int, _c_int, _c_ptr,
                                             _c_ptr, _c_ptr, _c_int, _c_int, _c_int, _c_int, _c_ptr, _c_int, _c_int,
                                             _c_int, _c_float, _c_int, _c_int, _c_ptr, _c_ptr, _c_int, _c_int, _c_ptr,
-                                            _c_int, _c_int, _c_ptr, _c_int, _c_int, _c_ptr, _c_int, _c_int, _c_ptr])
+                                            _c_int, _c_int, _c_ptr, _c_int, _c_int, _c_ptr, _c_int, _c_int, _c_int, _c_ptr])
         lib.tge_attention_mma_scratch_floats.argtypes = [_c_int, _c_int, _c_int]
         lib.tge_attention_mma_scratch_floats.restype = _c_ll
         if lib.tge_attention_mma_head_dim() != head_dim or lib.tge_attention_mma_value_dim() != value_dim:
@@ -772,7 +772,8 @@ def attention(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tensor, blo
               sink: Optional[torch.Tensor] = None, pool: int = 0, pooled_k: Optional[torch.Tensor] = None,
               pooled_v: Optional[torch.Tensor] = None, pool_table: Optional[torch.Tensor] = None,
               values_in_keys: int = 0, dist_bias: Optional[torch.Tensor] = None, keep_first: int = 0,
-              gate: Optional[torch.Tensor] = None) -> torch.Tensor:
+              gate: Optional[torch.Tensor] = None,
+              shared_keys: bool = False) -> torch.Tensor:
     """Paged causal attention of a flat batch of portions.
 
     q: [T, >= heads*head_dim] (dense rows, any row stride) holding rotated queries;
@@ -796,6 +797,8 @@ def attention(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tensor, blo
     ``keep_first`` (with a window): the first so many positions of a request stay visible beside the window.
     ``gate`` (run dtype [T, heads], dense rows, any row stride): logits of one gate per head; whoever writes a head's
     output multiplies it by their logistic function.  [T, heads * value_dim]: one gate per number of the output.
+    ``shared_keys`` (single tokens, values inside the keys): the heads go in ``kv_heads`` equal runs that all read the one
+    key/value head of the pages, one block per run; for the tensor-core kernels only.
     """
     v_pitch = 0
     if values_in_keys:
@@ -811,7 +814,7 @@ def attention(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tensor, blo
                     ("positions", positions), ("seq_of_token", seq_of_token)):
         _want(t, name, torch.int32)
     num_pages, page_kv, page_size, page_hd = k_pages.shape
-    if (page_kv != kv_heads or page_hd != head_dim or v_pages.dim() != 4
+    if (page_kv != (1 if shared_keys else kv_heads) or page_hd != head_dim or v_pages.dim() != 4
             or tuple(v_pages.shape[:3]) != tuple(k_pages.shape[:3])):
         raise KernelError(f"pages must be [pages, {kv_heads}, page_size, {head_dim}] and the like for the values, "
                           f"got {tuple(k_pages.shape)} and {tuple(v_pages.shape)}")
@@ -866,6 +869,8 @@ def attention(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tensor, blo
     use_mma = (q.dtype == torch.bfloat16 and USE_MMA_ATTENTION and not force_simt and pairs_ok
                and mma_attention_supports(head_dim, heads, kv_heads, page_size, value_dim)
                and not (v_pitch and value_dim == head_dim))
+    if shared_keys and not (use_mma and max_q_len <= 1 and values_in_keys and heads // kv_heads <= 16):
+        raise KernelError("attention: runs of heads over the same keys are for single tokens on the tensor-core kernels")
     if use_mma:
         lib = attention_lib(head_dim, value_dim)
         prefix = decode_prefix if decode_prefix >= MIN_DECODE_PREFIX and max_q_len > 1 and not pool else 0
@@ -888,8 +893,11 @@ def attention(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tensor, blo
             # the single tokens at the head of a mixed step are a decode batch of their own: a few of them deep in
             # long contexts want their keys cut although the portions beside them do not
             prefix_split = choose_attention_split(prefix, prefix, 1, span, heads, kv_heads, bound=span) if prefix else 0
-        count = lambda split: 1 if split == 0 or max_ctx_len <= split else -(-max_ctx_len // split)
-        splits = max(count(split_tokens), count(prefix_split) if prefix else 1)
+        # single tokens over a window cut the window's span (from its first tile on), everything else the whole context
+        narrow = heads // kv_heads <= 16 and window > 0 and keep_first == 0 and not pool
+        one_window = min(max_ctx_len, window + 63) if narrow else max_ctx_len
+        count = lambda split, reach: 1 if split == 0 or reach <= split else -(-reach // split)
+        splits = max(count(split_tokens, one_window if max_q_len <= 1 else max_ctx_len), count(prefix_split, one_window) if prefix else 1)
         need = lib.tge_attention_mma_scratch_floats(tokens, heads, splits)
         scratch = scratch_floats(need) if need > 0 else None
         _check(lib.tge_attention_mma(q.data_ptr(), q_stride, k_pages.data_ptr(), v_pages.data_ptr(),
@@ -898,7 +906,7 @@ def attention(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tensor, blo
                                      max_ctx_len, out.data_ptr(), out_stride, heads, kv_heads, float(scale), window,
                                      split_tokens, _ptr(scratch), status_word().data_ptr(), prefix, prefix_split,
                                      _ptr(sink), int(bool(pool)), v_pitch, _ptr(dist_bias), dist_span,
-                                     keep_first, _ptr(gate), gate_stride, gate_elements, _stream()), lib)
+                                     keep_first, _ptr(gate), gate_stride, gate_elements, int(shared_keys), _stream()), lib)
         if pool:
             core_lib = core()
             states = scratch.data_ptr()

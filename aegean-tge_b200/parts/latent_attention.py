@@ -182,10 +182,13 @@ class LatentAttention(Mixer):
             ops.rotate_runs(q[:, self.dim:], per_head, queries[:, self.kv_rank:], self.entry, self.heads, self.rot,
                                    self.cos, self.sin, self.rot_dims, ctx.positions, halves=self.halves)
         # single tokens: the decode kernels take the heads that share a key/value head as the rows of one tile of 16,
-        # so more heads than that go in equal runs of up to 16 (the entries are few bytes; reading them twice is cheap)
-        single = ctx.max_q_len <= 1 and dtype == torch.bfloat16
+        # so more heads than that go in runs of up to 16 (the entries are few bytes; reading them twice is cheap), equal
+        # ones in one launch
+        single = (ctx.max_q_len <= 1 and dtype == torch.bfloat16
+                  and ops.mma_attention_supports(self.entry, min(self.heads, 16), 1, pages.shape[2], self.kv_rank))
         runs = -(-self.heads // 16) if single else 1
         size = -(-self.heads // runs)
+        together = runs > 1 and self.heads % runs == 0 and self.rot > 0 and queries.stride(0) % 2 == 0
         split = ctx.attn_split_tokens
         if single and split == 0 and self.entry > 128:
             # entries this wide leave room for one block of the decode kernel per SM, so the keys are cut into just
@@ -193,15 +196,15 @@ class LatentAttention(Mixer):
             bound = max(ctx.typical_ctx_len or ctx.max_ctx_len, 1)
             if self.window is not None:
                 bound = min(bound, (-(-self.window // 64) + 1) * 64)
-            want = max(_sm_count(h.device) // max(ctx.num_seqs, 1), 1)
+            want = max(_sm_count(h.device) // max(ctx.num_seqs * (runs if together else 1), 1), 1)
             split = max(64 * -(-(-(-bound // want)) // 64), 128)
         attended = torch.empty((tokens, self.heads * self.kv_rank), dtype=dtype, device=h.device)
-        for lo in range(0, self.heads, size):
-            n = min(size, self.heads - lo)
+        for lo in range(0, self.heads, self.heads if together else size):
+            n = self.heads if together else min(size, self.heads - lo)
             ops.attention(queries[:, lo * self.entry:(lo + n) * self.entry], pages, None, table, ctx.q_start, ctx.start_pos,
-                          ctx.positions, ctx.seq_of_token, ctx.num_seqs, ctx.max_q_len, ctx.max_ctx_len, n, 1, self.entry,
+                          ctx.positions, ctx.seq_of_token, ctx.num_seqs, ctx.max_q_len, ctx.max_ctx_len, n, runs if together else 1, self.entry,
                           self.scale, window=self.window or 0, split_tokens=split, typical_ctx_len=ctx.typical_ctx_len,
-                          decode_prefix=ctx.decode_prefix, values_in_keys=self.kv_rank,
+                          decode_prefix=ctx.decode_prefix, values_in_keys=self.kv_rank, shared_keys=together,
                           out=attended[:, lo * self.kv_rank:(lo + n) * self.kv_rank])
         if out is None:
             out = torch.empty((tokens, self.heads * self.vdim), dtype=dtype, device=h.device)
