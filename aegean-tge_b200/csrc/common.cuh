@@ -122,7 +122,7 @@ __device__ __forceinline__ __nv_bfloat16 from_float<__nv_bfloat16>(float v) { re
 // The two usual forms of GELU, in float32.
 __device__ __forceinline__ float gelu_erf(float z) { return 0.5f * z * (1.0f + erff(z * 0.70710678118654752f)); }
 // The erf form for results that are rounded to bfloat16: the normal distribution's tail by the rational
-// approximation erfc(x) ~ t (a1 + t (a2 + t (a3 + t (a4 + t a5)))) exp(-x^2), t = 1 / (1 + p x), x >= 0 (absolute
+// approximation 7.1.26 of Abramowitz and Stegun's handbook, erfc(x) ~ t (a1 + t (a2 + t (a3 + t (a4 + t a5)))) exp(-x^2), t = 1 / (1 + p x), x >= 0 (absolute
 // error below 1.5e-7, a hundredth of a bfloat16 step of the result), with the fast exponential and division:
 // a dozen instructions where erff takes several dozen.  In a product's epilogue that is the difference between
 // an epilogue hidden behind the next tile and one the tensor cores wait for (a 2,048 x 28,416 x 3,584 product:

@@ -54,6 +54,10 @@ __global__ void __launch_bounds__(256) latent_prepare_kernel(
     T* __restrict__ pages, T* __restrict__ q_latent, float* __restrict__ gate, int* status) {
   __shared__ float scratch[32];
   pdl_trigger();
+  // the norms' weights are the model's: asked for before the rows are there
+  for (int i = threadIdx.x * 32; i < q_rank; i += blockDim.x * 32) asm volatile("prefetch.global.L2 [%0];\n" ::"l"(q_weight + i));
+  if (has_kv)
+    for (int i = threadIdx.x * 32; i < kv_rank; i += blockDim.x * 32) asm volatile("prefetch.global.L2 [%0];\n" ::"l"(kv_weight + i));
   pdl_wait();
   const int t = blockIdx.x;
   const float* row = raw + (size_t)t * ld_raw;

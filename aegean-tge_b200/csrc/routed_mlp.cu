@@ -53,7 +53,6 @@ __global__ void __launch_bounds__(128) router_topk_kernel(const float* __restric
                                                           float* __restrict__ weights) {
   extern __shared__ float router_smem[];
   pdl_trigger();
-  pdl_wait();
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int t = blockIdx.x * 4 + warp;
   if (t >= tokens) return;
@@ -61,13 +60,16 @@ __global__ void __launch_bounds__(128) router_topk_kernel(const float* __restric
   float* choice = score + outputs;
   float* group_best = choice + outputs;
   float* kept = group_best + outputs;
+  // the correction is the model's: fetched before the logits are there
+  for (int i = lane; i < outputs; i += 32) choice[i] = correction != nullptr ? correction[i] : 0.0f;
+  pdl_wait();
   const float* z = logits + (size_t)t * ld;
   if (logistic) {
     for (int i = lane; i < outputs; i += 32) {
       const float s = 1.0f / (1.0f + expf(-z[i]));
       score[i] = s;
       // the logits order like the scores and do not saturate (sums of two do not order alike)
-      choice[i] = correction != nullptr ? s + correction[i] : (group_pairs ? s : z[i]);
+      choice[i] = correction != nullptr || group_pairs ? s + choice[i] : z[i];
     }
   } else {
     float m = -INFINITY;
@@ -84,7 +86,7 @@ __global__ void __launch_bounds__(128) router_topk_kernel(const float* __restric
     for (int i = lane; i < outputs; i += 32) {
       const float s = score[i] * inv;
       score[i] = s;
-      choice[i] = s + (correction != nullptr ? correction[i] : 0.0f);
+      choice[i] += s;
     }
   }
   __syncwarp();
