@@ -44,7 +44,8 @@ __device__ __forceinline__ void warp_argmax(const float* values, int n, int lane
   }
 }
 
-// One warp per token.  Shared memory per warp: 4 arrays of `outputs` floats (scores, choice values, group maxima,
+// One warp per token.  Loops over the few outputs stay rolled: in a decode step the weights of a layer pass through the L2
+// between two launches, so every line of instructions is fetched from memory again.  Shared memory per warp: 4 arrays of `outputs` floats (scores, choice values, group maxima,
 // kept flags).
 __global__ void __launch_bounds__(128) router_topk_kernel(const float* __restrict__ logits, long long ld,
                                                           const float* __restrict__ correction, int tokens, int outputs,
@@ -61,10 +62,12 @@ __global__ void __launch_bounds__(128) router_topk_kernel(const float* __restric
   float* group_best = choice + outputs;
   float* kept = group_best + outputs;
   // the correction is the model's: fetched before the logits are there
+#pragma unroll 1
   for (int i = lane; i < outputs; i += 32) choice[i] = correction != nullptr ? correction[i] : 0.0f;
   pdl_wait();
   const float* z = logits + (size_t)t * ld;
   if (logistic) {
+#pragma unroll 1
     for (int i = lane; i < outputs; i += 32) {
       const float s = 1.0f / (1.0f + expf(-z[i]));
       score[i] = s;
@@ -93,9 +96,11 @@ __global__ void __launch_bounds__(128) router_topk_kernel(const float* __restric
   if (group_count > 1 && group_keep < group_count) {
     const int per = outputs / group_count;
     if (per <= 32) {
-      // small groups: a lane takes a group, and keeps it if fewer than group_keep others come before it
+      // small groups: a lane takes a group; an output stays if fewer than group_keep groups come before its own
+#pragma unroll 1
       for (int g = lane; g < group_count; g += 32) {
         float best = -INFINITY, second = -INFINITY;
+#pragma unroll 1
         for (int i = 0; i < per; ++i) {
           const float v = choice[g * per + i];
           second = fmaxf(second, fminf(best, v));
@@ -104,16 +109,18 @@ __global__ void __launch_bounds__(128) router_topk_kernel(const float* __restric
         group_best[g] = group_pairs && per > 1 ? best + second : best;
       }
       __syncwarp();
-      for (int g = lane; g < group_count; g += 32) {
+#pragma unroll 1
+      for (int i = lane; i < outputs; i += 32) {
+        const int g = i / per;
         const float own = group_best[g];
         int before = 0;
+#pragma unroll 1
         for (int other = 0; other < group_count; ++other) {
           const float v = group_best[other];
           before += v > own || (v == own && other < g);
         }
-        kept[g] = before < group_keep ? 1.0f : 0.0f;
+        if (before >= group_keep) choice[i] = -INFINITY;
       }
-      __syncwarp();
     } else {
       for (int g = 0; g < group_count; ++g) {
         float best = -INFINITY, second = -INFINITY;
@@ -144,20 +151,23 @@ __global__ void __launch_bounds__(128) router_topk_kernel(const float* __restric
         if (lane == 0 && where < group_count) { kept[where] = 1.0f; group_best[where] = -INFINITY; }
         __syncwarp();
       }
+      for (int i = lane; i < outputs; i += 32)
+        if (kept[i / per] == 0.0f) choice[i] = -INFINITY;
     }
-    for (int i = lane; i < outputs; i += 32)
-      if (kept[i / per] == 0.0f) choice[i] = -INFINITY;
     __syncwarp();
   }
   float chosen_sum = 0.0f;
   if (outputs <= 64) {
     // few outputs: every lane counts how many come before its own; the chosen ones meet in order of their rank
     int* order = reinterpret_cast<int*>(group_best);               // the groups are settled
+#pragma unroll 1
     for (int n = lane; n < top; n += 32) order[n] = 0;
     __syncwarp();
+#pragma unroll 1
     for (int i = lane; i < outputs; i += 32) {
       const float own = choice[i];
       int before = 0;
+#pragma unroll 1
       for (int other = 0; other < outputs; ++other) {
         const float v = choice[other];
         before += v > own || (v == own && other < i);
@@ -165,8 +175,10 @@ __global__ void __launch_bounds__(128) router_topk_kernel(const float* __restric
       if (before < top) order[before] = i;
     }
     __syncwarp();
+#pragma unroll 1
     for (int n = 0; n < top; ++n) chosen_sum += score[order[n]];
     chosen_sum = over_sum ? chosen_sum + 1e-20f : 1.0f;
+#pragma unroll 1
     for (int n = lane; n < top; n += 32) {
       ids[(size_t)t * top + n] = order[n];
       weights[(size_t)t * top + n] = score[order[n]] / chosen_sum * factor;

@@ -1077,7 +1077,7 @@ TGE_API int tge_gated_norm(const float* o, const void* gate, int is_bf16, long l
 
 namespace {
 
-constexpr int NRV_THREADS = 256;
+constexpr int NRV_THREADS = 512;    // at most
 
 // The same without a convolution, on eight bfloat16 at a time (head sizes and row strides multiples of 8, half the rotated
 // numbers as well): `lanes` lanes (a power of two, one per 16 bytes of a head) share a head; the number a rotated one is
@@ -1111,7 +1111,7 @@ __global__ void __launch_bounds__(NRV_THREADS) norm_rope_store_vec_kernel(
     at = 0;
   }
   const int per_head = dim / 8, total = heads + kv_heads;
-  const int mine = threadIdx.x & (lanes - 1), groups = NRV_THREADS / lanes;
+  const int mine = threadIdx.x & (lanes - 1), groups = blockDim.x / lanes;
   const int half = rotary >> 1, away = half >> 3;
   const bool turns = mine * 8 < rotary, low = mine < away;
   // a lane turns the same pairs in every head: its cosines and sines are read once
@@ -1170,7 +1170,7 @@ __global__ void __launch_bounds__(NRV_THREADS) norm_rope_store_vec_kernel(
   }
   if (!store) return;
   const uint4* v_row = row + total * per_head;
-  for (int u = threadIdx.x; u < kv_heads * vdim / 8; u += NRV_THREADS) {
+  for (int u = threadIdx.x; u < kv_heads * vdim / 8; u += blockDim.x) {
     const int h = u * 8 / vdim, d = u * 8 - h * vdim;
     *reinterpret_cast<uint4*>(v_pages + v_base + (size_t)h * page_size * vdim + d) = v_row[u];
   }
@@ -1204,7 +1204,11 @@ TGE_API int tge_conv_norm_rope_store(const void* raw, int is_bf16, long long ld,
       (((uintptr_t)raw | (uintptr_t)q_out | (uintptr_t)k_pages | (uintptr_t)v_pages | (uintptr_t)cos_table | (uintptr_t)sin_table) & 15) == 0) {
     int lanes = 1;
     while (lanes * 8 < dim) lanes *= 2;
-    tge_launch(norm_rope_store_vec_kernel, dim3(tokens), dim3(NRV_THREADS), 0, stream, (const __nv_bfloat16*)raw, ld, q_norm, k_norm,
+    int threads = ((heads + kv_heads) * lanes + 31) / 32 * 32;
+    // few tokens: all heads of one in a single pass; many: narrower blocks, more of them on an SM
+    const int most = tokens <= 2 * tge_sm_count() ? NRV_THREADS : NRV_THREADS / 2;
+    if (threads > most) threads = most;
+    tge_launch(norm_rope_store_vec_kernel, dim3(tokens), dim3(threads), 0, stream, (const __nv_bfloat16*)raw, ld, q_norm, k_norm,
                eps, cos_table, sin_table, table_positions, rotary, positions, seq_of_token, block_table, max_pages,
                (__nv_bfloat16*)k_pages, (__nv_bfloat16*)v_pages, num_pages, page_size, (__nv_bfloat16*)q_out, ld_q, heads, kv_heads,
                dim, vdim, store, norm_last, lanes, status);
